@@ -2,7 +2,6 @@
 // the KV-cached decode driver. Host logic above the kernels mirrors, in C++, the Rust items
 // cited in include/ferrum_cuda.h.
 #include <algorithm>
-#include <cstdarg>
 #include <cstdio>
 #include <cstdlib>
 #include <cstring>
@@ -14,52 +13,6 @@
 #include "mega.cuh"
 
 namespace fc {
-
-// ------------------------------------------------------------------------------- errors
-static thread_local char g_err[512] = "";
-thread_local int64_t g_launches = 0;
-DebugKnobs g_debug;
-
-void set_error(const char* fmt, ...) {
-    va_list ap;
-    va_start(ap, fmt);
-    vsnprintf(g_err, sizeof g_err, fmt, ap);
-    va_end(ap);
-}
-const char* g_err_text() { return g_err; }
-int fail(int code, const char* fmt, ...) {
-    va_list ap;
-    va_start(ap, fmt);
-    vsnprintf(g_err, sizeof g_err, fmt, ap);
-    va_end(ap);
-    return code;
-}
-int cuda_fail(cudaError_t e, const char* what, const char* file, int line) {
-    snprintf(g_err, sizeof g_err, "CUDA error %d (%s) at %s:%d in %s", (int)e, cudaGetErrorString(e), file, line, what);
-    return FC_E_CUDA;
-}
-
-// Refuses anything but a Blackwell data-centre part: there is no other code path.
-int select_device(int device) {
-    int n = 0;
-    if (cudaGetDeviceCount(&n) != cudaSuccess || n == 0) {
-        cudaGetLastError();
-        return fail(FC_E_CUDA, "no CUDA device is visible: libferrum_cuda has no CPU fallback");
-    }
-    if (device < 0 || device >= n) return fail(FC_E_ARG, "device %d out of range (0..%d)", device, n - 1);
-    int major = 0;
-    FC_CUDA(cudaDeviceGetAttribute(&major, cudaDevAttrComputeCapabilityMajor, device));
-    if (major != 10) return fail(FC_E_CUDA, "device %d has compute capability %d.x; this library is built for sm_100a only", device, major);
-    FC_CUDA(cudaSetDevice(device));
-    return FC_OK;
-}
-
-int upload_f32(Arena& ar, const float* host, size_t n, float** dev, cudaStream_t st) {
-    if (!host) return fail(FC_E_FORMAT, "a required f32 tensor is null");
-    FC_TRY(ar.alloc_n(dev, n));
-    FC_CUDA(cudaMemcpyAsync(*dev, host, n * sizeof(float), cudaMemcpyHostToDevice, st));
-    return FC_OK;
-}
 
 // loader/mod.rs:147-154: a matrix is Q8_0 only when its row length is a multiple of 32.
 int upload_q8(Arena& ar, const void* host, int N, int K, QMat* out, cudaStream_t st) {
@@ -480,25 +433,6 @@ static int score_device(fc_model* m, int B, int T) {
 //                                      C ABI
 // =====================================================================================
 extern "C" {
-
-const char* fc_last_error(void) { return fc::g_err; }
-
-int fc_device_count(void) {
-    int n = 0;
-    if (cudaGetDeviceCount(&n) != cudaSuccess) { cudaGetLastError(); return 0; }
-    int ok = 0;
-    for (int i = 0; i < n; ++i) {
-        int major = 0;
-        if (cudaDeviceGetAttribute(&major, cudaDevAttrComputeCapabilityMajor, i) == cudaSuccess && major == 10) ++ok;
-    }
-    return ok;
-}
-
-int64_t fc_take_launch_count(void) {
-    const int64_t n = g_launches;
-    g_launches = 0;
-    return n;
-}
 
 // ------------------------------------------------------------------ standalone linear
 int fc_qweight_upload(int device, const void* wq, int N, int K, fc_qweight** out) {
@@ -1804,13 +1738,6 @@ int fc_decode_batch_multi(fc_model* const* models, int n_models, int n_streams, 
     return run_on_models(n_models, n_streams, [&](int i, int a, int b) {
         return fc_decode_batch(models[i], b - a, prompts + (size_t)a * prompt_len, prompt_len, max_new, eos, out + (size_t)a * max_new, n_out + a);
     });
-}
-
-int fc_debug_set_wait_budget(long long cycles, int withhold_producers) {
-    if (cycles <= 0) return fail(FC_E_ARG, "fc_debug_set_wait_budget: cycles = %lld", cycles);
-    g_debug.wait_cycles = cycles;
-    g_debug.withhold = withhold_producers != 0;
-    return FC_OK;
 }
 
 }  // extern "C"

@@ -49,7 +49,7 @@ struct DebugKnobs {
 };
 extern DebugKnobs g_debug;
 
-// ---- host helpers shared by the API files (defined in api.cu) ---------------------------
+// ---- host helpers shared by the API files (common.cu; upload_q8: api.cu) ------------------
 // Owns device allocations until release().
 struct Arena {
     std::vector<void*> ptrs;
@@ -172,7 +172,7 @@ int launch_layernorm_planes(const float* x, const float* g, const float* b, int 
 // (append to queue) — and always the end-of-step bookkeeping (pos, fed).
 int launch_step_tail(const float* logits, int V, float* probs_or_null, int do_select, int* queue, int queue_cap,
                      StepState* state, float* sel_logit_or_null, cudaStream_t st);
-// End-of-step bookkeeping alone (steps that skip the head).
+// common.cu — end-of-step bookkeeping alone (steps that skip the head).
 int launch_step_advance(StepState* state, cudaStream_t st);
 int launch_step_advance_pdl(StepState* state, cudaStream_t st);
 // Scoring tail: per row of logits[R][ldl], target id (or -1) -> logprob, is_greedy.
