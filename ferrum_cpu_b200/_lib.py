@@ -11,7 +11,7 @@ LIB_PATH = os.path.join(_HERE, "libferrum_cuda.so")
 
 FC_OK = 0
 FC_E_SHAPE, FC_E_DIM, FC_E_FORMAT, FC_E_CUDA, FC_E_TIMEOUT, FC_E_CANCELLED, FC_E_ARG = -1, -2, -3, -4, -5, -6, -7
-FC_MATH_FP32, FC_MATH_BF16X3 = 0, 1
+FC_MATH_FP32, FC_MATH_BF16X3, FC_MATH_BF16 = 0, 1, 2
 
 
 class FcConfig(C.Structure):
@@ -61,6 +61,11 @@ class FcScore(C.Structure):
 class FcLayerStats(C.Structure):
     _fields_ = [("min", C.c_float), ("max", C.c_float), ("mean", C.c_float), ("nan_count", C.c_int64), ("inf_count", C.c_int64),
                 ("n_elements", C.c_int64)]
+
+
+class FcNurinexInfo(C.Structure):
+    _fields_ = [("vocab", C.c_int32), ("width", C.c_int32), ("n_layers", C.c_int32), ("n_own_layers", C.c_int32), ("ctx", C.c_int32),
+                ("pad", C.c_int32), ("weight_bytes", C.c_int64)]
 
 
 # name -> (restype, argtypes); every symbol include/ferrum_cuda.h declares
@@ -139,6 +144,22 @@ SIGNATURES = {
     "fc_llama_generate": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.POINTER(FcSampling), C.c_void_p, C.c_int,
                                     C.POINTER(C.c_uint64), C.c_void_p, C.c_void_p, C.POINTER(C.c_int)]),
     "fc_llama_last_decode_ms": (C.c_float, [C.c_void_p]),
+    "fc_model_dir_architecture": (C.c_int, [C.c_char_p, C.c_char_p, C.c_int]),
+    "fc_nurinex_probe": (C.c_int, [C.c_char_p, C.POINTER(FcNurinexInfo)]),
+    "fc_nurinex_load": (C.c_int, [C.c_char_p, C.c_int, C.c_int, C.c_int, C.POINTER(C.c_void_p)]),
+    "fc_nurinex_free": (None, [C.c_void_p]),
+    "fc_nurinex_get_info": (C.c_int, [C.c_void_p, C.POINTER(FcNurinexInfo)]),
+    "fc_nurinex_cache_create": (C.c_int, [C.c_void_p, C.POINTER(C.c_void_p)]),
+    "fc_nurinex_cache_free": (None, [C.c_void_p]),
+    "fc_nurinex_cache_clear": (C.c_int, [C.c_void_p]),
+    "fc_nurinex_cache_pos": (C.c_int, [C.c_void_p]),
+    "fc_nurinex_feed": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_void_p, C.c_int, C.c_void_p]),
+    "fc_nurinex_feed_layers": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_void_p]),
+    "fc_nurinex_score": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.POINTER(FcScore), C.c_void_p, C.c_void_p]),
+    "fc_nurinex_generate": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.POINTER(FcSampling), C.c_void_p, C.c_int,
+                                      C.POINTER(C.c_uint64), C.c_void_p, C.c_void_p, C.POINTER(C.c_int)]),
+    "fc_nurinex_last_forward_ms": (C.c_float, [C.c_void_p]),
+    "fc_nurinex_last_decode_ms": (C.c_float, [C.c_void_p]),
     "fc_rowq_packed_len": (C.c_size_t, [C.c_int, C.c_int, C.c_int]),
     "fc_rowq_from_f32": (C.c_int, [C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p, C.c_void_p]),
     "fc_rowq_to_f32": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p]),
@@ -152,18 +173,30 @@ SIGNATURES = {
 }
 
 _lib = None
+_path = LIB_PATH
+
+
+def use(path):
+    """Names the library this process loads: the complete one (the default) or one that holds a single model family
+    (build.ensure). Only before the first load."""
+    global _path
+    if _lib is not None and path != _path:
+        raise RuntimeError("the library is already loaded")
+    _path = path
 
 
 def lib():
     """The loaded library; raises if it has not been built."""
     global _lib
     if _lib is None:
-        if not os.path.exists(LIB_PATH):
+        if not os.path.exists(_path):
             raise RuntimeError(
-                f"{LIB_PATH} is missing: build it with `python -m ferrum_cpu_b200.build`. "
+                f"{_path} is missing: build it with `python -m ferrum_cpu_b200.build`. "
                 "There is no fallback implementation.")
-        handle = C.CDLL(LIB_PATH)
+        handle = C.CDLL(_path)
         for name, (res, args) in SIGNATURES.items():
+            if _path != LIB_PATH and not hasattr(handle, name):
+                continue                     # a library of one family has no symbols of the others
             fn = getattr(handle, name)
             fn.restype, fn.argtypes = res, args
         _lib = handle

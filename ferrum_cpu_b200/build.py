@@ -1,9 +1,16 @@
 """Builds libferrum_cuda.so in-tree with nvcc for sm_100a (cross-compiles without a GPU).
 
     python -m ferrum_cpu_b200.build [--verbose]
+
+A component is a library of its own with the sources one model family needs, for a host that serves
+only that family and has nothing built yet: `ensure(component)` returns the complete library when it is
+up to date, else builds the component (objects are shared with the complete build).
 """
 import concurrent.futures
+import contextlib
+import fcntl
 import os
+import shutil
 import subprocess
 import sys
 
@@ -11,11 +18,23 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libferrum_cuda.so")
-SOURCES = ["common.cu", "codec.cpp", "gguf_load.cpp", "gemv.cu", "gemv_stream.cu", "rowops.cu", "attn.cu", "gemm_simt.cu", "gemm_tc.cu", "attn_tc.cu", "decode_mega.cu", "decode_batch.cu", "sample.cu", "llama_ops.cu", "llama.cu", "rowq.cu", "ggml_linear.cu", "api.cu"]
+NURINEX = ["common.cu", "model_dir.cpp", "gemm_bf16.cu", "gemv_bf16.cu", "mix_rows.cu", "talk_attn.cu", "talk_attn_tc.cu", "wkv.cu",
+           "mixer_decode.cu", "llama_ops.cu", "sample.cu", "nurinex.cu"]
+SOURCES = ["codec.cpp", "gguf_load.cpp", "gemv.cu", "gemv_stream.cu", "rowops.cu", "attn.cu", "gemm_simt.cu", "gemm_tc.cu", "attn_tc.cu",
+           "decode_mega.cu", "decode_batch.cu", "llama.cu", "rowq.cu", "ggml_linear.cu", "api.cu"] + NURINEX
+COMPONENTS = {"nurinex": NURINEX}
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC", "-Xcompiler", "-Wall",
 ]
+
+
+def component_lib(component):
+    return os.path.join(HERE, f"libferrum_cuda_{component}.so")
+
+
+def _nvcc():
+    return shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
 
 
 def _newer(target, deps):
@@ -25,13 +44,17 @@ def _newer(target, deps):
     return all(os.path.getmtime(d) <= t for d in deps)
 
 
-def _compile(src, verbose):
-    obj = os.path.join(OBJ, src + ".o")
+def _deps(src):
     deps = [os.path.join(CSRC, src)] + [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
     deps.append(os.path.join(HERE, "..", "include", "ferrum_cuda.h"))
-    if _newer(obj, deps):
+    return deps
+
+
+def _compile(src, verbose):
+    obj = os.path.join(OBJ, src + ".o")
+    if _newer(obj, _deps(src)):
         return obj, ""
-    cmd = ["nvcc", *NVCC_FLAGS, "-x", "cu", "-c", os.path.join(CSRC, src), "-o", obj]
+    cmd = [_nvcc(), *NVCC_FLAGS, "-x", "cu", "-c", os.path.join(CSRC, src), "-o", obj]
     if verbose:
         cmd[1:1] = ["-Xptxas", "-v"]
     r = subprocess.run(cmd, capture_output=True, text=True)
@@ -40,18 +63,37 @@ def _compile(src, verbose):
     return obj, r.stderr
 
 
-def build(verbose=False):
+@contextlib.contextmanager
+def _lock():
     os.makedirs(OBJ, exist_ok=True)
-    with concurrent.futures.ThreadPoolExecutor(max_workers=8) as ex:
-        results = list(ex.map(lambda s: _compile(s, verbose), SOURCES))
-    objs = [o for o, _ in results]
-    log = "".join(l for _, l in results)
-    if not _newer(LIB, objs):
-        cmd = ["nvcc", "-shared", "-o", LIB, *objs, "-cudart", "static"]
-        r = subprocess.run(cmd, capture_output=True, text=True)
-        if r.returncode != 0:
-            raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
+    with open(os.path.join(OBJ, ".lock"), "w") as f:
+        fcntl.flock(f, fcntl.LOCK_EX)
+        yield
+
+
+def build(verbose=False, component=None):
+    sources, lib = (SOURCES, LIB) if component is None else (COMPONENTS[component], component_lib(component))
+    with _lock():
+        with concurrent.futures.ThreadPoolExecutor(max_workers=8) as ex:
+            results = list(ex.map(lambda s: _compile(s, verbose), sources))
+        objs = [o for o, _ in results]
+        log = "".join(l for _, l in results)
+        if not _newer(lib, objs):
+            part = f"{lib}.{os.getpid()}"
+            r = subprocess.run([_nvcc(), "-shared", "-o", part, *objs, "-cudart", "static"], capture_output=True, text=True)
+            if r.returncode != 0:
+                raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
+            os.replace(part, lib)
     return log
+
+
+def ensure(component):
+    """Path of a library that holds the component: the complete one when it is newer than every source, else the
+    component's own, compiled now if need be."""
+    if _newer(LIB, {d for s in SOURCES for d in _deps(s)}):
+        return LIB
+    build(component=component)
+    return component_lib(component)
 
 
 if __name__ == "__main__":

@@ -55,6 +55,14 @@ int upload_f32(Arena& ar, const float* host, size_t n, float** dev, cudaStream_t
 }
 
 // ------------------------------------------------------------------- end-of-step bookkeeping
+__global__ void step_set_kernel(StepState* st, int pos, int fed, int tail) {
+    st->pos = pos; st->fed = fed; st->tail = tail; st->done = 0; st->eos = -1; st->error = 0;
+}
+int launch_step_set(StepState* state, int pos, int fed, int tail, cudaStream_t st) {
+    step_set_kernel<<<1, 1, 0, st>>>(state, pos, fed, tail);
+    FC_LAUNCHED();
+    return FC_OK;
+}
 __global__ void step_advance_kernel(StepState* st) {
     pdl_trigger();
     pdl_wait();

@@ -174,6 +174,7 @@ int launch_step_tail(const float* logits, int V, float* probs_or_null, int do_se
                      StepState* state, float* sel_logit_or_null, cudaStream_t st);
 // common.cu — end-of-step bookkeeping alone (steps that skip the head).
 int launch_step_advance(StepState* state, cudaStream_t st);
+int launch_step_set(StepState* state, int pos, int fed, int tail, cudaStream_t st);
 int launch_step_advance_pdl(StepState* state, cudaStream_t st);
 // Scoring tail: per row of logits[R][ldl], target id (or -1) -> logprob, is_greedy.
 // `status` (device int, may be null) is raised to FC_E_TIMEOUT when a bounded wait runs out.

@@ -6,6 +6,7 @@
 #include <cstring>
 #include <vector>
 
+#include "decode_loop.cuh"
 #include "llama_native.h"
 #include "llama_ops.cuh"
 
@@ -423,10 +424,6 @@ int run_step(fc_llama_cache* s, int with_head) {
     return FC_OK;
 }
 
-__global__ void llama_set_state_kernel(StepState* st, int pos, int fed, int tail) {
-    st->pos = pos; st->fed = fed; st->tail = tail; st->done = 0; st->eos = -1; st->error = 0;
-}
-
 int read_state(fc_llama_cache* s, StepState* out) {
     int status = 0;
     FC_CUDA(cudaMemcpyAsync(out, s->state, sizeof(StepState), cudaMemcpyDeviceToHost, s->m->st));
@@ -445,8 +442,7 @@ int feed_ids(fc_llama_cache* s, const int32_t* ids, int n, int head_on_last) {
     if (s->host_pos + n > m->cfg.ctx)
         return fail(FC_E_DIM, "%d more tokens do not fit the model's %d-token context window (position %d)", n, m->cfg.ctx, s->host_pos);
     FC_CUDA(cudaMemcpyAsync(s->queue + s->host_pos, ids, (size_t)n * 4, cudaMemcpyHostToDevice, m->st));
-    llama_set_state_kernel<<<1, 1, 0, m->st>>>(s->state, s->host_pos, s->host_pos, s->host_pos + n);
-    FC_LAUNCHED();
+    FC_TRY(launch_step_set(s->state, s->host_pos, s->host_pos, s->host_pos + n, m->st));
     for (int i = 0; i < n; ++i) FC_TRY(run_step(s, head_on_last && i + 1 == n));
     s->host_pos += n;
     return FC_OK;
@@ -468,8 +464,7 @@ int prime_window(fc_llama_cache* s, const int32_t* ids, int n) {
     const int rc = forward_rows(m, 1, n, s);
     m->force_fp32 = false;
     FC_TRY(rc);
-    llama_set_state_kernel<<<1, 1, 0, st>>>(s->state, n, n, n);
-    FC_LAUNCHED();
+    FC_TRY(launch_step_set(s->state, n, n, n, st));
     // logits of the last row: the final norm was applied by forward_rows
     if (m->prec >= 0)
         FC_TRY(lin_apply(m->packed_head, m->n + (size_t)(n - 1) * c.d_model, nullptr, nullptr, s->logits, m->head.N_pad, 1, st));
@@ -800,8 +795,7 @@ void fc_llama_cache_free(fc_llama_cache* s) {
 int fc_llama_cache_clear(fc_llama_cache* s) {
     if (!s) return fail(FC_E_ARG, "fc_llama_cache_clear: null cache");
     FC_CUDA(cudaSetDevice(s->m->device));
-    llama_set_state_kernel<<<1, 1, 0, s->m->st>>>(s->state, 0, 0, 0);
-    FC_LAUNCHED();
+    FC_TRY(launch_step_set(s->state, 0, 0, 0, s->m->st));
     s->host_pos = 0;
     return FC_OK;
 }
@@ -858,50 +852,9 @@ int fc_llama_generate(fc_llama_cache* s, const int32_t* prompt, int n, int max_n
     FC_CUDA(cudaMemcpyAsync(s->rng_d, rng_state, 8, cudaMemcpyHostToDevice, st));
     if (n >= kPrimeBatchMin) FC_TRY(prime_window(s, prompt, n));
     else FC_TRY(feed_ids(s, prompt, n, 1));
-    // greedy without a penalty needs neither the sampler's sort nor, without stop ids, the host
-    const bool plain_greedy = params->temperature <= 0.0f && params->repetition_penalty == 1.0f;
-    const bool free_run = plain_greedy && n_stops == 0 && !cancel;
-    FC_CUDA(cudaEventRecord(s->ev0, st));
-    int made = 0;
-    int rc = FC_OK;
-    bool cancelled = false, timed = false;
-    while (made < max_new) {
-        if (cancel && *cancel) { cancelled = true; break; }
-        // recent = prompt + tokens so far = the queue (llm.rs:740-751)
-        rc = plain_greedy ? launch_llama_pick(s->logits, c.vocab, s->queue, s->queue_cap, s->state, st)
-                          : launch_sample(s->logits, c.vocab, 0, *params, s->queue, 0, s->rng_d, s->queue, s->queue_cap, s->state,
-                                          nullptr, st);
-        if (rc != FC_OK) break;
-        ++made;
-        bool stop = false;
-        if (!free_run) {
-            int32_t tok = 0;
-            if (cudaMemcpyAsync(&tok, s->queue + n + made - 1, 4, cudaMemcpyDeviceToHost, st) != cudaSuccess ||
-                cudaStreamSynchronize(st) != cudaSuccess) { rc = fail(FC_E_CUDA, "token download failed"); break; }
-            out[made - 1] = tok;
-            for (int i = 0; i < n_stops; ++i) stop |= stops[i] == tok;
-        }
-        if (stop) break;                                     // a stop id is kept in out and not fed (llm.rs:747-749)
-        // the forward of the last requested token keeps the cache continuable (llm.rs:750-751); its logits are not used
-        // here, so it stays outside the timed region
-        if (made == max_new) { FC_CUDA(cudaEventRecord(s->ev1, st)); timed = true; }
-        rc = run_step(s, 1);                                 // forward_one(next), the last token included (llm.rs:750-751)
-        if (rc != FC_OK) break;
-        s->host_pos += 1;
-    }
-    if (rc == FC_OK) {
-        if (!timed) FC_CUDA(cudaEventRecord(s->ev1, st));
-        if (free_run && made > 0) FC_CUDA(cudaMemcpyAsync(out, s->queue + n, (size_t)made * 4, cudaMemcpyDeviceToHost, st));
-        StepState hs;
-        rc = read_state(s, &hs);
-        if (rc == FC_OK && hs.error) rc = fail(hs.error, "the decode step rejected a token or position on the device");
-        if (rc == FC_OK) FC_CUDA(cudaEventElapsedTime(&s->last_decode_ms, s->ev0, s->ev1));
-    }
-    FC_CUDA(cudaMemcpy(rng_state, s->rng_d, 8, cudaMemcpyDeviceToHost));
-    if (rc != FC_OK) return rc;
-    *n_out = made;
-    if (cancelled) return fail(FC_E_CANCELLED, "generation cancelled after %d tokens", made);
-    return FC_OK;
+    const GenCtx g = {st, s->logits, c.vocab, s->queue, s->queue_cap, s->state, s->rng_d, s->ev0, s->ev1, &s->host_pos, &s->last_decode_ms};
+    return generate_tokens(g, n, max_new, params, stops, n_stops, rng_state, cancel, out, n_out, [&] { return run_step(s, 1); },
+                           [&](StepState* hs) { return read_state(s, hs); });
 }
 
 float fc_llama_last_decode_ms(const fc_llama_cache* s) { return s ? s->last_decode_ms : 0.0f; }

@@ -1,0 +1,210 @@
+// Attention whose heads' scores are mixed before the softmax ("talking heads"), with a learned bias per distance,
+// a sink in the denominator, a query temperature that grows with the position, and normed values.
+//
+// Mixing commutes with the product: the mixed score of head h is q'_h . (keys of all key/value heads side by side) with
+// q'_h = [sum_{g in group 0} talk[h][g] q_g | sum_{g in group 1} ... ], plus a per-head table of the distance whose
+// heads are mixed once at load. So after `talk_prep_kernel` this is ordinary attention with one wide shared key head.
+//
+//   talk_prep_kernel      one CTA per token: mixed queries out, key row and normed value row into the cache
+//   talk_prefill_kernel   16 query rows x one head per CTA, f32 CUDA cores, online softmax over key tiles of 32
+// Bound: prep HBM / L2; prefill fp32 FMA (the tcgen05 form is talk_attn_tc.cu).
+#include <algorithm>
+
+#include "bf16_ops.cuh"
+#include "tc_common.cuh"
+
+namespace fc {
+
+namespace {
+template <class T>
+__device__ __forceinline__ void put(T* p, float v) {
+    if constexpr (sizeof(T) == 2) *p = __bfloat16_as_ushort(__float2bfloat16_rn(v));
+    else *p = v;
+}
+template <class T>
+__device__ __forceinline__ float get(const T* p) {
+    if constexpr (sizeof(T) == 2) return __uint_as_float((uint32_t)*p << 16);
+    else return *p;
+}
+}  // namespace
+
+// PER: query heads per key/value head when it is one of the unrolled counts, 0: any.
+template <class T, int PER>
+__global__ void __launch_bounds__(256) talk_prep_kernel(const TalkAttn t, const float* __restrict__ proj, int ldp, int pos0, float factor,
+                                                        T* __restrict__ qm, T* __restrict__ kc, T* __restrict__ vc) {
+    extern __shared__ float sm[];              // talk [H][H] | q [H * dim]
+    const int tid = threadIdx.x, row = blockIdx.x, pos = pos0 + row, H = t.H, dim = t.dim, per = H / t.KV;
+    float* tk = sm;
+    float* q = sm + H * H;
+    const float* src = proj + (size_t)row * ldp;
+    const float temp = 1.0f + t.temp_coef * logf((float)(floor((double)(pos + 1) / t.temp_every) + 1.0));
+    for (int i = tid; i < H * H; i += 256) tk[i] = t.talk[i];
+    const float qs = t.scale * temp * factor;
+    for (int i = tid; i < H * dim; i += 256) q[i] = src[i] * qs;
+    __syncthreads();
+    const int width = t.KV * dim;
+    T* out = qm + (size_t)row * H * t.kd;
+    for (int f = tid; f < t.kd; f += 256) {
+        if (f >= width) {
+            for (int h = 0; h < H; ++h) put(out + (size_t)h * t.kd + f, 0.0f);
+            continue;
+        }
+        const int c = f / dim, e = f - c * dim;
+        const float* qc = q + (size_t)c * per * dim + e;
+        if constexpr (PER > 0) {
+            float qr[PER];
+#pragma unroll
+            for (int g = 0; g < PER; ++g) qr[g] = qc[g * dim];
+            for (int h = 0; h < H; ++h) {
+                const float* w = tk + h * H + c * PER;
+                float s = 0.0f;
+#pragma unroll
+                for (int g = 0; g < PER; ++g) s = fmaf(w[g], qr[g], s);
+                put(out + (size_t)h * t.kd + f, s);
+            }
+        } else {
+            for (int h = 0; h < H; ++h) {
+                const float* w = tk + h * H + c * per;
+                float s = 0.0f;
+                for (int g = 0; g < per; ++g) s = fmaf(w[g], qc[g * dim], s);
+                put(out + (size_t)h * t.kd + f, s);
+            }
+        }
+    }
+    const float* ks = src + H * dim;
+    for (int f = tid; f < t.kd; f += 256) put(kc + (size_t)pos * t.kd + f, f < width ? ks[f] : 0.0f);
+    const float* vs = ks + width;
+    for (int c = tid >> 5; c < t.KV; c += 8) {
+        const int lane = tid & 31;
+        float s = 0.0f;
+        for (int e = lane; e < t.vdim; e += 32) { const float v = vs[c * t.vdim + e]; s = fmaf(v, v, s); }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        const float inv = 1.0f / sqrtf(s / (float)t.vdim + t.eps);
+        for (int e = lane; e < t.vp; e += 32) put(vc + ((size_t)pos * t.KV + c) * t.vp + e, e < t.vdim ? vs[c * t.vdim + e] * inv : 0.0f);
+    }
+}
+
+template <class T>
+static int prep(const TalkAttn& t, const float* proj, int ldp, int M, int pos0, float factor, void* qm, void* kc, void* vc, cudaStream_t st) {
+    const size_t smem = (size_t)(t.H * t.H + t.H * t.dim) * sizeof(float);
+    if (smem > 200 * 1024) return fail(FC_E_SHAPE, "%d query heads of %d exceed the staging of the query mixing", t.H, t.dim);
+#define FC_PREP(P)                                                                                                              \
+    do {                                                                                                                        \
+        if (smem > 48 * 1024) FC_CUDA(cudaFuncSetAttribute(talk_prep_kernel<T, P>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+        talk_prep_kernel<T, P><<<M, 256, smem, st>>>(t, proj, ldp, pos0, factor, (T*)qm, (T*)kc, (T*)vc);                        \
+    } while (0)
+    switch (t.H / t.KV) {
+        case 1: FC_PREP(1); break;
+        case 2: FC_PREP(2); break;
+        case 3: FC_PREP(3); break;
+        case 4: FC_PREP(4); break;
+        case 8: FC_PREP(8); break;
+        default: FC_PREP(0);
+    }
+#undef FC_PREP
+    FC_LAUNCHED();
+    return FC_OK;
+}
+int launch_talk_prep(const TalkAttn& t, const float* proj, int ldp, int M, int pos0, float factor, void* qm, void* kc, void* vc, bool f32,
+                     cudaStream_t st) {
+    return f32 ? prep<float>(t, proj, ldp, M, pos0, factor, qm, kc, vc, st) : prep<uint16_t>(t, proj, ldp, M, pos0, factor, qm, kc, vc, st);
+}
+
+namespace {
+constexpr int QR = 16, KT = 32, KC = 64, PNT = 128, VCOLS = 2;     // value columns per thread: heads of at most 256
+}
+template <class T>
+__global__ void __launch_bounds__(PNT) talk_prefill_kernel(const TalkAttn t, const T* __restrict__ qm, const T* __restrict__ kc,
+                                                           const T* __restrict__ vc, int M, int pos0, T* __restrict__ out, int ldo) {
+    __shared__ float Qs[QR][KC + 1], Ks[KT][KC + 1], P[QR][KT + 1];
+    __shared__ float corr_s[QR], l_s[QR];
+    const int tid = threadIdx.x, h = blockIdx.y, row0 = (gridDim.x - 1 - blockIdx.x) * QR, kv = h / (t.H / t.KV);
+    const int rows = min(QR, M - row0), last = pos0 + row0 + rows - 1;
+    const int qi = tid >> 3, k8 = tid & 7, qpos = pos0 + row0 + qi;
+    const float* bias = t.bias + (size_t)h * (t.far + 1);
+    float m = t.sink[h], l = 1.0f;                 // the sink: weight exp(sink - m) = 1 so far, no key, no value
+    float acc[VCOLS][QR];
+#pragma unroll
+    for (int c = 0; c < VCOLS; ++c)
+#pragma unroll
+        for (int r = 0; r < QR; ++r) acc[c][r] = 0.0f;
+    for (int k0 = 0; k0 <= last; k0 += KT) {
+        float s[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+        for (int e0 = 0; e0 < t.kd; e0 += KC) {
+            __syncthreads();
+            for (int i = tid; i < QR * KC; i += PNT) {
+                const int r = i / KC, e = i - r * KC;
+                Qs[r][e] = r < rows && e0 + e < t.kd ? get(qm + ((size_t)(row0 + r) * t.H + h) * t.kd + e0 + e) : 0.0f;
+            }
+            for (int i = tid; i < KT * KC; i += PNT) {
+                const int r = i / KC, e = i - r * KC;
+                Ks[r][e] = k0 + r <= last && e0 + e < t.kd ? get(kc + (size_t)(k0 + r) * t.kd + e0 + e) : 0.0f;
+            }
+            __syncthreads();
+#pragma unroll 8
+            for (int e = 0; e < KC; ++e) {
+                const float q = Qs[qi][e];
+#pragma unroll
+                for (int x = 0; x < 4; ++x) s[x] = fmaf(q, Ks[k8 + 8 * x][e], s[x]);
+            }
+        }
+        float mx = -INFINITY;
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+            const int n = qpos - (k0 + k8 + 8 * x);
+            s[x] = n >= 0 ? s[x] + bias[min(n, t.far)] : -INFINITY;
+            mx = fmaxf(mx, s[x]);
+        }
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float mn = fmaxf(m, mx), corr = expf(m - mn);
+        float ps = 0.0f;
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+            const float p = expf(s[x] - mn);
+            P[qi][k8 + 8 * x] = p;
+            ps += p;
+        }
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
+        l = fmaf(l, corr, ps);
+        m = mn;
+        if (k8 == 0) { corr_s[qi] = corr; l_s[qi] = l; }
+        __syncthreads();
+        const int nk = min(KT, last - k0 + 1);
+#pragma unroll
+        for (int c = 0; c < VCOLS; ++c) {
+            const int col = tid + c * PNT;
+            if (col >= t.vdim) continue;
+#pragma unroll
+            for (int r = 0; r < QR; ++r) acc[c][r] *= corr_s[r];
+            const T* v = vc + ((size_t)k0 * t.KV + kv) * t.vp + col;
+            for (int j = 0; j < nk; ++j) {
+                const float x = get(v + (size_t)j * t.KV * t.vp);
+#pragma unroll
+                for (int r = 0; r < QR; ++r) acc[c][r] = fmaf(P[r][j], x, acc[c][r]);
+            }
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int c = 0; c < VCOLS; ++c) {
+        const int col = tid + c * PNT;
+        if (col >= t.vdim) continue;
+#pragma unroll
+        for (int r = 0; r < QR; ++r)
+            if (r < rows) put(out + (size_t)(row0 + r) * ldo + (size_t)h * t.vdim + col, acc[c][r] / l_s[r]);
+    }
+}
+int launch_talk_prefill(const TalkAttn& t, const void* qm, const void* kc, const void* vc, int M, int pos0, void* out, int ldo, bool f32,
+                        cudaStream_t st) {
+    const dim3 grid((M + QR - 1) / QR, t.H);
+    if (f32) talk_prefill_kernel<float><<<grid, PNT, 0, st>>>(t, (const float*)qm, (const float*)kc, (const float*)vc, M, pos0, (float*)out, ldo);
+    else talk_prefill_kernel<uint16_t><<<grid, PNT, 0, st>>>(t, (const uint16_t*)qm, (const uint16_t*)kc, (const uint16_t*)vc, M, pos0,
+                                                             (uint16_t*)out, ldo);
+    FC_LAUNCHED();
+    return FC_OK;
+}
+
+}  // namespace fc

@@ -1,0 +1,311 @@
+// The attention of talk_attn.cu on the tcgen05 tensor cores, for portions of a prompt: queries already mixed (bf16,
+// scale, temperature and log2(e) inside), keys and values straight from the bf16 cache.
+//
+// One CTA owns 128 query rows of one head; key tiles of 64.
+//   warp 4      TMA: the query tile once (k-chunks of 64 columns), then per key tile the chunks of the wide key row
+//               through a ring, and the value tile of the head's key/value head (two buffers)
+//   warp 5      tcgen05.mma: S = q' K^T into one of two score buffers, one tile ahead; O += P V (V consumed MN-major),
+//               P as bf16 hi + lo so that the weights keep 16 bits
+//   warps 0-3   one query row per thread: score + bias[distance] (a 191-entry slice of the head's table per tile, -inf
+//               for keys ahead of the query), online softmax in base 2 that starts from the sink (max = sink, sum = 1),
+//               P to shared memory. O stays in TMEM; it is rescaled only when a row's maximum has grown by more than 8.
+// Every mbarrier wait is bounded; on a timeout the status word is raised and the CTA leaves.
+//
+// Bound: tensor pipe / special-function unit. Per (query, key) pair and head KV * dim + 2 vdim multiply-adds executed.
+#include <algorithm>
+
+#include "bf16_ops.cuh"
+#include "tc_common.cuh"
+
+namespace fc {
+
+using namespace tc;
+
+namespace {
+constexpr int QT = 128, KT = 64, CH = 64;
+constexpr int Q_CHUNK = QT * CH * 2;       // 16 KiB
+constexpr int K_CHUNK = KT * CH * 2;       // 8 KiB
+constexpr int P_BYTES = QT * KT * 2;       // 16 KiB
+constexpr int MAX_KS = 8;
+constexpr int TMA_WARP = 4, MMA_WARP = 5, THREADS = 6 * 32;
+constexpr uint32_t IDESC_S = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(KT >> 3) << 17) | ((uint32_t)(QT >> 4) << 24);
+constexpr uint32_t IDESC_O = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(CH >> 3) << 17) | ((uint32_t)(QT >> 4) << 24);
+constexpr float GROW = 8.0f;               // log2: how far a row's maximum may run ahead of the one its sums are relative to
+
+struct Bars {
+    unsigned long long q_full, k_full[MAX_KS], k_empty[MAX_KS], v_full[2], v_empty[2], s_full[2], s_empty[2], p_full, o_done;
+    uint32_t tmem_base;
+    volatile int abort;
+    float bias[2][192];
+};
+struct Args {
+    int M, pos0, kd, nkc, ks, nv, H, KV, vdim, vp, far, ldo;
+    const float *bias, *sink;
+    uint16_t* out;
+    int* status;
+    long long wait_cycles;
+    int withhold;
+    uint32_t tmem_cols;
+};
+size_t smem_bytes(int nkc, int ks, int nv) {
+    return (size_t)nkc * Q_CHUNK + (size_t)ks * K_CHUNK + (size_t)2 * nv * K_CHUNK + 2 * P_BYTES + 1024 + sizeof(Bars);
+}
+// Key-ring stages that fit: as many as keep two CTAs on an SM, else as many as fit one. 0: the shape does not fit.
+int plan_stages(int nkc, int nv) {
+    for (int ks = MAX_KS; ks >= 3; --ks)
+        if (smem_bytes(nkc, ks, nv) <= 113 * 1024) return ks;
+    for (int ks = MAX_KS; ks >= 2; --ks)
+        if (smem_bytes(nkc, ks, nv) <= 226 * 1024) return ks;
+    return 0;
+}
+}  // namespace
+
+__global__ void __launch_bounds__(THREADS, 2)
+talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv,
+                       const Args a) {
+    extern __shared__ unsigned char smem_raw[];
+    unsigned char* smem = (unsigned char*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+    unsigned char* sk = smem + a.nkc * Q_CHUNK;
+    unsigned char* sv_ = sk + a.ks * K_CHUNK;
+    unsigned char* sp = sv_ + 2 * a.nv * K_CHUNK;
+    Bars* bars = (Bars*)(sp + 2 * P_BYTES);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * QT, h = blockIdx.y, kv = h / (a.H / a.KV);
+    const int last = a.pos0 + min(a.M, q0 + QT) - 1;       // the last key any row of the tile sees
+    const int n_kt = last / KT + 1;
+
+    if (threadIdx.x == 0) {
+        mbar_init(&bars->q_full, 1);
+        for (int i = 0; i < a.ks; ++i) { mbar_init(&bars->k_full[i], 1); mbar_init(&bars->k_empty[i], 1); }
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(&bars->v_full[i], 1); mbar_init(&bars->v_empty[i], 1);
+            mbar_init(&bars->s_full[i], 1); mbar_init(&bars->s_empty[i], 4);
+        }
+        mbar_init(&bars->p_full, 4);
+        mbar_init(&bars->o_done, 1);
+        bars->abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == MMA_WARP) tmem_alloc(&bars->tmem_base, a.tmem_cols);
+    fence_before();
+    __syncthreads();
+    fence_after();
+    const uint32_t tmem = bars->tmem_base, tmem_o = tmem + 2 * KT;
+    auto wait = [&](unsigned long long* b, uint32_t par) { return wait_bar(&bars->abort, b, par, a.status, a.wait_cycles); };
+
+    if (warp == TMA_WARP) {
+        if (lane == 0 && !a.withhold) {
+            mbar_expect_tx(&bars->q_full, a.nkc * Q_CHUNK);
+            for (int c = 0; c < a.nkc; ++c) tma_load_2d(smem + c * Q_CHUNK, &mq, h * a.kd + c * CH, q0, &bars->q_full);
+            int it = 0, nvt = 0;
+            bool ok = true;
+            for (int kt = 0; kt < n_kt && ok; ++kt) {
+                for (int c = 0; c < a.nkc && ok; ++c) {
+                    const int s = it % a.ks;
+                    ok = wait(&bars->k_empty[s], ((it / a.ks) & 1) ^ 1);
+                    if (!ok) break;
+                    mbar_expect_tx(&bars->k_full[s], K_CHUNK);
+                    tma_load_2d(sk + s * K_CHUNK, &mk, c * CH, kt * KT, &bars->k_full[s]);
+                    ++it;
+                }
+                const int b = kt & 1;
+                ok = ok && wait(&bars->v_empty[b], ((kt >> 1) & 1) ^ 1);
+                if (!ok) break;
+                mbar_expect_tx(&bars->v_full[b], a.nv * K_CHUNK);
+                for (int c = 0; c < a.nv; ++c) tma_load_2d(sv_ + (b * a.nv + c) * K_CHUNK, &mv, kv * a.vp + c * CH, kt * KT, &bars->v_full[b]);
+                ++nvt;
+            }
+            if (bars->abort) {                            // leaving early: no copy may still be on its way into this CTA
+                auto drain = [&](unsigned long long* b, uint32_t par) {
+                    const long long t0 = clock64();
+                    while (!mbar_try_wait(b, par) && clock64() - t0 < a.wait_cycles) {}
+                };
+                drain(&bars->q_full, 0);
+                for (int i = max(0, it - a.ks); i < it; ++i) drain(&bars->k_full[i % a.ks], (i / a.ks) & 1);
+                for (int i = max(0, nvt - 2); i < nvt; ++i) drain(&bars->v_full[i & 1], (i >> 1) & 1);
+            }
+        }
+    } else if (warp == MMA_WARP) {
+        if (lane == 0) {
+            const uint32_t sb = s32(smem), kb = s32(sk), vb = s32(sv_);
+            const uint64_t ph = smem_desc(s32(sp)), pl = smem_desc(s32(sp) + P_BYTES);
+            int it = 0;
+            auto scores = [&](int kt) -> bool {
+                const int b = kt & 1;
+                if (!wait(&bars->s_empty[b], ((kt >> 1) & 1) ^ 1)) return false;
+                fence_after();
+                for (int c = 0; c < a.nkc; ++c, ++it) {
+                    const int s = it % a.ks;
+                    if (!wait(&bars->k_full[s], (it / a.ks) & 1)) return false;
+                    fence_after();
+                    const uint64_t qd = smem_desc(sb + c * Q_CHUNK), kd = smem_desc(kb + s * K_CHUNK);
+#pragma unroll
+                    for (int ks = 0; ks < CH / 16; ++ks) umma(tmem + b * KT, qd + (uint64_t)(ks * 2), kd + (uint64_t)(ks * 2), IDESC_S, (c | ks) != 0);
+                    umma_commit(&bars->k_empty[s]);
+                }
+                umma_commit(&bars->s_full[b]);
+                return true;
+            };
+            bool ok = wait(&bars->q_full, 0) && scores(0);
+            for (int kt = 0; kt < n_kt && ok; ++kt) {
+                if (kt + 1 < n_kt && !(ok = scores(kt + 1))) break;
+                const int b = kt & 1;
+                ok = wait(&bars->v_full[b], (kt >> 1) & 1) && wait(&bars->p_full, kt & 1);
+                if (!ok) break;
+                fence_after();
+                for (int c = 0; c < a.nv; ++c) {
+                    const uint64_t vd = smem_desc(vb + (b * a.nv + c) * K_CHUNK);
+#pragma unroll
+                    for (int ks = 0; ks < KT / 16; ++ks) {
+                        umma(tmem_o + c * CH, ph + (uint64_t)(ks * 2), vd + (uint64_t)(ks * 128), IDESC_O, (kt | ks) != 0);
+                        umma(tmem_o + c * CH, pl + (uint64_t)(ks * 2), vd + (uint64_t)(ks * 128), IDESC_O, 1);
+                    }
+                }
+                umma_commit(&bars->v_empty[b]);
+                umma_commit(&bars->o_done);
+            }
+        }
+    } else {
+        const int r = threadIdx.x;                         // query row of the tile
+        const float* bias = a.bias + (size_t)h * (a.far + 1);
+        float m = a.sink[h] * kLog2e, l = 1.0f;
+        unsigned char* ph = sp + r * 128;
+        unsigned char* pl = ph + P_BYTES;
+        const uint32_t lane_addr = (uint32_t)(warp * 32) << 16;
+        bool ok = true;
+        for (int kt = 0; kt < n_kt; ++kt) {
+            const int b = kt & 1, base = a.pos0 + q0 - kt * KT - (KT - 1);
+            float* bt = bars->bias[b];
+            for (int x = r; x < QT + KT - 1; x += QT) {
+                const int n = base + x;
+                bt[x] = n < 0 ? -INFINITY : bias[min(n, a.far)] * kLog2e;
+            }
+            asm volatile("bar.sync 1, 128;" ::: "memory");
+            ok = __all_sync(0xffffffffu, wait(&bars->s_full[b], (kt >> 1) & 1));
+            // one warp's timeout must not leave the others at the named barrier: everybody goes on to it,
+            // tile by tile, with waits that the abort flag ends at once
+            float sv[KT];
+            float mx = -INFINITY;
+            if (ok) {
+                fence_after();
+                tmem_ld32(tmem + b * KT + lane_addr, (uint32_t*)sv);
+                tmem_ld32(tmem + b * KT + 32 + lane_addr, (uint32_t*)sv + 32);
+                fence_before();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(&bars->s_empty[b]);
+#pragma unroll
+                for (int j = 0; j < KT; ++j) {
+                    sv[j] += bt[r + (KT - 1) - j];
+                    mx = fmaxf(mx, sv[j]);
+                }
+                if (kt > 0) ok = wait(&bars->o_done, (kt - 1) & 1);   // P may be overwritten, O holds tiles 0 .. kt - 1
+            }
+            ok = __all_sync(0xffffffffu, ok);
+            if (ok) {
+                fence_after();
+                const bool grow = mx > m + GROW;
+                if (__any_sync(0xffffffffu, grow)) {
+                    const float mn = grow ? mx : m, corr = ex2_approx(m - mn);
+                    l *= corr;
+                    m = mn;
+                    if (kt > 0)
+                        for (int c = 0; c < 2 * a.nv; ++c) {
+                            uint32_t o[32];
+                            tmem_ld32(tmem_o + c * 32 + lane_addr, o);
+#pragma unroll
+                            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * corr);
+                            tmem_st32(tmem_o + c * 32 + lane_addr, o);
+                        }
+                }
+                float ps = 0.0f;
+#pragma unroll
+                for (int c = 0; c < KT / 8; ++c) {
+                    float p[8];
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) { p[e] = ex2_approx(sv[8 * c + e] - m); ps += p[e]; }
+                    uint4 hi, lo;
+                    split2(p[0], p[1], &hi.x, &lo.x);
+                    split2(p[2], p[3], &hi.y, &lo.y);
+                    split2(p[4], p[5], &hi.z, &lo.z);
+                    split2(p[6], p[7], &hi.w, &lo.w);
+                    const int chunk = (c ^ (r & 7)) * 16;
+                    *(uint4*)(ph + chunk) = hi;
+                    *(uint4*)(pl + chunk) = lo;
+                }
+                l += ps;
+                asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+                fence_before();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(&bars->p_full);
+            }
+        }
+        ok = __all_sync(0xffffffffu, wait(&bars->o_done, (n_kt - 1) & 1) && ok && !bars->abort);
+        if (ok) {
+            fence_after();
+            const float inv = 1.0f / l;
+            const bool store = q0 + r < a.M, vec = (a.vdim & 7) == 0 && (a.ldo & 7) == 0;
+            uint16_t* dst = a.out + (size_t)(q0 + r) * a.ldo + (size_t)h * a.vdim;
+            for (int c = 0; c < 2 * a.nv; ++c) {
+                if (c * 32 >= a.vdim) break;
+                uint32_t o[32];
+                tmem_ld32(tmem_o + c * 32 + lane_addr, o);
+                if (store) {
+                    if (vec) {
+#pragma unroll
+                        for (int i = 0; i < 4; ++i)
+                            if (c * 32 + 8 * i < a.vdim) {
+                                uint4 w;
+                                w.x = pack2(__uint_as_float(o[8 * i]) * inv, __uint_as_float(o[8 * i + 1]) * inv);
+                                w.y = pack2(__uint_as_float(o[8 * i + 2]) * inv, __uint_as_float(o[8 * i + 3]) * inv);
+                                w.z = pack2(__uint_as_float(o[8 * i + 4]) * inv, __uint_as_float(o[8 * i + 5]) * inv);
+                                w.w = pack2(__uint_as_float(o[8 * i + 6]) * inv, __uint_as_float(o[8 * i + 7]) * inv);
+                                *(uint4*)(dst + c * 32 + 8 * i) = w;
+                            }
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 32; ++i)
+                            if (c * 32 + i < a.vdim) dst[c * 32 + i] = __bfloat16_as_ushort(__float2bfloat16_rn(__uint_as_float(o[i]) * inv));
+                    }
+                }
+                __syncwarp();
+            }
+        }
+    }
+    fence_before();
+    __syncthreads();
+    if (warp == MMA_WARP) {
+        fence_after();
+        tmem_dealloc(tmem, a.tmem_cols);
+    }
+}
+
+bool talk_tc_fits(const TalkAttn& t) { return t.vdim <= 256 && plan_stages((t.kd + CH - 1) / CH, (t.vp + CH - 1) / CH) > 0; }
+
+int launch_talk_prefill_tc(const TalkAttn& t, const void* qm, const void* kc, const void* vc, int M, int pos0, int ctx, void* out, int ldo,
+                           int* status, cudaStream_t st) {
+    Args a = {};
+    a.nkc = (t.kd + CH - 1) / CH;
+    a.nv = (t.vp + CH - 1) / CH;
+    a.ks = plan_stages(a.nkc, a.nv);
+    if (!talk_tc_fits(t)) return fail(FC_E_SHAPE, "key rows of %d and value heads of %d do not fit the tensor-core attention", t.kd, t.vdim);
+    static bool attr_set[64] = {};
+    int dev = 0;
+    FC_CUDA(cudaGetDevice(&dev));
+    if (dev < 64 && !attr_set[dev]) {
+        FC_CUDA(cudaFuncSetAttribute(talk_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+        attr_set[dev] = true;
+    }
+    CUtensorMap mq, mk, mv;
+    FC_TRY(encode_bf16(&mq, qm, M, (size_t)t.H * t.kd, (size_t)t.H * t.kd, QT));
+    FC_TRY(encode_bf16(&mk, kc, ctx, t.kd, t.kd, KT));
+    FC_TRY(encode_bf16(&mv, vc, ctx, (size_t)t.KV * t.vp, (size_t)t.KV * t.vp, KT));
+    a.M = M; a.pos0 = pos0; a.kd = t.kd; a.H = t.H; a.KV = t.KV; a.vdim = t.vdim; a.vp = t.vp; a.far = t.far; a.ldo = ldo;
+    a.bias = t.bias; a.sink = t.sink; a.out = (uint16_t*)out; a.status = status;
+    a.wait_cycles = g_debug.wait_cycles; a.withhold = g_debug.withhold;
+    a.tmem_cols = a.nv <= 2 ? 256 : 512;
+    talk_prefill_tc_kernel<<<dim3((M + QT - 1) / QT, t.H), THREADS, smem_bytes(a.nkc, a.ks, a.nv), st>>>(mq, mk, mv, a);
+    FC_LAUNCHED();
+    return FC_OK;
+}
+
+}  // namespace fc

@@ -1,0 +1,104 @@
+"""Writer of model folders (config.json + model.safetensors) and synthetic Nurinex models, for tests and
+benchmarks. Reading is the library's (csrc/model_dir.cpp)."""
+import json
+import os
+import struct
+
+import numpy as np
+
+
+def to_bf16(a):
+    """f32 array -> uint16 bf16 bits, round to nearest even."""
+    u = np.ascontiguousarray(a, dtype=np.float32).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+
+
+def from_bf16(bits):
+    return (np.ascontiguousarray(bits, dtype=np.uint16).astype(np.uint32) << 16).view(np.float32)
+
+
+def write(path, config, tensors):
+    """tensors: name -> uint16 array of bf16 bits (shape kept)."""
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(config, f, indent=1)
+    head, at = {}, 0
+    for name, a in tensors.items():
+        head[name] = {"dtype": "BF16", "shape": list(a.shape), "data_offsets": [at, at + a.nbytes]}
+        at += a.nbytes
+    text = json.dumps(head).encode()
+    with open(os.path.join(path, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(text)))
+        f.write(text)
+        for a in tensors.values():
+            f.write(np.ascontiguousarray(a).tobytes())
+    return path
+
+
+def nurinex_layer(heads=4, kv_heads=2, dim=32, vdim=32, bias_max=100, scale=None, coef=0.3, every=16, r_heads=3, r_dim=32, ff=96,
+                  weights_of=None):
+    """One entry of `layers`. ff 0: no feed-forward."""
+    entry = {
+        "type": "parallel",
+        "mixer": {
+            "left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "bias_max": bias_max,
+                     "scale": dim ** -0.5 if scale is None else scale, "q_temp": {"coef": coef, "every": every}},
+            "right": {"heads": r_heads, "dim": r_dim},
+        },
+        "mlp": {"kind": "dense", "ff": ff} if ff else None,
+    }
+    if weights_of is not None:
+        entry["weights_of"] = weights_of
+    return entry
+
+
+def nurinex_config(vocab, width, layers, eps=1e-5, emb_scale=1.0):
+    return {"architecture": "Nurinex", "vocab": vocab, "width": width, "embedding": {"scale": emb_scale}, "norm": {"eps": eps}, "layers": layers}
+
+
+def nurinex_tensors(config, seed=0, bias_rows=12, rank=8):
+    """Random bf16 weights of the shapes a configuration asks for: name -> uint16 array. bias_rows and rank are numbers
+    or one per layer."""
+    rng = np.random.default_rng(seed)
+    d, V = config["width"], config["vocab"]
+    out = {}
+
+    def put(name, shape, std, mean=0.0):
+        out[name] = to_bf16(rng.standard_normal(shape, dtype=np.float32) * np.float32(std) + np.float32(mean))
+
+    put("embed", (V, d), 1.0 / max(config["embedding"]["scale"], 1e-6))
+    for i, layer in enumerate(config["layers"]):
+        if layer.get("weights_of") is not None:
+            continue
+        p, l, r = f"l{i}.", layer["mixer"]["left"], layer["mixer"]["right"]
+        rows = bias_rows[i] if isinstance(bias_rows, (list, tuple)) else bias_rows
+        rk = rank[i] if isinstance(rank, (list, tuple)) else rank
+        H, G, rd = l["heads"], l["kv_heads"], r["heads"] * r["dim"]
+        put(p + "norm1", (d,), 0.2, 1.0)
+        put(p + "mix.left.q", (H * l["dim"], d), d ** -0.5 * 1.5)
+        put(p + "mix.left.k", (G * l["dim"], d), d ** -0.5 * 1.5)
+        put(p + "mix.left.v", (G * l["vdim"], d), d ** -0.5)
+        put(p + "mix.left.rel", (rows, H), 1.0)
+        out[p + "mix.left.talk"] = to_bf16(np.eye(H, dtype=np.float32) + rng.standard_normal((H, H), dtype=np.float32) * np.float32(0.25))
+        put(p + "mix.left.sink", (H,), 1.0, 1.0)
+        put(p + "mix.left.o", (d, H * l["vdim"]), (H * l["vdim"]) ** -0.5)
+        for s in "rkvgw":
+            put(p + "mix.right.mu." + s, (d,), 0.25, 0.5)
+        for s in "rkvg":
+            put(p + "mix.right." + s, (rd, d), d ** -0.5)
+        put(p + "mix.right.w1", (rk, d), d ** -0.5)
+        put(p + "mix.right.w2", (rd, rk), rk ** -0.5)
+        put(p + "mix.right.w0", (rd,), 1.5, -3.0)
+        put(p + "mix.right.u", (r["heads"], r["dim"]), 0.5, 0.5)
+        put(p + "mix.right.norm", (rd,), 0.2, 1.0)
+        put(p + "mix.right.o", (d, rd), rd ** -0.5)
+        put(p + "mix.left.out", (d,), 0.2, 1.0)
+        put(p + "mix.right.out", (d,), 0.2, 1.0)
+        if layer.get("mlp"):
+            ff = layer["mlp"]["ff"]
+            put(p + "mlp.up", (ff, d), d ** -0.5)
+            put(p + "mlp.down", (d, ff), ff ** -0.5)
+            put(p + "mlp.act", (2,), 0.5, 0.3)
+    put("final.norm", (d,), 0.2, 1.0)
+    put("head", (V, d), d ** -0.5)
+    return out

@@ -39,6 +39,7 @@ extern "C" {
 /* Math modes of the prefill GEMM. Decode always runs fp32 FMA on CUDA cores. */
 #define FC_MATH_FP32 0      /* fp32 CUDA-core GEMM (exactly rounded products) */
 #define FC_MATH_BF16X3 1    /* tcgen05 kind::f16 bf16 operands, 3-term split, fp32 TMEM accumulate */
+#define FC_MATH_BF16 2      /* bf16 operands as they are (models stored in bf16), fp32 TMEM accumulate */
 
 /* Dimensions of a gpt2-architecture GGUF (ferrum_core/src/loader/gpt2.rs:201-215). */
 typedef struct fc_config {
@@ -451,6 +452,46 @@ int fc_llama_generate(fc_llama_cache* c, const int32_t* prompt, int n, int max_n
                       const int32_t* stops, int n_stops, uint64_t* rng_state, const volatile int32_t* cancel,
                       int32_t* out, int* n_out);
 float fc_llama_last_decode_ms(const fc_llama_cache* c);
+
+/* ---- model folders (config.json + model.safetensors) ------------------------------- */
+/* The architecture a folder's config.json names ("architecture"), for choosing the model class. */
+int fc_model_dir_architecture(const char* dir, char* out, int cap);
+
+/* Nurinex: a decoder whose layers put attention (scores mixed across heads, learned distance bias, sink, query
+ * temperature, normed values), a linear-attention recurrence with per-channel decay (RWKV form) and a dense feed-forward
+ * side by side on one norm. No counterpart in the reference; it is served as the imported models are. Every size and
+ * constant comes from the folder's config.json; a layer may use another layer's tensors. Weights are bf16 and stay so.
+ * math_mode: FC_MATH_BF16 (bf16 operands and caches; norms, scores, softmax, decays, recurrence and the residual are f32)
+ * or FC_MATH_FP32 (f32 everywhere, caches too). ctx: positions a cache holds. */
+typedef struct fc_nurinex fc_nurinex;
+typedef struct fc_nurinex_cache fc_nurinex_cache;   /* key / value rows, recurrence states, token-shift rows, position */
+typedef struct fc_nurinex_info {
+    int32_t vocab, width, n_layers, n_own_layers, ctx, pad;
+    int64_t weight_bytes;   /* bytes of matrices one decoded token reads */
+} fc_nurinex_info;
+/* Validates a folder without a GPU. */
+int fc_nurinex_probe(const char* dir, fc_nurinex_info* out);
+int fc_nurinex_load(const char* dir, int device, int math_mode, int ctx, fc_nurinex** out);
+void fc_nurinex_free(fc_nurinex* m);
+int fc_nurinex_get_info(const fc_nurinex* m, fc_nurinex_info* out);
+int fc_nurinex_cache_create(fc_nurinex* m, fc_nurinex_cache** out);
+void fc_nurinex_cache_free(fc_nurinex_cache* c);
+int fc_nurinex_cache_clear(fc_nurinex_cache* c);
+int fc_nurinex_cache_pos(const fc_nurinex_cache* c);
+/* The next n tokens of the cache's sequence: one token runs the decode step, more run as a portion of a prompt, cut
+ * anywhere. logits [n_want][vocab] (host) of the places want[] among them, in that order; n_want may be 0. */
+int fc_nurinex_feed(fc_nurinex_cache* c, const int32_t* ids, int n, const int32_t* want, int n_want, float* logits);
+/* The same for one portion (n <= 2048), leaving the residual stream after every layer: layers [n_layers][n][width]. */
+int fc_nurinex_feed_layers(fc_nurinex_cache* c, const int32_t* ids, int n, float* layers);
+/* Clears the cache and scores ids[from..] given what precedes them, as fc_llama_score_from does for one window: ln
+ * softmax(logits)[target], no probability floor. The sequence must fit the cache. */
+int fc_nurinex_score(fc_nurinex_cache* c, const int32_t* ids, int n, int from, fc_score* score, float* lp, uint8_t* is_greedy);
+/* fc_llama_generate for this decoder: the same sampling, stops, cancel flag and generator state. */
+int fc_nurinex_generate(fc_nurinex_cache* c, const int32_t* prompt, int n, int max_new, const fc_sampling* params,
+                        const int32_t* stops, int n_stops, uint64_t* rng_state, const volatile int32_t* cancel,
+                        int32_t* out, int* n_out);
+float fc_nurinex_last_forward_ms(const fc_nurinex* m);
+float fc_nurinex_last_decode_ms(const fc_nurinex_cache* c);
 
 /* ---- per-row-scale int8 / int4 weights (quant.rs:122-263 QWeight, ops.rs:268-377 qlinear) ---- */
 /* The in-memory quantised weight of the reference: [rows = in_features][cols = out_features]
