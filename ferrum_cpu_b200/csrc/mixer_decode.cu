@@ -128,7 +128,7 @@ __device__ void attention(const MixerDecode& a, float* sm) {
     const int per_split = ((len + splits - 1) / splits + KT - 1) / KT * KT;
     const int k_begin = sp * per_split, k_end = min(len, k_begin + per_split);
     // rows of queries and cached keys are a few banks apart
-    const int dq = (dim + 3) & ~3, qst = dq + 4, hk = H * (KT + 1), khs = dq + (sizeof(T) == 2 ? 8 : 4), kst = t.KV * khs;
+    const int dq = (dim + 3) & ~3, qst = dq + 4, hk = H * (KT + 1), khs = dq + (sizeof(T) == 2 ? 8 : 4), kst = a.kv_block * khs;
     T* ks = (T*)sm;                              // [KT][kst]
     float* q = sm + KT * kst * sizeof(T) / 4;    // [H][qst]
     float* talk = q + H * qst;                   // [H][H], transposed: talk[g][h]
@@ -161,44 +161,47 @@ __device__ void attention(const MixerDecode& a, float* sm) {
         }
     }
     __syncthreads();
-    const int groups = max(1, NT / H);           // groups of keys side by side
     for (int k0 = k_begin; k0 < k_end; k0 += KT) {
         const int nk = min(KT, k_end - k0);
-        for (int i = tid; i < nk * width; i += NT) {
-            const int j = i / width, f = i - j * width, c = f / dim;
-            ks[j * kst + c * khs + (f - c * dim)] = kc[(size_t)(k0 + j) * t.kd + f];
-        }
-        __syncthreads();
-        for (int w = tid; w < H * groups; w += NT) {
-            const int g = w % H, kg = w / H;
-            const float* qg = q + g * qst;
-            const T* kb = ks + (g / per) * khs;
-            for (int jb = kg; jb < KT; jb += groups * KPT) {
-                float s[KPT];
+        for (int c0 = 0; c0 < t.KV; c0 += a.kv_block) {              // as many key heads at a time as shared memory holds
+            const int nc = min(a.kv_block, t.KV - c0), wb = nc * dim, Hb = nc * per, groups = max(1, NT / Hb);
+            if (c0) __syncthreads();
+            for (int i = tid; i < nk * wb; i += NT) {
+                const int j = i / wb, f = i - j * wb, c = f / dim;
+                ks[j * kst + c * khs + (f - c * dim)] = kc[(size_t)(k0 + j) * t.kd + c0 * dim + f];
+            }
+            __syncthreads();
+            for (int w = tid; w < Hb * groups; w += NT) {
+                const int gl = w % Hb, kg = w / Hb, g = c0 * per + gl;
+                const float* qg = q + g * qst;
+                const T* kb = ks + (gl / per) * khs;
+                for (int jb = kg; jb < KT; jb += groups * KPT) {
+                    float s[KPT];
 #pragma unroll
-                for (int x = 0; x < KPT; ++x) s[x] = 0.0f;
-                for (int e0 = 0; e0 < dq; e0 += QREG) {
-                    float4 qr[QREG / 4];
+                    for (int x = 0; x < KPT; ++x) s[x] = 0.0f;
+                    for (int e0 = 0; e0 < dq; e0 += QREG) {
+                        float4 qr[QREG / 4];
 #pragma unroll
-                    for (int e = 0; e < QREG / 4; ++e) qr[e] = e0 + 4 * e < dq ? *(const float4*)(qg + e0 + 4 * e) : make_float4(0, 0, 0, 0);
+                        for (int e = 0; e < QREG / 4; ++e) qr[e] = e0 + 4 * e < dq ? *(const float4*)(qg + e0 + 4 * e) : make_float4(0, 0, 0, 0);
 #pragma unroll
-                    for (int x = 0; x < KPT; ++x) {
-                        const int j = jb + x * groups;
-                        if (j < KT) {
-                            const T* kr = kb + j * kst + e0;
+                        for (int x = 0; x < KPT; ++x) {
+                            const int j = jb + x * groups;
+                            if (j < KT) {
+                                const T* kr = kb + j * kst + e0;
 #pragma unroll
-                            for (int e = 0; e < QREG / 4; ++e)
-                                if (e0 + 4 * e < dq) {
-                                    const float4 k4 = get4(kr + 4 * e);
-                                    s[x] = fmaf(qr[e].x, k4.x, s[x]); s[x] = fmaf(qr[e].y, k4.y, s[x]);
-                                    s[x] = fmaf(qr[e].z, k4.z, s[x]); s[x] = fmaf(qr[e].w, k4.w, s[x]);
-                                }
+                                for (int e = 0; e < QREG / 4; ++e)
+                                    if (e0 + 4 * e < dq) {
+                                        const float4 k4 = get4(kr + 4 * e);
+                                        s[x] = fmaf(qr[e].x, k4.x, s[x]); s[x] = fmaf(qr[e].y, k4.y, s[x]);
+                                        s[x] = fmaf(qr[e].z, k4.z, s[x]); s[x] = fmaf(qr[e].w, k4.w, s[x]);
+                                    }
+                            }
                         }
                     }
-                }
 #pragma unroll
-                for (int x = 0; x < KPT; ++x)
-                    if (jb + x * groups < KT) raw[g * (KT + 1) + jb + x * groups] = s[x];
+                    for (int x = 0; x < KPT; ++x)
+                        if (jb + x * groups < KT) raw[g * (KT + 1) + jb + x * groups] = s[x];
+                }
             }
         }
         __syncthreads();
@@ -315,10 +318,13 @@ __global__ void __launch_bounds__(NT) mixer_decode_kernel(const MixerDecode a) {
     else attention<T>(a, sm);
 }
 
-int launch_mixer_decode(const MixerDecode& a, cudaStream_t st) {
+int launch_mixer_decode(MixerDecode a, cudaStream_t st) {
     const TalkAttn& t = a.t;
     const int dq = (t.dim + 3) & ~3, el = a.f32_cache ? 4 : 2, khs = dq + (a.f32_cache ? 4 : 8);
-    const size_t att = (size_t)(t.H * (dq + 4) + t.H * t.H + 2 * t.H * (KT + 1) + t.H * t.vdim + 3 * t.H) * 4 + (size_t)KT * t.KV * khs * el;
+    const size_t fixed = (size_t)(t.H * (dq + 4) + t.H * t.H + 2 * t.H * (KT + 1) + t.H * t.vdim + 3 * t.H) * 4, head = (size_t)KT * khs * el;
+    a.kv_block = t.KV;
+    while (a.kv_block > 1 && fixed + a.kv_block * head > 220 * 1024) a.kv_block = (a.kv_block + 1) / 2;
+    const size_t att = fixed + a.kv_block * head;
     const size_t rec = (size_t)(4 * a.rdim + a.rank + std::max(1, NT / a.rdim) * a.rdim) * 4;
     const size_t smem = std::max(att, rec);
     if (smem > 220 * 1024) return fail(FC_E_SHAPE, "the decode mixers need %zu bytes of shared memory", smem);
