@@ -2,7 +2,7 @@
 """Benchmark of the Q8_0 GPT-2 forward path on B200.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--workload ...] [--impl ours|reference]
-    python bench.py --case decode|score|linear|rowq|ggml-linear|streams|llama-decode|llama-score [...]
+    python bench.py --case decode|score|linear|rowq|ggml-linear|streams|llama-*|nurinex-* [...]
 
 Workloads (synthetic, seeded; shapes of the reference's configurations):
   decode        : GPT-2-small-shaped Q8_0 model, batch 1, 32-token prompt, 256 greedy tokens with a
@@ -19,6 +19,8 @@ Workloads (synthetic, seeded; shapes of the reference's configurations):
                   oracle's matmul engine.
   tiny          : the 4-block CPU-sized configuration (16-token prompt, 64 greedy tokens).
   llama-1b      : the imported Llama-shaped decoder.
+  nurinex       : prefill, scoring and batch-1 decode of the Nurinex decoder at a few sizes (bf16, random weights),
+                  each beside the Llama-shaped decoder with layers of the same sizes.
 
 --case runs one small, self-terminating piece of the same kernels (a few tokens / windows / one
 product) and prints CUDA-event times: these are the command lines the profiler notes under
@@ -265,6 +267,110 @@ def run_sweep(fcb, synth, torch, shapes, reps, with_oracle):
     return rows
 
 
+def nurinex_work(name, T, p_first, n_new):
+    """Algorithmic work of a named Nurinex shape: matrix weights a token meets, FLOP of a T-token prompt (head on every row),
+    HBM bytes of one decoded token averaged over n_new positions from p_first (weights once, cached rows, states in and out)."""
+    from ferrum_cpu_b200 import model_dir
+    V, d, n, H, G, hd, rH, rD, ff, rank = model_dir.NURINEX_SHAPES[name]
+    rd = rH * rD
+    per_layer = d * (H * hd + 2 * G * hd + 2 * ff + 5 * rd + rank + H * hd) + rd * rank
+    weights = n * per_layer + V * d
+    pair = n * H * (2 * hd + 2 * hd + 2 * H)                     # scores, values, head mixing
+    flop = 2.0 * weights * T + pair * T * (T + 1) / 2 + n * 8.0 * rH * rD * rD * T
+    byts = 2.0 * weights + n * 2 * rH * rD * rD * 4
+    byts += sum(n * 2 * (p + 1) * G * hd * 2 for p in range(p_first, p_first + n_new)) / n_new
+    return weights, flop, byts
+
+
+def llama_twin(name):
+    """The Llama-shaped model with the layer sizes of a named Nurinex shape: SynthLlama arguments."""
+    from ferrum_cpu_b200 import model_dir
+    V, d, n, H, G, hd, rH, rD, ff, rank = model_dir.NURINEX_SHAPES[name]
+    return (V, d, n, H, G, hd, ff, 2304)
+
+
+def run_nurinex(a, names, prompts=(256, 1024, 2048), with_llama=True):
+    """Prefill (one sequence, logits of the last row), scoring (logits of every row) and greedy decode, device-timed by the
+    library's CUDA events; weights of every shape exceed the L2."""
+    import tempfile
+
+    import ferrum_cpu_b200 as fcb
+    from ferrum_cpu_b200 import model_dir, synth
+    from ferrum_cpu_b200.engine import sampling
+    from ferrum_cpu_b200.llama import CudaLlama
+    from ferrum_cpu_b200.nurinex import CudaNurinex
+    hbm, tf, kind = peaks()
+    greedy = sampling(temperature=0.0)
+    rows = []
+    for name in names:
+        V = model_dir.NURINEX_SHAPES[name][0]
+        row = {"shape": name, "sizes": dict(zip(("vocab", "width", "layers", "heads", "kv_heads", "dim", "r_heads", "r_dim", "ff", "rank"),
+                                                model_dir.NURINEX_SHAPES[name]))}
+        with tempfile.TemporaryDirectory() as tmp:
+            model_dir.nurinex_named(tmp, name)
+            m = CudaNurinex(tmp, ctx=2304)
+        cache = m.new_cache()
+        fcb.take_launch_count()
+
+        def best(fn, read, reps):
+            fn()
+            fn()
+            fn()
+            vals = []
+            for _ in range(reps):
+                fn()
+                vals.append(read())
+            return statistics.median(vals)
+
+        for T in prompts:
+            ids = synth.token_ids(1, T + 1, V)
+
+            def prefill():
+                cache.clear()
+                m.feed(ids[:T], cache, [T - 1])
+            ms = best(prefill, lambda: m.last_forward_ms, a.steps)
+            _, flop, _ = nurinex_work(name, T, 0, 1)
+            flop_p = flop - 2.0 * V * model_dir.NURINEX_SHAPES[name][1] * (T - 1)
+            row[f"prefill_{T}"] = {"tokens_per_s": T / ms * 1e3, "ms": ms, "tflops": flop_p / ms / 1e9, "frac": flop_p / ms / 1e9 / tf}
+            ms = best(lambda: m.score_from(ids, 1), lambda: m.last_forward_ms, a.steps)
+            row[f"score_{T}"] = {"positions_per_s": T / ms * 1e3, "ms": ms, "tflops": flop / ms / 1e9, "frac": flop / ms / 1e9 / tf}
+        for start in (PROMPT, 1920):
+            prompt = synth.token_ids(0, start, V)
+            n_new = NEW_TOKENS
+            ms = best(lambda: m.generate(prompt, n_new, greedy, cache=cache), lambda: cache.last_decode_ms, a.steps)
+            _, _, byts = nurinex_work(name, 1, start, n_new)
+            row[f"decode_from_{start}"] = {"tokens_per_s": n_new / ms * 1e3, "us_per_token": ms / n_new * 1e3,
+                                           "gbs": byts * n_new / ms / 1e6, "frac": byts * n_new / ms / 1e6 / hbm}
+        row["gpu_launches"] = int(fcb.take_launch_count())
+        m.close()
+        if with_llama:
+            sml = synth.SynthLlama(*llama_twin(name), math_mode=fcb.FC_MATH_BF16X3)
+            gl = CudaLlama.from_synth(sml)
+            lc = gl.new_cache()
+            c = sml.dims
+            qd, kvd = c["n_head"] * c["head_dim"], c["n_kv_head"] * c["head_dim"]
+            for T in prompts:
+                ids = synth.token_ids(1, T, V).reshape(1, T)
+                ms = best(lambda: gl.score_sequences(ids, batch_windows=1), lambda: gl.last_score_ms, a.steps)
+                flop = 2.0 * sml.q8_weight_bytes * 32 / 34 * T + c["n_layer"] * 4.0 * qd * T * (T + 1) / 2
+                row[f"llama_score_{T}"] = {"positions_per_s": T / ms * 1e3, "ms": ms, "tflops": flop / ms / 1e9, "frac": flop / ms / 1e9 / tf}
+            for start in (PROMPT, 1920):
+                prompt = synth.token_ids(0, start, V)
+                ms = best(lambda: gl.generate(prompt, NEW_TOKENS, greedy, cache=lc), lambda: lc.last_decode_ms, a.steps)
+                byts = sml.q8_weight_bytes + c["n_layer"] * 2 * (start + NEW_TOKENS / 2) * kvd * 4
+                row[f"llama_decode_from_{start}"] = {"tokens_per_s": NEW_TOKENS / ms * 1e3, "us_per_token": ms / NEW_TOKENS * 1e3,
+                                                     "gbs": byts * NEW_TOKENS / ms / 1e6, "frac": byts * NEW_TOKENS / ms / 1e6 / hbm}
+            gl.close()
+        rows.append(row)
+    main_row = rows[len(rows) // 2]
+    print(json.dumps({
+        "metric": "Nurinex batch-1 greedy decode tokens/s (bf16)", "value": main_row[f"decode_from_{PROMPT}"]["tokens_per_s"], "unit": "tokens/s",
+        "n_gpus": 1, "steps": a.steps, "warmup": 3, "higher_is_better": True, "scaling": "n/a", "vs_baseline": None, "dtype": "bf16",
+        "data": "synthetic", "config": {"workload": "random weights; value is the middle shape; %d-token prompt + %d greedy tokens; weights of every "
+                                                    "shape exceed the L2" % (PROMPT, NEW_TOKENS)},
+        "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "kind": kind}, "shapes": rows}))
+
+
 def run_case(a):
     """Small self-terminating cases for profiler captures (same kernels as the workloads)."""
     import ctypes as C
@@ -325,6 +431,31 @@ def run_case(a):
             byts = raw.size + 4 * a.m * (a.k + a.n)
             print(f"ggml type {t} M={a.m} K={a.k} N={a.n}: {ms * 1e3:.1f} us, {byts / ms / 1e6:.1f} GB/s")
         _lib.lib().fc_ggml_weight_free(h)
+        return
+    if a.case.startswith("nurinex"):
+        import tempfile
+        from ferrum_cpu_b200 import model_dir
+        from ferrum_cpu_b200.engine import sampling
+        from ferrum_cpu_b200.nurinex import CudaNurinex
+        name = a.model if a.model in model_dir.NURINEX_SHAPES else "nurinex-1b"
+        if a.layers:
+            shape = list(model_dir.NURINEX_SHAPES[name])
+            shape[2] = a.layers
+            model_dir.NURINEX_SHAPES[name] = tuple(shape)
+        with tempfile.TemporaryDirectory() as tmp:
+            model_dir.nurinex_named(tmp, name)
+            m = CudaNurinex(tmp, ctx=2304)
+        cache = m.new_cache()
+        ids = synth.token_ids(1, a.prompt, m.info.vocab)
+        for _ in range(a.reps):
+            if a.case == "nurinex-prefill":
+                cache.clear()
+                m.feed(ids, cache, [a.prompt - 1])
+                print(f"{name} prefill {a.prompt} tokens: device {m.last_forward_ms:.3f} ms, launches {fcb.take_launch_count()}")
+            else:
+                m.generate(ids, a.tokens, sampling(temperature=0.0), cache=cache)
+                print(f"{name} decode {a.tokens} tokens: device {cache.last_decode_ms / a.tokens * 1e3:.1f} us/token, launches {fcb.take_launch_count()}")
+        m.close()
         return
     if a.case.startswith("llama"):
         from ferrum_cpu_b200.engine import sampling
@@ -460,14 +591,17 @@ def main():
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=5)
     ap.add_argument("--warmup", type=int, default=3)
-    ap.add_argument("--workload", choices=["decode", "score", "both", "streams-medium", "score-medium", "sweep", "tiny", "llama-1b"],
+    ap.add_argument("--workload", choices=["decode", "score", "both", "streams-medium", "score-medium", "sweep", "tiny", "llama-1b", "nurinex"],
                     default="both", help="see the module docstring")
-    ap.add_argument("--case", choices=["decode", "score", "linear", "rowq", "ggml-linear", "streams", "llama-decode", "llama-score"], default=None,
+    ap.add_argument("--case", choices=["decode", "score", "linear", "rowq", "ggml-linear", "streams", "llama-decode", "llama-score",
+                                       "nurinex-decode", "nurinex-prefill"], default=None,
                     help="run one small self-terminating case (for profiler captures) instead of a workload")
     ap.add_argument("--model", default="small")
     ap.add_argument("--tokens", type=int, default=8)
     ap.add_argument("--prompt", type=int, default=32)
     ap.add_argument("--windows", type=int, default=4)
+    ap.add_argument("--layers", type=int, default=0, help="--case nurinex-*: layers of the shape (0: its own number)")
+    ap.add_argument("--shapes", default="nurinex-small,nurinex-1b,nurinex-7b-layers", help="--workload nurinex: which shapes")
     ap.add_argument("--streams", type=int, default=8)
     ap.add_argument("--m", type=int, default=1)
     ap.add_argument("--k", type=int, default=768)
@@ -527,6 +661,12 @@ def main():
         return float(t.item())
 
     hbm_peak, tf_peak, peak_kind = peaks()
+    if args.workload == "nurinex":
+        if rank == 0:
+            run_nurinex(args, args.shapes.split(","))
+        if world > 1:
+            dist.destroy_process_group()
+        return
     if args.workload == "streams-medium":
         # the decode half of the medium-shaped configuration: 64 streams split over the ranks
         res = run_streams(fcb, synth, shard, "medium", 64, local, rank, world, args.steps, barrier, max_over_ranks, hbm_peak, peak_kind)

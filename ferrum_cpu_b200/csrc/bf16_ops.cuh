@@ -103,14 +103,13 @@ struct TalkAttn {
 // proj rows: q | k | v. qm [M][H * kd], bf16 or f32; caches in the same type.
 int launch_talk_prep(const TalkAttn& t, const float* proj, int ldp, int M, int pos0, float factor, void* qm, void* kc, void* vc, bool f32,
                      cudaStream_t st);
-// Rows of a portion against the cache (positions 0 .. pos0 + i), CUDA cores, f32 arithmetic; out rows ldo apart.
-// f32: queries, caches and output are f32, else bf16. Queries prepared with factor 1.
-int launch_talk_prefill(const TalkAttn& t, const void* qm, const void* kc, const void* vc, int M, int pos0, void* out, int ldo, bool f32,
-                        cudaStream_t st);
-// The same on tcgen05 (bf16, shapes of talk_tc_fits), queries prepared with factor log2(e).
+// Rows of a portion against an f32 cache (positions 0 .. pos0 + i) on CUDA cores; out rows ldo apart. Queries prepared
+// with factor 1; value heads of at most 256.
+int launch_talk_prefill_f32(const TalkAttn& t, const float* qm, const float* kc, const float* vc, int M, int pos0, float* out, int ldo,
+                            cudaStream_t st);
+// The same on tcgen05 with bf16 queries, cache and output; queries prepared with factor log2(e).
 int launch_talk_prefill_tc(const TalkAttn& t, const void* qm, const void* kc, const void* vc, int M, int pos0, int ctx, void* out, int ldo,
                            int* status, cudaStream_t st);
-bool talk_tc_fits(const TalkAttn& t);
 constexpr float kLog2e = 1.4426950408889634f;
 
 // ---- wkv.cu: linear-attention state with per-channel decay and a bonus for the current token --------

@@ -490,10 +490,9 @@ int layer_forward(fc_nurinex* m, fc_nurinex_cache* s, int l, int M, int pos0, in
         FC_TRY(launch_wkv_finish(m->wkv_o, rd, m->proj + w.off_g, ldp, w.rnorm, (float)m->cfg.eps, M, w.rH, w.rdim, m->ro, w.ro.K_pad, m->f32, m->side));
     }
     FC_CUDA(cudaEventRecord(m->join, m->side));
-    const bool tensor = !m->f32 && talk_tc_fits(w.t);
-    FC_TRY(launch_talk_prep(w.t, m->proj, ldp, M, pos0, tensor ? kLog2e : 1.0f, m->qm, s->kc[l], s->vc[l], m->f32, st));
-    if (tensor) FC_TRY(launch_talk_prefill_tc(w.t, m->qm, s->kc[l], s->vc[l], M, pos0, m->ctx, m->att, w.lo.K_pad, m->status, st));
-    else FC_TRY(launch_talk_prefill(w.t, m->qm, s->kc[l], s->vc[l], M, pos0, m->att, w.lo.K_pad, m->f32, st));
+    FC_TRY(launch_talk_prep(w.t, m->proj, ldp, M, pos0, m->f32 ? 1.0f : kLog2e, m->qm, s->kc[l], s->vc[l], m->f32, st));
+    if (m->f32) FC_TRY(launch_talk_prefill_f32(w.t, (const float*)m->qm, (const float*)s->kc[l], (const float*)s->vc[l], M, pos0, (float*)m->att, w.lo.K_pad, st));
+    else FC_TRY(launch_talk_prefill_tc(w.t, m->qm, s->kc[l], s->vc[l], M, pos0, m->ctx, m->att, w.lo.K_pad, m->status, st));
     FC_CUDA(cudaStreamWaitEvent(st, m->join, 0));
     const size_t stride = (size_t)R * d;
     if (m->f32) {

@@ -5,8 +5,8 @@
 // q'_h = [sum_{g in group 0} talk[h][g] q_g | sum_{g in group 1} ... ], plus a per-head table of the distance whose
 // heads are mixed once at load. So after `talk_prep_kernel` this is ordinary attention with one wide shared key head.
 //
-//   talk_prep_kernel      one CTA per token: mixed queries out, key row and normed value row into the cache
-//   talk_prefill_kernel   16 query rows x one head per CTA, f32 CUDA cores, online softmax over key tiles of 32
+//   talk_prep_kernel          one CTA per token: mixed queries out, key row and normed value row into the cache
+//   talk_prefill_f32_kernel   16 query rows x one head per CTA, CUDA cores, online softmax over key tiles of 32
 // Bound: prep HBM / L2; prefill fp32 FMA (the tcgen05 form is talk_attn_tc.cu).
 #include <algorithm>
 
@@ -20,11 +20,6 @@ template <class T>
 __device__ __forceinline__ void put(T* p, float v) {
     if constexpr (sizeof(T) == 2) *p = __bfloat16_as_ushort(__float2bfloat16_rn(v));
     else *p = v;
-}
-template <class T>
-__device__ __forceinline__ float get(const T* p) {
-    if constexpr (sizeof(T) == 2) return __uint_as_float((uint32_t)*p << 16);
-    else return *p;
 }
 }  // namespace
 
@@ -114,9 +109,8 @@ int launch_talk_prep(const TalkAttn& t, const float* proj, int ldp, int M, int p
 namespace {
 constexpr int QR = 16, KT = 32, KC = 64, PNT = 128, VCOLS = 2;     // value columns per thread: heads of at most 256
 }
-template <class T>
-__global__ void __launch_bounds__(PNT) talk_prefill_kernel(const TalkAttn t, const T* __restrict__ qm, const T* __restrict__ kc,
-                                                           const T* __restrict__ vc, int M, int pos0, T* __restrict__ out, int ldo) {
+__global__ void __launch_bounds__(PNT) talk_prefill_f32_kernel(const TalkAttn t, const float* __restrict__ qm, const float* __restrict__ kc,
+                                                               const float* __restrict__ vc, int M, int pos0, float* __restrict__ out, int ldo) {
     __shared__ float Qs[QR][KC + 1], Ks[KT][KC + 1], P[QR][KT + 1];
     __shared__ float corr_s[QR], l_s[QR];
     const int tid = threadIdx.x, h = blockIdx.y, row0 = (gridDim.x - 1 - blockIdx.x) * QR, kv = h / (t.H / t.KV);
@@ -135,11 +129,11 @@ __global__ void __launch_bounds__(PNT) talk_prefill_kernel(const TalkAttn t, con
             __syncthreads();
             for (int i = tid; i < QR * KC; i += PNT) {
                 const int r = i / KC, e = i - r * KC;
-                Qs[r][e] = r < rows && e0 + e < t.kd ? get(qm + ((size_t)(row0 + r) * t.H + h) * t.kd + e0 + e) : 0.0f;
+                Qs[r][e] = r < rows && e0 + e < t.kd ? qm[((size_t)(row0 + r) * t.H + h) * t.kd + e0 + e] : 0.0f;
             }
             for (int i = tid; i < KT * KC; i += PNT) {
                 const int r = i / KC, e = i - r * KC;
-                Ks[r][e] = k0 + r <= last && e0 + e < t.kd ? get(kc + (size_t)(k0 + r) * t.kd + e0 + e) : 0.0f;
+                Ks[r][e] = k0 + r <= last && e0 + e < t.kd ? kc[(size_t)(k0 + r) * t.kd + e0 + e] : 0.0f;
             }
             __syncthreads();
 #pragma unroll 8
@@ -179,9 +173,9 @@ __global__ void __launch_bounds__(PNT) talk_prefill_kernel(const TalkAttn t, con
             if (col >= t.vdim) continue;
 #pragma unroll
             for (int r = 0; r < QR; ++r) acc[c][r] *= corr_s[r];
-            const T* v = vc + ((size_t)k0 * t.KV + kv) * t.vp + col;
+            const float* v = vc + ((size_t)k0 * t.KV + kv) * t.vp + col;
             for (int j = 0; j < nk; ++j) {
-                const float x = get(v + (size_t)j * t.KV * t.vp);
+                const float x = v[(size_t)j * t.KV * t.vp];
 #pragma unroll
                 for (int r = 0; r < QR; ++r) acc[c][r] = fmaf(P[r][j], x, acc[c][r]);
             }
@@ -194,15 +188,13 @@ __global__ void __launch_bounds__(PNT) talk_prefill_kernel(const TalkAttn t, con
         if (col >= t.vdim) continue;
 #pragma unroll
         for (int r = 0; r < QR; ++r)
-            if (r < rows) put(out + (size_t)(row0 + r) * ldo + (size_t)h * t.vdim + col, acc[c][r] / l_s[r]);
+            if (r < rows) out[(size_t)(row0 + r) * ldo + (size_t)h * t.vdim + col] = acc[c][r] / l_s[r];
     }
 }
-int launch_talk_prefill(const TalkAttn& t, const void* qm, const void* kc, const void* vc, int M, int pos0, void* out, int ldo, bool f32,
-                        cudaStream_t st) {
-    const dim3 grid((M + QR - 1) / QR, t.H);
-    if (f32) talk_prefill_kernel<float><<<grid, PNT, 0, st>>>(t, (const float*)qm, (const float*)kc, (const float*)vc, M, pos0, (float*)out, ldo);
-    else talk_prefill_kernel<uint16_t><<<grid, PNT, 0, st>>>(t, (const uint16_t*)qm, (const uint16_t*)kc, (const uint16_t*)vc, M, pos0,
-                                                             (uint16_t*)out, ldo);
+int launch_talk_prefill_f32(const TalkAttn& t, const float* qm, const float* kc, const float* vc, int M, int pos0, float* out, int ldo,
+                            cudaStream_t st) {
+    if (t.vdim > VCOLS * PNT) return fail(FC_E_SHAPE, "value heads of %d: at most %d", t.vdim, VCOLS * PNT);
+    talk_prefill_f32_kernel<<<dim3((M + QR - 1) / QR, t.H), PNT, 0, st>>>(t, qm, kc, vc, M, pos0, out, ldo);
     FC_LAUNCHED();
     return FC_OK;
 }

@@ -2,8 +2,8 @@
 // scale, temperature and log2(e) inside), keys and values straight from the bf16 cache.
 //
 // One CTA owns 128 query rows of one head; key tiles of 64.
-//   warp 4      TMA: the query tile once (k-chunks of 64 columns), then per key tile the chunks of the wide key row
-//               through a ring, and the value tile of the head's key/value head (two buffers)
+//   warp 4      TMA: the query tile once (k-chunks of 64 columns; a tile too wide to stay travels again with every key
+//               tile), then per key tile the chunks of the wide key row through a ring, and the value tile of the head's key/value head (two buffers)
 //   warp 5      tcgen05.mma: S = q' K^T into one of two score buffers, one tile ahead; O += P V (V consumed MN-major),
 //               P as bf16 hi + lo so that the weights keep 16 bits
 //   warps 0-3   one query row per thread: score + bias[distance] (a 191-entry slice of the head's table per tile, -inf
@@ -40,6 +40,7 @@ struct Bars {
 };
 struct Args {
     int M, pos0, kd, nkc, ks, nv, H, KV, vdim, vp, far, ldo;
+    int q_stream;        // the query tile is too wide to stay in shared memory: its chunks travel with the key chunks
     const float *bias, *sink;
     uint16_t* out;
     int* status;
@@ -47,15 +48,17 @@ struct Args {
     int withhold;
     uint32_t tmem_cols;
 };
-size_t smem_bytes(int nkc, int ks, int nv) {
-    return (size_t)nkc * Q_CHUNK + (size_t)ks * K_CHUNK + (size_t)2 * nv * K_CHUNK + 2 * P_BYTES + 1024 + sizeof(Bars);
+size_t smem_bytes(int nkc, int ks, int nv, bool q_stream) {
+    return (q_stream ? (size_t)ks * Q_CHUNK : (size_t)nkc * Q_CHUNK) + (size_t)ks * K_CHUNK + (size_t)2 * nv * K_CHUNK + 2 * P_BYTES + 1024 +
+           sizeof(Bars);
 }
-// Key-ring stages that fit: as many as keep two CTAs on an SM, else as many as fit one. 0: the shape does not fit.
-int plan_stages(int nkc, int nv) {
-    for (int ks = MAX_KS; ks >= 3; --ks)
-        if (smem_bytes(nkc, ks, nv) <= 113 * 1024) return ks;
+// Key-ring stages: as many as keep two CTAs on an SM, else as many as fit one. 0: does not fit.
+int plan_stages(int nkc, int nv, bool q_stream) {
+    if (!q_stream)
+        for (int ks = MAX_KS; ks >= 3; --ks)
+            if (smem_bytes(nkc, ks, nv, false) <= 113 * 1024) return ks;
     for (int ks = MAX_KS; ks >= 2; --ks)
-        if (smem_bytes(nkc, ks, nv) <= 226 * 1024) return ks;
+        if (smem_bytes(nkc, ks, nv, q_stream) <= 226 * 1024) return ks;
     return 0;
 }
 }  // namespace
@@ -65,7 +68,7 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
                        const Args a) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char* smem = (unsigned char*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
-    unsigned char* sk = smem + a.nkc * Q_CHUNK;
+    unsigned char* sk = smem + (a.q_stream ? a.ks : a.nkc) * Q_CHUNK;
     unsigned char* sv_ = sk + a.ks * K_CHUNK;
     unsigned char* sp = sv_ + 2 * a.nv * K_CHUNK;
     Bars* bars = (Bars*)(sp + 2 * P_BYTES);
@@ -95,8 +98,8 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
 
     if (warp == TMA_WARP) {
         if (lane == 0 && !a.withhold) {
-            mbar_expect_tx(&bars->q_full, a.nkc * Q_CHUNK);
-            for (int c = 0; c < a.nkc; ++c) tma_load_2d(smem + c * Q_CHUNK, &mq, h * a.kd + c * CH, q0, &bars->q_full);
+            if (!a.q_stream) mbar_expect_tx(&bars->q_full, a.nkc * Q_CHUNK);
+            for (int c = 0; !a.q_stream && c < a.nkc; ++c) tma_load_2d(smem + c * Q_CHUNK, &mq, h * a.kd + c * CH, q0, &bars->q_full);
             int it = 0, nvt = 0;
             bool ok = true;
             for (int kt = 0; kt < n_kt && ok; ++kt) {
@@ -104,7 +107,8 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
                     const int s = it % a.ks;
                     ok = wait(&bars->k_empty[s], ((it / a.ks) & 1) ^ 1);
                     if (!ok) break;
-                    mbar_expect_tx(&bars->k_full[s], K_CHUNK);
+                    mbar_expect_tx(&bars->k_full[s], a.q_stream ? K_CHUNK + Q_CHUNK : K_CHUNK);
+                    if (a.q_stream) tma_load_2d(smem + s * Q_CHUNK, &mq, h * a.kd + c * CH, q0, &bars->k_full[s]);
                     tma_load_2d(sk + s * K_CHUNK, &mk, c * CH, kt * KT, &bars->k_full[s]);
                     ++it;
                 }
@@ -120,7 +124,7 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
                     const long long t0 = clock64();
                     while (!mbar_try_wait(b, par) && clock64() - t0 < a.wait_cycles) {}
                 };
-                drain(&bars->q_full, 0);
+                if (!a.q_stream) drain(&bars->q_full, 0);
                 for (int i = max(0, it - a.ks); i < it; ++i) drain(&bars->k_full[i % a.ks], (i / a.ks) & 1);
                 for (int i = max(0, nvt - 2); i < nvt; ++i) drain(&bars->v_full[i & 1], (i >> 1) & 1);
             }
@@ -138,7 +142,7 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
                     const int s = it % a.ks;
                     if (!wait(&bars->k_full[s], (it / a.ks) & 1)) return false;
                     fence_after();
-                    const uint64_t qd = smem_desc(sb + c * Q_CHUNK), kd = smem_desc(kb + s * K_CHUNK);
+                    const uint64_t qd = smem_desc(sb + (a.q_stream ? s : c) * Q_CHUNK), kd = smem_desc(kb + s * K_CHUNK);
 #pragma unroll
                     for (int ks = 0; ks < CH / 16; ++ks) umma(tmem + b * KT, qd + (uint64_t)(ks * 2), kd + (uint64_t)(ks * 2), IDESC_S, (c | ks) != 0);
                     umma_commit(&bars->k_empty[s]);
@@ -146,7 +150,7 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
                 umma_commit(&bars->s_full[b]);
                 return true;
             };
-            bool ok = wait(&bars->q_full, 0) && scores(0);
+            bool ok = (a.q_stream || wait(&bars->q_full, 0)) && scores(0);
             for (int kt = 0; kt < n_kt && ok; ++kt) {
                 if (kt + 1 < n_kt && !(ok = scores(kt + 1))) break;
                 const int b = kt & 1;
@@ -279,15 +283,14 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
     }
 }
 
-bool talk_tc_fits(const TalkAttn& t) { return t.vdim <= 256 && plan_stages((t.kd + CH - 1) / CH, (t.vp + CH - 1) / CH) > 0; }
-
 int launch_talk_prefill_tc(const TalkAttn& t, const void* qm, const void* kc, const void* vc, int M, int pos0, int ctx, void* out, int ldo,
                            int* status, cudaStream_t st) {
     Args a = {};
     a.nkc = (t.kd + CH - 1) / CH;
     a.nv = (t.vp + CH - 1) / CH;
-    a.ks = plan_stages(a.nkc, a.nv);
-    if (!talk_tc_fits(t)) return fail(FC_E_SHAPE, "key rows of %d and value heads of %d do not fit the tensor-core attention", t.kd, t.vdim);
+    if (t.vdim > 256) return fail(FC_E_SHAPE, "value heads of %d do not fit the tensor-core attention", t.vdim);
+    a.ks = plan_stages(a.nkc, a.nv, false);
+    if (!a.ks) { a.q_stream = 1; a.ks = plan_stages(a.nkc, a.nv, true); }
     static bool attr_set[64] = {};
     int dev = 0;
     FC_CUDA(cudaGetDevice(&dev));
@@ -303,7 +306,7 @@ int launch_talk_prefill_tc(const TalkAttn& t, const void* qm, const void* kc, co
     a.bias = t.bias; a.sink = t.sink; a.out = (uint16_t*)out; a.status = status;
     a.wait_cycles = g_debug.wait_cycles; a.withhold = g_debug.withhold;
     a.tmem_cols = a.nv <= 2 ? 256 : 512;
-    talk_prefill_tc_kernel<<<dim3((M + QT - 1) / QT, t.H), THREADS, smem_bytes(a.nkc, a.ks, a.nv), st>>>(mq, mk, mv, a);
+    talk_prefill_tc_kernel<<<dim3((M + QT - 1) / QT, t.H), THREADS, smem_bytes(a.nkc, a.ks, a.nv, a.q_stream), st>>>(mq, mk, mv, a);
     FC_LAUNCHED();
     return FC_OK;
 }

@@ -56,6 +56,24 @@ def nurinex_config(vocab, width, layers, eps=1e-5, emb_scale=1.0):
     return {"architecture": "Nurinex", "vocab": vocab, "width": width, "embedding": {"scale": emb_scale}, "norm": {"eps": eps}, "layers": layers}
 
 
+# name -> (vocab, width, layers, query heads, key/value heads, head dim, recurrence heads, recurrence dim, ff, decay rank):
+# layers as those of real models, few of them. The first has the layer sizes of the 1B-class Llama shape in synth.py.
+NURINEX_SHAPES = {
+    "nurinex-small": (32000, 1024, 12, 16, 4, 64, 16, 64, 4096, 32),
+    "nurinex-1b": (32000, 2048, 8, 32, 8, 64, 32, 64, 8192, 64),
+    "nurinex-7b-layers": (32000, 4096, 3, 32, 8, 128, 64, 64, 11008, 64),
+}
+
+
+def nurinex_named(path, name, seed=0):
+    """Writes a synthetic model of a named shape; returns its configuration."""
+    V, d, n, H, G, hd, rH, rD, ff, rank = NURINEX_SHAPES[name]
+    layer = nurinex_layer(heads=H, kv_heads=G, dim=hd, vdim=hd, bias_max=1024, every=512, r_heads=rH, r_dim=rD, ff=ff)
+    config = nurinex_config(V, d, [layer] * n)
+    write(path, config, nurinex_tensors(config, seed=seed, bias_rows=32, rank=rank))
+    return config
+
+
 def nurinex_tensors(config, seed=0, bias_rows=12, rank=8):
     """Random bf16 weights of the shapes a configuration asks for: name -> uint16 array. bias_rows and rank are numbers
     or one per layer."""

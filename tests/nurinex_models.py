@@ -32,7 +32,7 @@ def configs():
             L(heads=8, kv_heads=8, dim=16, vdim=32, bias_max=64, every=20, r_heads=1, r_dim=136, ff=64, weights_of=1),
             L(heads=8, kv_heads=8, dim=16, vdim=32, bias_max=64, every=20, r_heads=1, r_dim=136, ff=64),
         ], emb_scale=3.0), [0, 8], [0, 40]),
-        # beyond what the tensor-core attention holds (its f32 form takes over), value heads of 200
+        # query tiles too wide to stay in shared memory, value heads of four chunks
         "huge": (MD.nurinex_config(150, 64, [
             L(heads=10, kv_heads=10, dim=120, vdim=200, bias_max=50, every=9, r_heads=1, r_dim=32, ff=64),
         ]), 6, 4),
