@@ -157,7 +157,6 @@ struct MixerDecode {
     float* att;                        // [H * vdim]
     float *part, *part_ml;             // [splits][H][vdim], [splits][H][2]
     int max_splits; unsigned int* counter;
-    int kv_block;                      // filled by the launcher: key heads staged at a time
     // recurrence
     int rH, rdim, rank;
     const float *r, *k, *v, *g, *w1;   // projections of the row (w1: [rank])
@@ -166,6 +165,6 @@ struct MixerDecode {
     float* wkv_state; float* ro;
     StepState* state;
 };
-int launch_mixer_decode(MixerDecode a, cudaStream_t st);
+int launch_mixer_decode(const MixerDecode& a, cudaStream_t st);
 
 }  // namespace fc

@@ -427,13 +427,25 @@ int check_status(fc_nurinex* m) {
 }
 
 // ---------------------------------------------------------------------- a portion of tokens
-// How many partial sums the feed-forward's second product is cut into: few output tiles leave SMs idle while the
-// longest K decides, so short portions split it.
+// How many partial sums the feed-forward's second product is cut into. The tiles of the three output products go round
+// robin over the SMs, the longest first; with few tiles the feed-forward's long K decides, so the number is the one whose
+// busiest SM has the least to do (each further partial sum counts as a little extra traffic).
 int ff_splits(const NxWeights& w, int M) {
     if (!w.ff) return 0;
-    const int tiles = 3 * ((w.down.N + 127) / 128) * ((M + 255) / 256), kb = w.down.K_pad / 64, other = std::max(w.lo.K_pad, w.ro.K_pad) / 64;
-    if (tiles >= 4 * 148) return 1;
-    return std::max(1, std::min({kFfSplits, kb / std::max(other, 8), kb}));
+    const int tiles = ((w.down.N + 127) / 128) * ((M + 255) / 256), kb = w.down.K_pad / 64, lo = w.lo.K_pad / 64, ro = w.ro.K_pad / 64;
+    int best = 1;
+    double least = 1e30;
+    for (int f = 1; f <= std::min(kFfSplits, kb); ++f) {
+        std::vector<int> load(148, 0);
+        int at = 0;
+        auto add = [&](int n, int cost) { for (int i = 0; i < n; ++i) load[at++ % 148] += cost + 4; };
+        add(tiles * f, (kb + f - 1) / f);
+        add(tiles, lo);
+        add(tiles, ro);
+        const double cost = *std::max_element(load.begin(), load.end()) * (1.0 + 0.03 * (f - 1));
+        if (cost < least) { least = cost; best = f; }
+    }
+    return best;
 }
 
 SideOutputs outputs_of(const NxWeights& w, const float* outs, size_t stride, int n_ff) {

@@ -39,31 +39,40 @@ __global__ void __launch_bounds__(256) talk_prep_kernel(const TalkAttn t, const 
     __syncthreads();
     const int width = t.KV * dim;
     T* out = qm + (size_t)row * H * t.kd;
-    for (int f = tid; f < t.kd; f += 256) {
-        if (f >= width) {
-            for (int h = 0; h < H; ++h) put(out + (size_t)h * t.kd + f, 0.0f);
-            continue;
-        }
-        const int c = f / dim, e = f - c * dim;
-        const float* qc = q + (size_t)c * per * dim + e;
+    // two neighbouring columns a thread (kd is even); they may belong to different key/value heads
+    for (int f = 2 * tid; f < t.kd; f += 512) {
+        const int c0 = min(f, width - 1) / dim, c1 = min(f + 1, width - 1) / dim;
+        const float z0 = f < width ? 1.0f : 0.0f, z1 = f + 1 < width ? 1.0f : 0.0f;
+        const float* q0 = q + (size_t)c0 * per * dim + (min(f, width - 1) - c0 * dim);
+        const float* q1 = q + (size_t)c1 * per * dim + (min(f + 1, width - 1) - c1 * dim);
+        auto store = [&](int h, float a, float b) {
+            T* to = out + (size_t)h * t.kd + f;
+            if constexpr (sizeof(T) == 2) *(uint32_t*)to = tc::pack2(a, b);
+            else *(float2*)to = make_float2(a, b);
+        };
         if constexpr (PER > 0) {
-            float qr[PER];
+            float a[PER], b[PER];
 #pragma unroll
-            for (int g = 0; g < PER; ++g) qr[g] = qc[g * dim];
-            for (int h = 0; h < H; ++h) {
-                const float* w = tk + h * H + c * PER;
-                float s = 0.0f;
+            for (int g = 0; g < PER; ++g) { a[g] = q0[g * dim] * z0; b[g] = q1[g * dim] * z1; }
+            if (c0 == c1) {
+#pragma unroll 4
+                for (int h = 0; h < H; ++h) {
+                    const float* w = tk + h * H + c0 * PER;
+                    float x = 0.0f, y = 0.0f;
 #pragma unroll
-                for (int g = 0; g < PER; ++g) s = fmaf(w[g], qr[g], s);
-                put(out + (size_t)h * t.kd + f, s);
+                    for (int g = 0; g < PER; ++g) { x = fmaf(w[g], a[g], x); y = fmaf(w[g], b[g], y); }
+                    store(h, x, y);
+                }
+                continue;
             }
-        } else {
-            for (int h = 0; h < H; ++h) {
-                const float* w = tk + h * H + c * per;
-                float s = 0.0f;
-                for (int g = 0; g < per; ++g) s = fmaf(w[g], qc[g * dim], s);
-                put(out + (size_t)h * t.kd + f, s);
+        }
+        for (int h = 0; h < H; ++h) {
+            float x = 0.0f, y = 0.0f;
+            for (int g = 0; g < per; ++g) {
+                x = fmaf(tk[h * H + c0 * per + g], q0[g * dim] * z0, x);
+                y = fmaf(tk[h * H + c1 * per + g], q1[g * dim] * z1, y);
             }
+            store(h, x, y);
         }
     }
     const float* ks = src + H * dim;

@@ -2,13 +2,14 @@
 // scale, temperature and log2(e) inside), keys and values straight from the bf16 cache.
 //
 // One CTA owns 128 query rows of one head; key tiles of 64.
-//   warp 4      TMA: the query tile once (k-chunks of 64 columns; a tile too wide to stay travels again with every key
-//               tile), then per key tile the chunks of the wide key row through a ring, and the value tile of the head's key/value head (two buffers)
-//   warp 5      tcgen05.mma: S = q' K^T into one of two score buffers, one tile ahead; O += P V (V consumed MN-major),
+//   warp 8      TMA: the query tile once (k-chunks of 64 columns; a tile too wide to stay travels again with every key
+//               tile), then per key tile the chunks of the wide key row through a ring, and the value tile of the head's
+//               key/value head (two buffers)
+//   warp 9      tcgen05.mma: S = q' K^T into one of two score buffers, one tile ahead; O += P V (V consumed MN-major),
 //               P as bf16 hi + lo so that the weights keep 16 bits
-//   warps 0-3   one query row per thread: score + bias[distance] (a 191-entry slice of the head's table per tile, -inf
-//               for keys ahead of the query), online softmax in base 2 that starts from the sink (max = sink, sum = 1),
-//               P to shared memory. O stays in TMEM; it is rescaled only when a row's maximum has grown by more than 8.
+//   warps 0-7   two threads per query row, 32 keys each: score + bias[distance] (a 191-entry slice of the head's table per
+//               tile, -inf for keys ahead of the query), online softmax in base 2 that starts from the sink (max = sink,
+//               sum = 1), P to shared memory. O stays in TMEM; it is rescaled only when a row's maximum has grown by more than 8.
 // Every mbarrier wait is bounded; on a timeout the status word is raised and the CTA leaves.
 //
 // Bound: tensor pipe / special-function unit. Per (query, key) pair and head KV * dim + 2 vdim multiply-adds executed.
@@ -27,7 +28,7 @@ constexpr int Q_CHUNK = QT * CH * 2;       // 16 KiB
 constexpr int K_CHUNK = KT * CH * 2;       // 8 KiB
 constexpr int P_BYTES = QT * KT * 2;       // 16 KiB
 constexpr int MAX_KS = 8;
-constexpr int TMA_WARP = 4, MMA_WARP = 5, THREADS = 6 * 32;
+constexpr int SM_WARPS = 8, TMA_WARP = 8, MMA_WARP = 9, THREADS = 10 * 32;
 constexpr uint32_t IDESC_S = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(KT >> 3) << 17) | ((uint32_t)(QT >> 4) << 24);
 constexpr uint32_t IDESC_O = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(CH >> 3) << 17) | ((uint32_t)(QT >> 4) << 24);
 constexpr float GROW = 8.0f;               // log2: how far a row's maximum may run ahead of the one its sums are relative to
@@ -37,6 +38,7 @@ struct Bars {
     uint32_t tmem_base;
     volatile int abort;
     float bias[2][192];
+    float half[2][2][QT];            // per buffer, half of the tile's keys: a row's largest score; at the end its sums
 };
 struct Args {
     int M, pos0, kd, nkc, ks, nv, H, KV, vdim, vp, far, ldo;
@@ -63,7 +65,7 @@ int plan_stages(int nkc, int nv, bool q_stream) {
 }
 }  // namespace
 
-__global__ void __launch_bounds__(THREADS, 2)
+__global__ void __launch_bounds__(THREADS, 1)
 talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv,
                        const Args a) {
     extern __shared__ unsigned char smem_raw[];
@@ -73,7 +75,7 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
     unsigned char* sp = sv_ + 2 * a.nv * K_CHUNK;
     Bars* bars = (Bars*)(sp + 2 * P_BYTES);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * QT, h = blockIdx.y, kv = h / (a.H / a.KV);
+    const int q0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * QT, h = blockIdx.x, kv = h / (a.H / a.KV);
     const int last = a.pos0 + min(a.M, q0 + QT) - 1;       // the last key any row of the tile sees
     const int n_kt = last / KT + 1;
 
@@ -82,9 +84,9 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
         for (int i = 0; i < a.ks; ++i) { mbar_init(&bars->k_full[i], 1); mbar_init(&bars->k_empty[i], 1); }
         for (int i = 0; i < 2; ++i) {
             mbar_init(&bars->v_full[i], 1); mbar_init(&bars->v_empty[i], 1);
-            mbar_init(&bars->s_full[i], 1); mbar_init(&bars->s_empty[i], 4);
+            mbar_init(&bars->s_full[i], 1); mbar_init(&bars->s_empty[i], SM_WARPS);
         }
-        mbar_init(&bars->p_full, 4);
+        mbar_init(&bars->p_full, SM_WARPS);
         mbar_init(&bars->o_done, 1);
         bars->abort = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -133,13 +135,30 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
         if (lane == 0) {
             const uint32_t sb = s32(smem), kb = s32(sk), vb = s32(sv_);
             const uint64_t ph = smem_desc(s32(sp)), pl = smem_desc(s32(sp) + P_BYTES);
-            int it = 0;
+            int it = 0, next_pv = 0;
+            // O += P V of tile next_pv; its P and V have been waited for
+            auto pv = [&]() {
+                const int kt = next_pv++, b = kt & 1;
+                fence_after();
+                for (int c = 0; c < a.nv; ++c) {
+                    const uint64_t vd = smem_desc(vb + (b * a.nv + c) * K_CHUNK);
+#pragma unroll
+                    for (int ks = 0; ks < KT / 16; ++ks) {
+                        umma(tmem_o + c * CH, ph + (uint64_t)(ks * 2), vd + (uint64_t)(ks * 128), IDESC_O, (kt | ks) != 0);
+                        umma(tmem_o + c * CH, pl + (uint64_t)(ks * 2), vd + (uint64_t)(ks * 128), IDESC_O, 1);
+                    }
+                }
+                umma_commit(&bars->v_empty[b]);
+                umma_commit(&bars->o_done);
+            };
             auto scores = [&](int kt) -> bool {
                 const int b = kt & 1;
                 if (!wait(&bars->s_empty[b], ((kt >> 1) & 1) ^ 1)) return false;
                 fence_after();
                 for (int c = 0; c < a.nkc; ++c, ++it) {
                     const int s = it % a.ks;
+                    // the tile before may have become ready while these keys are still on their way
+                    if (next_pv < kt && mbar_test(&bars->p_full, next_pv & 1) && mbar_test(&bars->v_full[next_pv & 1], (next_pv >> 1) & 1)) pv();
                     if (!wait(&bars->k_full[s], (it / a.ks) & 1)) return false;
                     fence_after();
                     const uint64_t qd = smem_desc(sb + (a.q_stream ? s : c) * Q_CHUNK), kd = smem_desc(kb + s * K_CHUNK);
@@ -153,57 +172,57 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
             bool ok = (a.q_stream || wait(&bars->q_full, 0)) && scores(0);
             for (int kt = 0; kt < n_kt && ok; ++kt) {
                 if (kt + 1 < n_kt && !(ok = scores(kt + 1))) break;
-                const int b = kt & 1;
-                ok = wait(&bars->v_full[b], (kt >> 1) & 1) && wait(&bars->p_full, kt & 1);
-                if (!ok) break;
-                fence_after();
-                for (int c = 0; c < a.nv; ++c) {
-                    const uint64_t vd = smem_desc(vb + (b * a.nv + c) * K_CHUNK);
-#pragma unroll
-                    for (int ks = 0; ks < KT / 16; ++ks) {
-                        umma(tmem_o + c * CH, ph + (uint64_t)(ks * 2), vd + (uint64_t)(ks * 128), IDESC_O, (kt | ks) != 0);
-                        umma(tmem_o + c * CH, pl + (uint64_t)(ks * 2), vd + (uint64_t)(ks * 128), IDESC_O, 1);
-                    }
-                }
-                umma_commit(&bars->v_empty[b]);
-                umma_commit(&bars->o_done);
+                if (next_pv > kt) continue;
+                ok = wait(&bars->v_full[kt & 1], (kt >> 1) & 1) && wait(&bars->p_full, kt & 1);
+                if (ok) pv();
             }
         }
     } else {
-        const int r = threadIdx.x;                         // query row of the tile
+        // two threads a query row, each with half of the tile's keys (and of the output's columns)
+        const int hf = warp >> 2, r = (warp & 3) * 32 + lane, tid = threadIdx.x;
         const float* bias = a.bias + (size_t)h * (a.far + 1);
-        float m = a.sink[h] * kLog2e, l = 1.0f;
+        float m = a.sink[h] * kLog2e, l = hf == 0 ? 1.0f : 0.0f;
         unsigned char* ph = sp + r * 128;
         unsigned char* pl = ph + P_BYTES;
-        const uint32_t lane_addr = (uint32_t)(warp * 32) << 16;
+        const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
+        constexpr int HK = KT / 2;
+        auto bias_at = [&](int kt) -> float {              // entry tid of tile kt's slice of the table
+            const int n = a.pos0 + q0 - kt * KT - (KT - 1) + tid;
+            return n < 0 ? -INFINITY : __ldg(bias + min(n, a.far)) * kLog2e;
+        };
+        float next_bias = bias_at(0);
         bool ok = true;
         for (int kt = 0; kt < n_kt; ++kt) {
-            const int b = kt & 1, base = a.pos0 + q0 - kt * KT - (KT - 1);
+            const int b = kt & 1;
             float* bt = bars->bias[b];
-            for (int x = r; x < QT + KT - 1; x += QT) {
-                const int n = base + x;
-                bt[x] = n < 0 ? -INFINITY : bias[min(n, a.far)] * kLog2e;
-            }
-            asm volatile("bar.sync 1, 128;" ::: "memory");
+            if (tid < QT + KT - 1) bt[tid] = next_bias;
+            if (kt + 1 < n_kt) next_bias = bias_at(kt + 1);
             ok = __all_sync(0xffffffffu, wait(&bars->s_full[b], (kt >> 1) & 1));
-            // one warp's timeout must not leave the others at the named barrier: everybody goes on to it,
-            // tile by tile, with waits that the abort flag ends at once
-            float sv[KT];
+            uint32_t sr[HK];
             float mx = -INFINITY;
             if (ok) {
                 fence_after();
-                tmem_ld32(tmem + b * KT + lane_addr, (uint32_t*)sv);
-                tmem_ld32(tmem + b * KT + 32 + lane_addr, (uint32_t*)sv + 32);
+                tmem_ld32(tmem + b * KT + hf * HK + lane_addr, sr);
                 fence_before();
                 __syncwarp();
                 if (lane == 0) mbar_arrive(&bars->s_empty[b]);
-#pragma unroll
-                for (int j = 0; j < KT; ++j) {
-                    sv[j] += bt[r + (KT - 1) - j];
-                    mx = fmaxf(mx, sv[j]);
-                }
-                if (kt > 0) ok = wait(&bars->o_done, (kt - 1) & 1);   // P may be overwritten, O holds tiles 0 .. kt - 1
             }
+            // one warp's timeout must not leave the others at a named barrier: everybody goes on to them, tile by tile, with
+            // waits that the abort flag ends at once
+            asm volatile("bar.sync 1, 256;" ::: "memory");
+            if (ok) {
+#pragma unroll
+                for (int j = 0; j < HK; ++j) {
+                    const float s = __uint_as_float(sr[j]) + bt[r + (KT - 1) - hf * HK - j];
+                    sr[j] = __float_as_uint(s);
+                    mx = fmaxf(mx, s);
+                }
+                bars->half[b][hf][r] = mx;
+            }
+            // the two warps of these 32 rows
+            asm volatile("bar.sync %0, 64;" ::"r"(2 + (warp & 3)) : "memory");
+            if (ok) mx = fmaxf(mx, bars->half[b][hf ^ 1][r]);
+            if (ok && kt > 0) ok = wait(&bars->o_done, (kt - 1) & 1);     // P may be overwritten, O holds tiles 0 .. kt - 1
             ok = __all_sync(0xffffffffu, ok);
             if (ok) {
                 fence_after();
@@ -213,7 +232,7 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
                     l *= corr;
                     m = mn;
                     if (kt > 0)
-                        for (int c = 0; c < 2 * a.nv; ++c) {
+                        for (int c = hf; c < 2 * a.nv; c += 2) {
                             uint32_t o[32];
                             tmem_ld32(tmem_o + c * 32 + lane_addr, o);
 #pragma unroll
@@ -223,16 +242,16 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
                 }
                 float ps = 0.0f;
 #pragma unroll
-                for (int c = 0; c < KT / 8; ++c) {
+                for (int c = 0; c < HK / 8; ++c) {
                     float p[8];
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) { p[e] = ex2_approx(sv[8 * c + e] - m); ps += p[e]; }
+                    for (int e = 0; e < 8; ++e) { p[e] = ex2_approx(__uint_as_float(sr[8 * c + e]) - m); ps += p[e]; }
                     uint4 hi, lo;
                     split2(p[0], p[1], &hi.x, &lo.x);
                     split2(p[2], p[3], &hi.y, &lo.y);
                     split2(p[4], p[5], &hi.z, &lo.z);
                     split2(p[6], p[7], &hi.w, &lo.w);
-                    const int chunk = (c ^ (r & 7)) * 16;
+                    const int chunk = ((hf * (HK / 8) + c) ^ (r & 7)) * 16;
                     *(uint4*)(ph + chunk) = hi;
                     *(uint4*)(pl + chunk) = lo;
                 }
@@ -244,12 +263,14 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
             }
         }
         ok = __all_sync(0xffffffffu, wait(&bars->o_done, (n_kt - 1) & 1) && ok && !bars->abort);
+        bars->half[n_kt & 1][hf][r] = l;                   // not the buffer of the last tile's maxima
+        asm volatile("bar.sync %0, 64;" ::"r"(2 + (warp & 3)) : "memory");
         if (ok) {
             fence_after();
-            const float inv = 1.0f / l;
+            const float inv = 1.0f / (bars->half[n_kt & 1][0][r] + bars->half[n_kt & 1][1][r]);
             const bool store = q0 + r < a.M, vec = (a.vdim & 7) == 0 && (a.ldo & 7) == 0;
             uint16_t* dst = a.out + (size_t)(q0 + r) * a.ldo + (size_t)h * a.vdim;
-            for (int c = 0; c < 2 * a.nv; ++c) {
+            for (int c = hf; c < 2 * a.nv; c += 2) {
                 if (c * 32 >= a.vdim) break;
                 uint32_t o[32];
                 tmem_ld32(tmem_o + c * 32 + lane_addr, o);
@@ -306,7 +327,7 @@ int launch_talk_prefill_tc(const TalkAttn& t, const void* qm, const void* kc, co
     a.bias = t.bias; a.sink = t.sink; a.out = (uint16_t*)out; a.status = status;
     a.wait_cycles = g_debug.wait_cycles; a.withhold = g_debug.withhold;
     a.tmem_cols = a.nv <= 2 ? 256 : 512;
-    talk_prefill_tc_kernel<<<dim3((M + QT - 1) / QT, t.H), THREADS, smem_bytes(a.nkc, a.ks, a.nv, a.q_stream), st>>>(mq, mk, mv, a);
+    talk_prefill_tc_kernel<<<dim3(t.H, (M + QT - 1) / QT), THREADS, smem_bytes(a.nkc, a.ks, a.nv, a.q_stream), st>>>(mq, mk, mv, a);
     FC_LAUNCHED();
     return FC_OK;
 }
