@@ -113,9 +113,12 @@ int launch_talk_prefill_tc(const TalkAttn& t, const void* qm, const void* kc, co
 constexpr float kLog2e = 1.4426950408889634f;
 
 // ---- wkv.cu: linear-attention state with per-channel decay and a bonus for the current token --------
-// o_t = (S + diag(u) k_t v_t^T)^T r_t, S <- diag(w_t) S + k_t v_t^T; state [H][dim][dim] f32 in and out.
+// o_t = (S + diag(u) k_t v_t^T)^T r_t, S <- diag(w_t) S + k_t v_t^T; state [H][dim][dim] f32 in and out. scratch:
+// wkv_scratch_floats(H, dim), for portions long enough to be cut into segments.
+constexpr int kWkvSegments = 8;
+size_t wkv_scratch_floats(int H, int dim);
 int launch_wkv_scan(const float* r, const float* k, const float* v, int ld, const float* w, int ldw, const float* u, float* state, float* o,
-                    int ldo, int M, int H, int dim, cudaStream_t st);
+                    int ldo, int M, int H, int dim, float* scratch, cudaStream_t st);
 // o / rms(o) per head, times norm, times silu(gate): rows of ldy elements, bf16 or f32.
 int launch_wkv_finish(const float* o, int ldo, const float* gate, int ldg, const float* norm, float eps, int M, int H, int dim, void* y,
                       int ldy, bool f32, cudaStream_t st);

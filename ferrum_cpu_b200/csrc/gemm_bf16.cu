@@ -202,36 +202,44 @@ int launch_gemm_bf16_group(const GemmMaps& maps, GemmGroup g, int M, int* status
 }
 
 // ------------------------------------------------------------------------------ true f32 on CUDA cores
-// 64 x 64 tiles, k-steps of 16, 4 x 4 outputs per thread; the bf16 weights are exact in f32, every product and sum is f32.
+// 64 x 64 tiles, k-steps of 32, 4 x 4 outputs per thread; the bf16 weights are exact in f32, every product and sum is f32.
 namespace {
-constexpr int FM = 64, FN = 64, FK = 16;
+constexpr int FM = 64, FN = 64, FK = 32;
 }
 __global__ void __launch_bounds__(256) gemm_bf16w_f32_kernel(const uint16_t* __restrict__ w, int K_pad, int n, const GemmF32 p, int M) {
     __shared__ __align__(16) float As[FK][FM + 4], Bs[FK][FN + 4];
     const int t = threadIdx.x, m0 = blockIdx.y * FM, n0 = blockIdx.x * FN;
-    const int row = t >> 2, k4 = (t & 3) * 4;             // this thread loads 4 consecutive k of one row
+    const int row = t >> 2, k8 = (t & 3) * 8;             // this thread loads 8 consecutive k of one row
     const bool va = m0 + row < M, vb = n0 + row < n;
-    const float* ap = p.a + (size_t)(va ? m0 + row : 0) * p.lda + k4;
-    const uint16_t* bp = w + (size_t)(vb ? n0 + row : 0) * K_pad + k4;
+    const float* ap = p.a + (size_t)(va ? m0 + row : 0) * p.lda + k8;
+    const uint16_t* bp = w + (size_t)(vb ? n0 + row : 0) * K_pad + k8;
     float acc[4][4];
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[i][j] = 0.0f;
     const int ty = t >> 4, tx = t & 15;
-    float4 av = make_float4(0, 0, 0, 0);
-    uint2 bv = make_uint2(0, 0);
+    float4 av[2] = {};
+    uint4 bv = make_uint4(0, 0, 0, 0);
     auto load = [&](int k0) {
-        if (va) av = *(const float4*)(ap + k0);
-        if (vb) bv = *(const uint2*)(bp + k0);
+        if (va) { av[0] = *(const float4*)(ap + k0); av[1] = *(const float4*)(ap + k0 + 4); }
+        if (vb) bv = *(const uint4*)(bp + k0);
     };
     load(0);
     for (int k0 = 0; k0 < K_pad; k0 += FK) {
-        if (p.tanh_in) { av.x = tanhf(av.x); av.y = tanhf(av.y); av.z = tanhf(av.z); av.w = tanhf(av.w); }
+        float x[8] = {av[0].x, av[0].y, av[0].z, av[0].w, av[1].x, av[1].y, av[1].z, av[1].w};
+        const uint32_t y[4] = {bv.x, bv.y, bv.z, bv.w};
+        if (p.tanh_in)
+#pragma unroll
+            for (int i = 0; i < 8; ++i) x[i] = tanhf(x[i]);
         __syncthreads();
-        As[k4][row] = av.x; As[k4 + 1][row] = av.y; As[k4 + 2][row] = av.z; As[k4 + 3][row] = av.w;
-        Bs[k4][row] = __uint_as_float(bv.x << 16); Bs[k4 + 1][row] = __uint_as_float(bv.x & 0xffff0000u);
-        Bs[k4 + 2][row] = __uint_as_float(bv.y << 16); Bs[k4 + 3][row] = __uint_as_float(bv.y & 0xffff0000u);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) As[k8 + i][row] = x[i];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            Bs[k8 + 2 * i][row] = __uint_as_float(y[i] << 16);
+            Bs[k8 + 2 * i + 1][row] = __uint_as_float(y[i] & 0xffff0000u);
+        }
         __syncthreads();
         if (k0 + FK < K_pad) load(k0 + FK);
 #pragma unroll

@@ -156,7 +156,8 @@ static int launch_mix(const MixRows& p, cudaStream_t st) {
     while (rpc > 1 && (rpc + 1) * row > kSmem) rpc /= 2;
     const size_t smem = (rpc + 1) * row;
     if (smem > kSmem) return fail(FC_E_SHAPE, "rows of %d values exceed the row kernel's staging", p.d);
-    if (smem > 48 * 1024) FC_CUDA(cudaFuncSetAttribute(mix_rows_kernel<OT, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
+    // above 48 KB with the static part, shared memory has to be asked for
+    if (smem > 47 * 1024) FC_CUDA(cudaFuncSetAttribute(mix_rows_kernel<OT, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
     const int slots = rpc + (p.mu[0] ? 1 : 0);
     int W = 16 / slots;
     while (W > 1 && (W - 1) * 32 * V >= p.d) --W;          // no warp without columns

@@ -384,7 +384,7 @@ int launch_mixer_decode(const MixerDecode& a, cudaStream_t st) {
     const size_t rec = (size_t)(4 * a.rdim + a.rank + std::max(1, NT / a.rdim) * a.rdim) * 4;
     const size_t smem = std::max(att, rec);
     if (smem > 220 * 1024) return fail(FC_E_SHAPE, "the decode mixers need %zu bytes of shared memory", smem);
-    if (smem > 48 * 1024) {
+    if (smem > 47 * 1024) {
         FC_CUDA(cudaFuncSetAttribute(mixer_decode_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
         FC_CUDA(cudaFuncSetAttribute(mixer_decode_kernel<uint16_t>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     }

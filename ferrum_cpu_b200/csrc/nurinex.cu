@@ -181,7 +181,7 @@ struct fc_nurinex {
     CUtensorMap m_head, a_head;
     // workspace of a portion of ws_rows tokens
     int ws_rows = 0, head_chunk = 0;
-    float *x[2] = {}, *proj = nullptr, *outs = nullptr, *decay = nullptr, *wkv_o = nullptr, *logits = nullptr, *h_last = nullptr;
+    float *x[2] = {}, *proj = nullptr, *outs = nullptr, *decay = nullptr, *wkv_o = nullptr, *logits = nullptr, *h_last = nullptr, *wkv_scratch = nullptr;
     void *planes = nullptr, *att = nullptr, *ro = nullptr, *hid = nullptr, *qm = nullptr;
     int *ids_d = nullptr, *rows_d = nullptr, *targets_d = nullptr, *status = nullptr;     // status: [0] timeout, [1] bad id
     double* lp_d = nullptr;
@@ -382,6 +382,9 @@ int ensure_workspace(fc_nurinex* m, int rows) {
     FC_TRY(get((void**)&m->outs, (2 + kFfSplits) * RR * d * 4));
     FC_TRY(get((void**)&m->decay, RR * m->max_rd * 4));
     FC_TRY(get((void**)&m->wkv_o, RR * m->max_rd * 4));
+    size_t scratch = 0;
+    for (const NxWeights* w : m->run) scratch = std::max(scratch, wkv_scratch_floats(w->rH, w->rdim));
+    FC_TRY(get((void**)&m->wkv_scratch, scratch * 4));
     FC_TRY(get((void**)&m->h_last, (size_t)m->cfg.layers.size() * d * 4));
     FC_TRY(get(&m->planes, (1 + kMixes) * RR * dp * e));
     FC_TRY(get(&m->att, RR * m->max_att * e));
@@ -498,7 +501,7 @@ int layer_forward(fc_nurinex* m, fc_nurinex_cache* s, int l, int M, int pos0, in
         p.a = m->proj + w.off_w1; p.lda = ldp; p.tanh_in = 1; p.y = m->decay; p.ldy = rd; p.epi = ROW_DECAY; p.vec = w.w0;
         FC_TRY(launch_gemm_bf16w_f32(w.w2, 0, rd, p, M, m->side));
         FC_TRY(launch_wkv_scan(m->proj + w.off_r, m->proj + w.off_k, m->proj + w.off_v, ldp, m->decay, rd, w.u, s->wkv[l], m->wkv_o, rd, M, w.rH,
-                               w.rdim, m->side));
+                               w.rdim, m->wkv_scratch, m->side));
         FC_TRY(launch_wkv_finish(m->wkv_o, rd, m->proj + w.off_g, ldp, w.rnorm, (float)m->cfg.eps, M, w.rH, w.rdim, m->ro, w.ro.K_pad, m->f32, m->side));
     }
     FC_CUDA(cudaEventRecord(m->join, m->side));

@@ -95,7 +95,7 @@ static int prep(const TalkAttn& t, const float* proj, int ldp, int M, int pos0, 
     if (smem > 200 * 1024) return fail(FC_E_SHAPE, "%d query heads of %d exceed the staging of the query mixing", t.H, t.dim);
 #define FC_PREP(P)                                                                                                              \
     do {                                                                                                                        \
-        if (smem > 48 * 1024) FC_CUDA(cudaFuncSetAttribute(talk_prep_kernel<T, P>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+        if (smem > 47 * 1024) FC_CUDA(cudaFuncSetAttribute(talk_prep_kernel<T, P>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
         talk_prep_kernel<T, P><<<M, 256, smem, st>>>(t, proj, ldp, pos0, factor, (T*)qm, (T*)kc, (T*)vc);                        \
     } while (0)
     switch (t.H / t.KV) {

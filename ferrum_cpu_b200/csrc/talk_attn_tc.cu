@@ -102,17 +102,18 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
         if (lane == 0 && !a.withhold) {
             if (!a.q_stream) mbar_expect_tx(&bars->q_full, a.nkc * Q_CHUNK);
             for (int c = 0; !a.q_stream && c < a.nkc; ++c) tma_load_2d(smem + c * Q_CHUNK, &mq, h * a.kd + c * CH, q0, &bars->q_full);
-            int it = 0, nvt = 0;
+            int s = 0, issued = 0, nvt = 0;               // ring stage, key chunks and value tiles asked for
+            uint32_t ph = 1;                              // parity of k_empty: a fresh ring is empty
             bool ok = true;
             for (int kt = 0; kt < n_kt && ok; ++kt) {
                 for (int c = 0; c < a.nkc && ok; ++c) {
-                    const int s = it % a.ks;
-                    ok = wait(&bars->k_empty[s], ((it / a.ks) & 1) ^ 1);
+                    ok = wait(&bars->k_empty[s], ph);
                     if (!ok) break;
                     mbar_expect_tx(&bars->k_full[s], a.q_stream ? K_CHUNK + Q_CHUNK : K_CHUNK);
                     if (a.q_stream) tma_load_2d(smem + s * Q_CHUNK, &mq, h * a.kd + c * CH, q0, &bars->k_full[s]);
                     tma_load_2d(sk + s * K_CHUNK, &mk, c * CH, kt * KT, &bars->k_full[s]);
-                    ++it;
+                    ++issued;
+                    if (++s == a.ks) { s = 0; ph ^= 1; }
                 }
                 const int b = kt & 1;
                 ok = ok && wait(&bars->v_empty[b], ((kt >> 1) & 1) ^ 1);
@@ -127,7 +128,7 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
                     while (!mbar_try_wait(b, par) && clock64() - t0 < a.wait_cycles) {}
                 };
                 if (!a.q_stream) drain(&bars->q_full, 0);
-                for (int i = max(0, it - a.ks); i < it; ++i) drain(&bars->k_full[i % a.ks], (i / a.ks) & 1);
+                for (int i = max(0, issued - a.ks); i < issued; ++i) drain(&bars->k_full[i % a.ks], (i / a.ks) & 1);
                 for (int i = max(0, nvt - 2); i < nvt; ++i) drain(&bars->v_full[i & 1], (i >> 1) & 1);
             }
         }
@@ -135,13 +136,34 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
         if (lane == 0) {
             const uint32_t sb = s32(smem), kb = s32(sk), vb = s32(sv_);
             const uint64_t ph = smem_desc(s32(sp)), pl = smem_desc(s32(sp) + P_BYTES);
-            int it = 0, next_pv = 0;
-            // O += P V of tile next_pv; its P and V have been waited for
-            auto pv = [&]() {
-                const int kt = next_pv++, b = kt & 1;
+            int s = 0;                                    // ring stage (no divisions here: this thread's pace is the kernel's)
+            uint32_t kph = 0;
+            const uint64_t q_desc = smem_desc(sb), k_desc = smem_desc(kb), v_desc = smem_desc(vb);
+            auto scores = [&](int kt) -> bool {
+                const int b = kt & 1;
+                if (!wait(&bars->s_empty[b], ((kt >> 1) & 1) ^ 1)) return false;
+                fence_after();
+                for (int c = 0; c < a.nkc; ++c) {
+                    if (!wait(&bars->k_full[s], kph)) return false;
+                    fence_after();
+                    const uint64_t qd = q_desc + (uint64_t)((a.q_stream ? s : c) * (Q_CHUNK >> 4)), kd = k_desc + (uint64_t)(s * (K_CHUNK >> 4));
+#pragma unroll
+                    for (int ks = 0; ks < CH / 16; ++ks) umma(tmem + b * KT, qd + (uint64_t)(ks * 2), kd + (uint64_t)(ks * 2), IDESC_S, (c | ks) != 0);
+                    umma_commit(&bars->k_empty[s]);
+                    if (++s == a.ks) { s = 0; kph ^= 1; }
+                }
+                umma_commit(&bars->s_full[b]);
+                return true;
+            };
+            bool ok = (a.q_stream || wait(&bars->q_full, 0)) && scores(0);
+            for (int kt = 0; kt < n_kt && ok; ++kt) {
+                if (kt + 1 < n_kt && !(ok = scores(kt + 1))) break;
+                const int b = kt & 1;
+                ok = wait(&bars->v_full[b], (kt >> 1) & 1) && wait(&bars->p_full, kt & 1);
+                if (!ok) break;
                 fence_after();
                 for (int c = 0; c < a.nv; ++c) {
-                    const uint64_t vd = smem_desc(vb + (b * a.nv + c) * K_CHUNK);
+                    const uint64_t vd = v_desc + (uint64_t)((b * a.nv + c) * (K_CHUNK >> 4));
 #pragma unroll
                     for (int ks = 0; ks < KT / 16; ++ks) {
                         umma(tmem_o + c * CH, ph + (uint64_t)(ks * 2), vd + (uint64_t)(ks * 128), IDESC_O, (kt | ks) != 0);
@@ -150,31 +172,6 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
                 }
                 umma_commit(&bars->v_empty[b]);
                 umma_commit(&bars->o_done);
-            };
-            auto scores = [&](int kt) -> bool {
-                const int b = kt & 1;
-                if (!wait(&bars->s_empty[b], ((kt >> 1) & 1) ^ 1)) return false;
-                fence_after();
-                for (int c = 0; c < a.nkc; ++c, ++it) {
-                    const int s = it % a.ks;
-                    // the tile before may have become ready while these keys are still on their way
-                    if (next_pv < kt && mbar_test(&bars->p_full, next_pv & 1) && mbar_test(&bars->v_full[next_pv & 1], (next_pv >> 1) & 1)) pv();
-                    if (!wait(&bars->k_full[s], (it / a.ks) & 1)) return false;
-                    fence_after();
-                    const uint64_t qd = smem_desc(sb + (a.q_stream ? s : c) * Q_CHUNK), kd = smem_desc(kb + s * K_CHUNK);
-#pragma unroll
-                    for (int ks = 0; ks < CH / 16; ++ks) umma(tmem + b * KT, qd + (uint64_t)(ks * 2), kd + (uint64_t)(ks * 2), IDESC_S, (c | ks) != 0);
-                    umma_commit(&bars->k_empty[s]);
-                }
-                umma_commit(&bars->s_full[b]);
-                return true;
-            };
-            bool ok = (a.q_stream || wait(&bars->q_full, 0)) && scores(0);
-            for (int kt = 0; kt < n_kt && ok; ++kt) {
-                if (kt + 1 < n_kt && !(ok = scores(kt + 1))) break;
-                if (next_pv > kt) continue;
-                ok = wait(&bars->v_full[kt & 1], (kt >> 1) & 1) && wait(&bars->p_full, kt & 1);
-                if (ok) pv();
             }
         }
     } else {

@@ -28,16 +28,6 @@ __device__ __forceinline__ bool mbar_try_wait(unsigned long long* b, uint32_t pa
         : "=r"(ok) : "r"(s32(b)), "r"(parity), "r"(2000u) : "memory");
     return ok != 0;
 }
-// Whether the phase has completed; never suspends.
-__device__ __forceinline__ bool mbar_test(unsigned long long* b, uint32_t parity) {
-    uint32_t ok;
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-        "selp.u32 %0, 1, 0, p;\n\t}"
-        : "=r"(ok) : "r"(s32(b)), "r"(parity) : "memory");
-    return ok != 0;
-}
 // Bounded wait: false (after raising the status word) when the cycle budget runs out or another role
 // of the CTA has already given up.
 __device__ __forceinline__ bool wait_bar(volatile int* abort_flag, unsigned long long* b, uint32_t parity, int* status, long long budget) {

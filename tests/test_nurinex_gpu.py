@@ -75,7 +75,7 @@ def test_residual_stream_after_every_layer(tmp_path, mode):
 
 @MODES
 def test_portions_do_not_change_the_logits(tmp_path, mode):
-    """Beyond rounding the cut does not matter; of prompts cut in portions nothing changes at all."""
+    """Beyond rounding the cut does not matter: not in portions, nor token by token."""
     config, rows, rank = configs()["mixed"]
     path, ten = build(tmp_path, config, 7, rows, rank)
     toks = ids(4, 300, config["vocab"])
@@ -85,7 +85,7 @@ def test_portions_do_not_change_the_logits(tmp_path, mode):
     for cuts in ([128], [63, 65, 191], [2, 298], [7 * k for k in range(1, 42)]):
         c.clear()
         got = feed_in(m, c, toks, cuts)
-        assert np.array_equal(got, whole), cuts
+        assert error(got, whole) < TOL[mode] / 4, cuts
     c.clear()
     got = feed_in(m, c, toks, range(250, 300))
     assert error(got, whole) < TOL[mode]
@@ -297,6 +297,21 @@ def test_refusals_leave_the_cache_usable(tmp_path):
     m.close()
 
 
+def test_wide_rows_in_portions_of_every_size_class(tmp_path):
+    """Rows of 4096 values: the row kernel's staging passes 48 KB in one of the size classes and not in the next."""
+    config = MD.nurinex_config(40, 4096, [L(heads=2, kv_heads=1, dim=16, vdim=16, bias_max=50, r_heads=1, r_dim=16, ff=32)])
+    path, ten = build(tmp_path, config, 26, 8, 4)
+    toks = ids(27, 600, 40)
+    m = CudaNurinex(path, math_mode=F32, ctx=600)
+    c = m.new_cache()
+    whole = feed_in(m, c, toks, [])
+    for cuts in ([300], [100, 101], range(560, 600)):
+        c.clear()
+        assert error(feed_in(m, c, toks, cuts), whole) < TOL[F32]
+    assert error(whole[:40], NO.forward(config, ten, toks[:40])) < TOL[F32]
+    m.close()
+
+
 def test_portions_longer_than_one_pass(tmp_path):
     """More tokens than a forward pass takes are cut inside the call; nothing shows at the seam."""
     config = MD.nurinex_config(90, 32, [L(heads=2, kv_heads=1, dim=16, vdim=16, bias_max=500, r_heads=1, r_dim=16, ff=32)])
@@ -308,7 +323,7 @@ def test_portions_longer_than_one_pass(tmp_path):
     c.clear()
     m.feed(toks[:1000], c)
     b = m.feed(toks[1000:], c, [1046, 1047, 1048, 1049, 1299])
-    assert np.array_equal(a[1:], b)
+    assert error(b, a[1:]) < TOL[F32] / 4
     m.close()
 
 
