@@ -136,12 +136,13 @@ template <class T>
 __device__ __forceinline__ void scores_of(const T* kr, const float* q, int qst, int dim, bool vec, float (&s)[PER]) {
     constexpr int V = kVec<T>;
     if (vec) {
-        for (int e0 = 0; e0 < dim; e0 += 4 * V) {        // four loads in flight
-            uint4 w[4];
+        constexpr int F = 8;                             // loads in flight
+        for (int e0 = 0; e0 < dim; e0 += F * V) {
+            uint4 w[F];
 #pragma unroll
-            for (int x = 0; x < 4; ++x) w[x] = e0 + x * V < dim ? *(const uint4*)(kr + e0 + x * V) : make_uint4(0, 0, 0, 0);
+            for (int x = 0; x < F; ++x) w[x] = e0 + x * V < dim ? *(const uint4*)(kr + e0 + x * V) : make_uint4(0, 0, 0, 0);
 #pragma unroll
-            for (int x = 0; x < 4; ++x)
+            for (int x = 0; x < F; ++x)
                 if (e0 + x * V < dim) {
                     float kv[V];
                     unpack<T>(w[x], kv);
@@ -192,6 +193,14 @@ __device__ void attention(const MixerDecode& a, float* sm) {
     const int mst = Hp + 4;
     float* acc = mix + KT * mst;                 // [2][H][vd]: halves of the keys
     float* ml = acc + 2 * H * vd;                // [H][3]: max, sum, correction
+    float* bsm = ml + 3 * H;                     // [H][RST]: bias of the tile's distances
+    auto load_bias = [&](int k0) {
+        for (int i = tid; i < H * KT; i += NT) {
+            const int h = i / KT, j = i - h * KT;
+            bsm[h * RST + j] = __ldg(t.bias + (size_t)h * (t.far + 1) + min(max(pos - (k0 + j), 0), t.far));
+        }
+    };
+    if (sp < splits) load_bias(k_begin);
     for (int i = tid; i < H * H; i += NT) { const int h = i / H, g = i - h * H; talk[g * Hp + h] = t.talk[i]; }
     for (int i = tid; i < 2 * H * vd; i += NT) acc[i] = 0.0f;
     for (int h = tid; h < H; h += NT) { ml[3 * h] = -INFINITY; ml[3 * h + 1] = 0.0f; ml[3 * h + 2] = 0.0f; }
@@ -220,6 +229,7 @@ __device__ void attention(const MixerDecode& a, float* sm) {
     const bool vec = dim % kVec<T> == 0;         // every key part starts on 16 bytes then
     for (int k0 = k_begin; k0 < k_end; k0 += KT) {
         const int nk = min(KT, k_end - k0);
+        if (k0 > k_begin) load_bias(k0);
         for (int i = tid; i < nk * t.KV; i += NT) {
             const int j = i / t.KV, c = i - j * t.KV;
             const T* kr = kc + (size_t)(k0 + j) * t.kd + c * dim;
@@ -246,12 +256,11 @@ __device__ void attention(const MixerDecode& a, float* sm) {
             for (int z = 0; z < 4; ++z) {
                 const int h = h0 + z;
                 if (h >= H) break;
-                const float* bias = t.bias + (size_t)h * (t.far + 1);
                 float b[2];
 #pragma unroll
                 for (int y = 0; y < 2; ++y) {
                     const int j = lane + 32 * y;
-                    b[y] = j < nk ? s[z][y] + bias[min(pos - (k0 + j), t.far)] : -INFINITY;
+                    b[y] = j < nk ? s[z][y] + bsm[h * RST + j] : -INFINITY;
                 }
                 float mx = fmaxf(b[0], b[1]);
 #pragma unroll
@@ -279,10 +288,10 @@ __device__ void attention(const MixerDecode& a, float* sm) {
             for (int g0 = 0; g0 < per; g0 += PER) {
                 float s[PER][2] = {};
                 const float* mp = mix + c * per + g0;
-                for (int j0 = kh ? half : 0; j0 < j_end; j0 += 8) {
-                    float vv[8][2];
+                for (int j0 = kh ? half : 0; j0 < j_end; j0 += 16) {
+                    float vv[16][2];
 #pragma unroll
-                    for (int x = 0; x < 8; ++x) {
+                    for (int x = 0; x < 16; ++x) {
                         vv[x][0] = vv[x][1] = 0.0f;
                         if (j0 + x < j_end) {
                             const T* p = v + (size_t)(j0 + x) * vst;
@@ -296,7 +305,7 @@ __device__ void attention(const MixerDecode& a, float* sm) {
                         }
                     }
 #pragma unroll
-                    for (int x = 0; x < 8; ++x) {
+                    for (int x = 0; x < 16; ++x) {
                         const float* mr = mp + min(j0 + x, KT - 1) * mst;
 #pragma unroll
                         for (int y = 0; y < PER; ++y) {
@@ -380,7 +389,7 @@ int launch_mixer_decode(const MixerDecode& a, cudaStream_t st) {
     const TalkAttn& t = a.t;
     const int qd = (t.dim + 3) & ~3, Hp = (t.H + 3) & ~3;
     if (a.max_splits > KT) return fail(FC_E_SHAPE, "%d attention splits (at most %d)", a.max_splits, KT);
-    const size_t att = (size_t)(t.KV * (t.H / t.KV * qd + 4) + PER * qd + t.H * Hp + (t.H + PER) * RST + KT * (Hp + 4) + 2 * t.H * t.vdim + 3 * t.H) * 4;
+    const size_t att = (size_t)(t.KV * (t.H / t.KV * qd + 4) + PER * qd + t.H * Hp + (t.H + PER) * RST + KT * (Hp + 4) + 2 * t.H * t.vdim + 3 * t.H + t.H * RST) * 4;
     const size_t rec = (size_t)(4 * a.rdim + a.rank + std::max(1, NT / a.rdim) * a.rdim) * 4;
     const size_t smem = std::max(att, rec);
     if (smem > 220 * 1024) return fail(FC_E_SHAPE, "the decode mixers need %zu bytes of shared memory", smem);
