@@ -18,6 +18,7 @@ pub const FC_E_CANCELLED: c_int = -6;
 pub const FC_E_ARG: c_int = -7;
 pub const FC_MATH_FP32: c_int = 0;
 pub const FC_MATH_BF16X3: c_int = 1;
+pub const FC_MATH_BF16: c_int = 2;
 pub const FC_DECODE_PERSISTENT: c_int = 0;
 pub const FC_DECODE_PER_KERNEL: c_int = 1;
 pub const FC_ROPE_NORM: c_int = 0;
