@@ -298,7 +298,7 @@ def run_nurinex(a, names, prompts=(256, 1024, 2048), with_llama=True):
     from ferrum_cpu_b200 import model_dir, synth
     from ferrum_cpu_b200.engine import sampling
     from ferrum_cpu_b200.llama import CudaLlama
-    from ferrum_cpu_b200.nurinex import CudaNurinex
+    from ferrum_cpu_b200.decoder import CudaNurinex
     hbm, tf, kind = peaks()
     greedy = sampling(temperature=0.0)
     rows = []
@@ -436,7 +436,7 @@ def run_case(a):
         import tempfile
         from ferrum_cpu_b200 import model_dir
         from ferrum_cpu_b200.engine import sampling
-        from ferrum_cpu_b200.nurinex import CudaNurinex
+        from ferrum_cpu_b200.decoder import CudaNurinex
         name = a.model if a.model in model_dir.NURINEX_SHAPES else "nurinex-1b"
         if a.layers:
             shape = list(model_dir.NURINEX_SHAPES[name])

@@ -63,7 +63,7 @@ class FcLayerStats(C.Structure):
                 ("n_elements", C.c_int64)]
 
 
-class FcNurinexInfo(C.Structure):
+class FcDecoderInfo(C.Structure):
     _fields_ = [("vocab", C.c_int32), ("width", C.c_int32), ("n_layers", C.c_int32), ("n_own_layers", C.c_int32), ("ctx", C.c_int32),
                 ("pad", C.c_int32), ("weight_bytes", C.c_int64)]
 
@@ -145,21 +145,21 @@ SIGNATURES = {
                                     C.POINTER(C.c_uint64), C.c_void_p, C.c_void_p, C.POINTER(C.c_int)]),
     "fc_llama_last_decode_ms": (C.c_float, [C.c_void_p]),
     "fc_model_dir_architecture": (C.c_int, [C.c_char_p, C.c_char_p, C.c_int]),
-    "fc_nurinex_probe": (C.c_int, [C.c_char_p, C.POINTER(FcNurinexInfo)]),
-    "fc_nurinex_load": (C.c_int, [C.c_char_p, C.c_int, C.c_int, C.c_int, C.POINTER(C.c_void_p)]),
-    "fc_nurinex_free": (None, [C.c_void_p]),
-    "fc_nurinex_get_info": (C.c_int, [C.c_void_p, C.POINTER(FcNurinexInfo)]),
-    "fc_nurinex_cache_create": (C.c_int, [C.c_void_p, C.POINTER(C.c_void_p)]),
-    "fc_nurinex_cache_free": (None, [C.c_void_p]),
-    "fc_nurinex_cache_clear": (C.c_int, [C.c_void_p]),
-    "fc_nurinex_cache_pos": (C.c_int, [C.c_void_p]),
-    "fc_nurinex_feed": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_void_p, C.c_int, C.c_void_p]),
-    "fc_nurinex_feed_layers": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_void_p]),
-    "fc_nurinex_score": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.POINTER(FcScore), C.c_void_p, C.c_void_p]),
-    "fc_nurinex_generate": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.POINTER(FcSampling), C.c_void_p, C.c_int,
+    "fc_decoder_probe": (C.c_int, [C.c_char_p, C.POINTER(FcDecoderInfo)]),
+    "fc_decoder_load": (C.c_int, [C.c_char_p, C.c_int, C.c_int, C.c_int, C.POINTER(C.c_void_p)]),
+    "fc_decoder_free": (None, [C.c_void_p]),
+    "fc_decoder_get_info": (C.c_int, [C.c_void_p, C.POINTER(FcDecoderInfo)]),
+    "fc_decoder_cache_create": (C.c_int, [C.c_void_p, C.POINTER(C.c_void_p)]),
+    "fc_decoder_cache_free": (None, [C.c_void_p]),
+    "fc_decoder_cache_clear": (C.c_int, [C.c_void_p]),
+    "fc_decoder_cache_pos": (C.c_int, [C.c_void_p]),
+    "fc_decoder_feed": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_void_p, C.c_int, C.c_void_p]),
+    "fc_decoder_feed_layers": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_void_p]),
+    "fc_decoder_score": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.POINTER(FcScore), C.c_void_p, C.c_void_p]),
+    "fc_decoder_generate": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.POINTER(FcSampling), C.c_void_p, C.c_int,
                                       C.POINTER(C.c_uint64), C.c_void_p, C.c_void_p, C.POINTER(C.c_int)]),
-    "fc_nurinex_last_forward_ms": (C.c_float, [C.c_void_p]),
-    "fc_nurinex_last_decode_ms": (C.c_float, [C.c_void_p]),
+    "fc_decoder_last_forward_ms": (C.c_float, [C.c_void_p]),
+    "fc_decoder_last_decode_ms": (C.c_float, [C.c_void_p]),
     "fc_rowq_packed_len": (C.c_size_t, [C.c_int, C.c_int, C.c_int]),
     "fc_rowq_from_f32": (C.c_int, [C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p, C.c_void_p]),
     "fc_rowq_to_f32": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p]),

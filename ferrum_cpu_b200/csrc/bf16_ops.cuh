@@ -3,6 +3,7 @@
 // nothing here belongs to one model.
 #pragma once
 #include <cuda.h>
+#include <cuda_bf16.h>
 
 #include "fc_common.cuh"
 
@@ -16,11 +17,13 @@ struct BMat {
 inline int pad_to(int v, int m) { return (v + m - 1) / m * m; }
 
 // What happens to a product before it is stored. XIELU: z > 0: c0 z^2 + z / 2, else c1 (e^z - 1 - z) + z / 2.
-// DECAY: exp(-exp(v + vec[n])).
-enum RowEpi : int { ROW_NONE = 0, ROW_XIELU = 1, ROW_DECAY = 2 };
+// DECAY: exp(-exp(v + vec[n])). GELU: the exact form, z / 2 (1 + erf(z / sqrt 2)).
+enum RowEpi : int { ROW_NONE = 0, ROW_XIELU = 1, ROW_DECAY = 2, ROW_GELU = 3 };
 __device__ __forceinline__ float xielu_f(float z, float c0, float c1) {
     return z > 0.0f ? fmaf(c0 * z, z, 0.5f * z) : fmaf(c1, expm1f(z) - z, 0.5f * z);
 }
+
+__device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
 
 // ---- gemm_bf16.cu: several products in one launch ---------------------------------------------------
 // Segment: columns [0, n) of Y = A W^T with A rows taken from a plane of one of the operand maps and W rows
@@ -35,15 +38,26 @@ struct GemmSeg {
 };
 constexpr int kGemmSegs = 16;
 struct GemmMaps { CUtensorMap a[3], b[3]; };
+// Row tiles of a product with runs of rows: {first row, rows, index of the run's weights, 0}, and how many there are.
+struct Ragged {
+    const int4* table;
+    const int* n;
+    int b_step;       // weight rows from one index to the next
+};
 struct GemmGroup {
     GemmSeg seg[kGemmSegs];
     int n_seg, M, n_tiles;
     int* status;
     long long wait_cycles;
     int withhold;
+    Ragged ragged;
 };
 constexpr int kGemmBoxRows = 128;     // rows of every box of the operand and weight maps
 int launch_gemm_bf16_group(const GemmMaps& maps, GemmGroup g, int M, int* status, cudaStream_t st);
+// One product whose rows fall into runs, each with weights of its own (rows of one expert after the other): the segment's
+// b_row0 and b_step give the first weight row of a run's index. Tiles are counted on the device; at most max_tiles entries.
+constexpr int kRaggedRows = 256, kRaggedRowsF32 = 64;   // most rows of a table entry
+int launch_gemm_bf16_ragged(const GemmMaps& maps, const GemmSeg& seg, const Ragged& r, int max_entries, int* status, cudaStream_t st);
 // One product in true f32 on CUDA cores: Y[M][n] = f(A)[M][K] W^T, A f32 rows lda apart (K = w.K_pad columns are
 // read), W rows row0.. of the matrix; tanh_in applies tanh to A on the way in. y or yb.
 struct GemmF32 {
@@ -52,6 +66,8 @@ struct GemmF32 {
     int epi; float c0, c1; const float* vec;
 };
 int launch_gemm_bf16w_f32(const BMat& w, int row0, int n, const GemmF32& p, int M, cudaStream_t st);
+// The same over runs of rows (table entries of at most kRaggedRowsF32 rows): weight rows index * b_step ..
+int launch_gemm_bf16w_f32_ragged(const BMat& w, int n, const GemmF32& p, const Ragged& r, int max_entries, cudaStream_t st);
 
 // ---- rows of side-by-side layers (mix_rows.cu) ------------------------------------------------------
 // Residual update of the layer before (x + (half the sum of two normed outputs + feed-forward partials)), the norm of
@@ -83,7 +99,63 @@ struct MixRows {
 };
 int launch_mix_rows(const MixRows& p, bool f32_planes, cudaStream_t st);
 
-// ---- talk_attn.cu / talk_attn_tc.cu: attention with mixed heads ------------------------------------
+// ---- rows of layers that norm what a sublayer adds (post_norm_rows.cu) --------------------------------------
+// x' = x + rms(y) w, y = sum of parts, part s of a row being weight[row * n_parts + s] y[index[row * n_parts + s]] (index null:
+// row s * part_rows + row of y; weight null: 1). Without y: x' = rms(embed[id]) w.
+struct PostNorm {
+    const float* y = nullptr;
+    int n_parts = 0, part_rows = 0;
+    const int* index = nullptr;
+    const float* weight = nullptr;
+    const float* norm_w = nullptr;
+};
+// Value c of the sum of a row's parts.
+__device__ __forceinline__ float post_norm_sum(const PostNorm& p, size_t row, int c, int d) {
+    float y = 0.0f;
+    for (int s = 0; s < p.n_parts; ++s) {
+        const size_t at = row * p.n_parts + s, r = p.index ? (size_t)p.index[at] : (size_t)s * p.part_rows + row;
+        const float v = p.y[r * d + c];
+        y = p.weight ? fmaf(p.weight[at], v, y) : y + v;
+    }
+    return y;
+}
+struct PostNormRows {
+    PostNorm add;
+    EmbedSrc embed; const int* ids;    // used when add.y is null and ids is set
+    float* x;                          // [M][d] residual, updated in place (rows row_idx[r] of it when that is set)
+    const int* row_idx;
+    const float* out_norm_w;           // not null: the plane receives rms(x') out_norm_w, and x stays as it is when add.y is null
+    float eps;
+    int M, d, ld;
+    void* plane;                       // [M][ld], bf16 or f32: x', or its norm
+    int* error_flag;
+};
+int launch_post_norm_rows(const PostNormRows& p, bool f32_plane, cudaStream_t st);
+
+// ---- flash_tc.cu / flash_f32.cu: attention of a portion's rows over cached keys ---------------------------
+// score[h](i, j) = q_h(i) . k_h(j) (+ bias[h][min(i - j, far)]) for 0 <= i - j < window; softmax, with one extra exp(sink) in
+// the denominator when there is a sink. A key row is a part of the head's own (head h reads key/value head h / (H / KV);
+// head_stride 0: all read the same) and, when k1.p is set, a part all heads share. Columns col + head * head_stride +
+// 0 .. width - 1 of rows ld elements apart; row r holds position pos0 + r. Widths, strides and first columns are multiples of 16.
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr int kNoWindow = 1 << 30;
+struct FlashPart {
+    const void* p = nullptr;
+    int rows = 0, ld = 0, col = 0, head_stride = 0, width = 0, pos0 = 0;
+};
+struct Flash {
+    int H = 0, KV = 0, vdim = 0;
+    FlashPart k0, k1, v;
+    int window = kNoWindow;
+    const float* bias = nullptr; int far = 0;       // [H][far + 1]
+    bool has_sink = false; const float* sink = nullptr;   // [H]; null: a score of 0 for every head
+};
+// Rows at positions pos0 .. pos0 + M - 1. q [M][H * (k0.width + k1.width)]; out rows ldo apart, head by head; value heads of at
+// most 256. tcgen05 form: bf16 everywhere, queries times log2(e).
+int launch_flash_tc(const Flash& f, const void* q, int M, int pos0, void* out, int ldo, int* status, cudaStream_t st);
+int launch_flash_f32(const Flash& f, const float* q, int M, int pos0, float* out, int ldo, cudaStream_t st);
+
+// ---- talk_attn.cu: attention with mixed heads --------------------------------------------------------
 // score[h](i, j) = sum_g talk[h][g] (scale temp(i) q_g(i) . k_kv(g)(j) + rel[bucket(i - j)][g]), softmax with one extra
 // exp(sink[h]) in the denominator, values divided by their root mean square. Mixing is linear, so it is applied to the
 // queries: with q'_h = the concatenation over key/value heads c of sum_{g in c} talk[h][g] q_g, the mixed score is
@@ -103,14 +175,7 @@ struct TalkAttn {
 // proj rows: q | k | v. qm [M][H * kd], bf16 or f32; caches in the same type.
 int launch_talk_prep(const TalkAttn& t, const float* proj, int ldp, int M, int pos0, float factor, void* qm, void* kc, void* vc, bool f32,
                      cudaStream_t st);
-// Rows of a portion against an f32 cache (positions 0 .. pos0 + i) on CUDA cores; out rows ldo apart. Queries prepared
-// with factor 1; value heads of at most 256.
-int launch_talk_prefill_f32(const TalkAttn& t, const float* qm, const float* kc, const float* vc, int M, int pos0, float* out, int ldo,
-                            cudaStream_t st);
-// The same on tcgen05 with bf16 queries, cache and output; queries prepared with factor log2(e).
-int launch_talk_prefill_tc(const TalkAttn& t, const void* qm, const void* kc, const void* vc, int M, int pos0, int ctx, void* out, int ldo,
-                           int* status, cudaStream_t st);
-constexpr float kLog2e = 1.4426950408889634f;
+Flash talk_flash(const TalkAttn& t, const void* kc, const void* vc, int ctx);
 
 // ---- wkv.cu: linear-attention state with per-channel decay and a bonus for the current token --------
 // o_t = (S + diag(u) k_t v_t^T)^T r_t, S <- diag(w_t) S + k_t v_t^T; state [H][dim][dim] f32 in and out. scratch:
@@ -128,18 +193,22 @@ int launch_wkv_finish(const float* o, int ldo, const float* gate, int ldg, const
 // prologue, or x[src]).
 struct GemvSeg {
     const uint16_t* w;    // first row; rows ldw apart, K_pad weights of each (a multiple of 64), K inputs
+    const int* index;     // not null: the rows begin *index * w_step weights further on (an expert chosen on the device)
+    size_t w_step;
     int n, ldw, K_pad, src, K;
     float* y;
     int epi;
     float c0, c1;
     long long cost0;      // filled by the launcher
 };
-constexpr int kGemvSegs = 16;
+constexpr int kGemvSegs = 32, kGemvInputs = 32;
 struct GemvGroup {
     GemvSeg seg[kGemvSegs];
     int n_seg;
-    const float* x[8];                 // plain inputs (mode 0)
-    int mode;                          // 0: plain inputs; 1: residual + norm + mixes of the row; 2: residual + norm
+    const float* x[kGemvInputs];       // plain inputs (mode 0)
+    int mode;                          // 0: plain inputs; 1: residual + norm + mixes of the row; 2: residual + norm;
+                                       // 3: residual of PostNorm; 4: the same and a norm (norm_w)
+    PostNorm post;                     // modes 3 and 4 (x_in, x_out, queue and embed as in the others)
     EmbedSrc embed; const int* queue; int ctx;
     SideOutputs prev;
     const float* x_in; float* x_out;
@@ -151,6 +220,99 @@ struct GemvGroup {
     long long total_cost;
 };
 int launch_gemv_bf16_group(GemvGroup g, cudaStream_t st);
+
+// ---- rot_attn.cu: what attention with rotated positions needs around the softmax ----------------------------
+// Pair i of `dims` elements turns by position * base^(-2i/dims); freq[i] is that power in double. neighbours: elements 2i and
+// 2i + 1 form a pair, else i and i + dims / 2.
+struct Rot {
+    int dims = 0;
+    bool neighbours = false;
+    const double* freq = nullptr;
+};
+// Grouped-query attention: q and k normed over their whole projection (q_norm / k_norm null: not), rotated on the first
+// rot.dims elements of every head; scores times scale. Cached rows: KV heads of kp (keys) and vp (values) elements.
+struct RotAttn {
+    int H = 0, KV = 0, dim = 0, vdim = 0, kp = 0, vp = 0;
+    float scale = 1.0f, eps = 0.0f;
+    Rot rot;
+    const float *q_norm = nullptr, *k_norm = nullptr;
+    int window = kNoWindow;
+    bool has_sink = false;             // one more exp(0) in the denominator
+    bool own_kv = true;                // false: the keys and values of another layer's cache
+};
+// Rows at pos0 ..: q [M][H * kp] (times scale and factor) and, with own_kv, cache rows. proj rows: q | k | v.
+int launch_rot_prep(const RotAttn& t, const float* proj, int ldp, int M, int pos0, float factor, void* q, void* kc, void* vc, bool f32, cudaStream_t st);
+Flash rot_flash(const RotAttn& t, const void* kc, const void* vc, int ctx);
+
+// Latent attention: a cached row is one normed latent of `rank` values, then one rotated key part of `rot.dims`, both shared by
+// all heads; a head's own key part and its values are products of the latent. Row: [lat | rot_p], lat = rank up to 64s.
+struct LatentAttn {
+    int H = 0, dim = 0, vdim = 0, rank = 0;
+    int dp = 0, vp = 0, lat = 0, rot_p = 0;     // elements of a head's expanded key / value row, of either part of a cached row
+    float scale = 1.0f, eps = 0.0f;
+    Rot rot;
+    const float* c_norm = nullptr;
+    int window = kNoWindow;
+    const uint16_t *uk = nullptr, *uv = nullptr;     // [H * dp][lat], [H * vp][lat]: rows of a head padded with zeros
+    int row() const { return lat + rot_p; }
+};
+// Rows at pos0 ..: q [M][H * (dp + rot_p)] (times scale and factor), cache rows. proj rows: q | latent | shared key part.
+int launch_latent_prep(const LatentAttn& t, const float* proj, int ldp, int M, int pos0, float factor, void* q, void* cache, bool f32,
+                       cudaStream_t st);
+// Keys and values of positions base .. as expanded by products of the cached latents (rows of H * dp and H * vp).
+Flash latent_flash(const LatentAttn& t, const void* k, const void* v, int rows, int base, const void* cache, int ctx);
+
+// One token (attn_decode.cu). Latent: q' = [W_uk^T q | rotated part] per head, f32 [H][lat + rot_p], and the token's cache row.
+int launch_latent_absorb(const LatentAttn& t, const float* proj, float* q, void* cache, bool f32, const StepState* state, cudaStream_t st);
+// Splits of the visible cached rows against all heads. Grouped-query: prepares q itself, writes the token's cache row (own_kv),
+// and the last split of a block of heads merges into out [H * vdim].
+struct AttnDecode {
+    int H = 0, KV = 0, kw = 0, vw = 0;               // values of a key / value row of one head (kw a multiple of 8)
+    int k_ld = 0, k_head = 0, v_ld = 0, v_head = 0;  // row stride and head stride of the caches
+    void *kc = nullptr, *vc = nullptr;               // vc null: the values are the first vw of a key row
+    bool f32 = false;
+    int window = kNoWindow;
+    bool has_sink = false;
+    RotAttn prep;                                    // H 0: q is ready (f32 [H][kw], scaled), the cache row written
+    const float* q = nullptr;                        // the projection row q | k | v, or the ready queries
+    float *part = nullptr, *part_ml = nullptr;       // [splits][H][vw up to 4s], [splits][H][2]
+    int max_splits = 1;
+    unsigned int* counter = nullptr;                 // one a block of heads; null: the splits stay as they are
+    float* out = nullptr;
+    const StepState* state = nullptr;
+};
+constexpr int kMaxSplitsRow = 64;                     // most splits of a token
+int launch_attn_decode_rows(const AttnDecode& a, cudaStream_t st);
+int attn_decode_blocks(const AttnDecode& a);         // blocks of heads: counters needed
+// Merges the splits of latent decoding and expands the values: out [H * vdim].
+int launch_latent_expand(const LatentAttn& t, const AttnDecode& a, float* out, cudaStream_t st);
+
+// ---- experts.cu: routed feed-forwards -----------------------------------------------------------------
+struct Router {
+    int experts = 0, top = 0, groups = 1, keep = 1;
+    const uint16_t* w = nullptr; int ld = 0;         // [experts][ld]
+};
+// Routes M rows of x (f32, d apart; the same as operand rows in `plane`, ld apart): chosen expert and weight (softmax over all
+// experts, not renormalised) of every slot, the places of the slots' rows once they are grouped by expert, those rows (bf16 or
+// f32, ld apart) and the row tiles of the products. counts starts as zeros.
+struct RouteRows {
+    Router r;
+    const float* x; int M, d;
+    int *expert, *index, *counts; float* weight;     // [M][top], [M][top], [experts], [M][top]
+    void* rows; int ld;
+    int4* table; int* n_table; int tile_rows;
+};
+int max_row_tiles(const Router& r, int M, int tile_rows);
+int launch_route_rows(const RouteRows& p, const void* plane, bool f32_rows, cudaStream_t st);
+// One token: the residual before it (PostNorm), logits, choice. expert / weight [top]; scratch: logits [experts] and a counter.
+struct RouteStep {
+    Router r;
+    PostNorm post; const float* x_in; float* x_out; float eps; int d;
+    float* z; unsigned int* counter;
+    int* expert; float* weight;
+    const StepState* state;
+};
+int launch_route_step(const RouteStep& p, cudaStream_t st);
 
 // mixer_decode.cu: attention splits and recurrence heads of one token in one launch.
 struct MixerDecode {

@@ -1,0 +1,273 @@
+// Routing of feed-forwards that are cut into experts: which experts a token uses and with what weight, and the rows of a
+// portion regrouped so that every expert's products read consecutive rows.
+//
+//   route_rows_kernel    8 tokens a CTA: logits in f32 (rows in shared memory piece by piece, a warp holds four experts), softmax
+//                        over all experts, the best groups (a group's score is its largest), the best experts in them; a slot's
+//                        place within its expert from an atomic counter (the order of an expert's rows does not matter)
+//   gather_rows_kernel   a CTA per token: places become rows (prefix sums of the counts), its operand row copied to each; the
+//                        first CTA writes the table of row tiles
+//   route_step_kernel    one token: residual and norm ahead of it, a warp per expert, the last CTA to finish chooses
+// The products themselves: launch_gemm_bf16_ragged (portions), launch_gemv_bf16_group with indexed segments (one token).
+//
+// Bound: fp32 FMA (2 experts d FLOP per token) and L2; the gather HBM / L2.
+#include <algorithm>
+
+#include "pdl.cuh"
+#include "rot_rows.cuh"
+
+namespace fc {
+
+namespace {
+constexpr int NT = 256, TOK = 8, EPW = 4, KC = 512;      // tokens a CTA, experts a warp holds at once, columns staged at once
+constexpr int kMaxExperts = 1024, kMaxGroups = 256;
+
+// Place of column k in shared memory: within 256 values, lane l's eight are two float4 at 4 l and 128 + 4 l.
+__device__ __forceinline__ int spot(int k) {
+    const int e = k & 7;
+    return (k & ~255) + ((k >> 3) & 31) * 4 + (e & 3) + (e & 4) * 32;
+}
+__device__ __forceinline__ void dot8(const uint4& w, const float4& u, const float4& v, float& s) {
+    s = fmaf(__uint_as_float(w.x << 16), u.x, s); s = fmaf(__uint_as_float(w.x & 0xffff0000u), u.y, s);
+    s = fmaf(__uint_as_float(w.y << 16), u.z, s); s = fmaf(__uint_as_float(w.y & 0xffff0000u), u.w, s);
+    s = fmaf(__uint_as_float(w.z << 16), v.x, s); s = fmaf(__uint_as_float(w.z & 0xffff0000u), v.y, s);
+    s = fmaf(__uint_as_float(w.w << 16), v.z, s); s = fmaf(__uint_as_float(w.w & 0xffff0000u), v.w, s);
+}
+// The place and value of the largest entry (the first of equals), in every lane. n may exceed what a lane sees.
+__device__ __forceinline__ int warp_argmax(const float* z, int n, float* best) {
+    const int lane = threadIdx.x & 31;
+    float b = -INFINITY;
+    int at = 1 << 30;
+    for (int i = lane; i < n; i += 32)
+        if (z[i] > b) { b = z[i]; at = i; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, b, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+        if (ob > b || (ob == b && oa < at)) { b = ob; at = oa; }
+    }
+    *best = b;
+    return at;
+}
+// One warp chooses from logits z (overwritten) of a token; gs: room for the groups' scores. emit(slot, expert, weight) runs in
+// lane 0. Softmax keeps the logits' order, so they are compared in its place.
+template <class F>
+__device__ void choose(float* z, float* gs, const Router& r, F emit) {
+    const int lane = threadIdx.x & 31, E = r.experts;
+    float top;
+    warp_argmax(z, E, &top);
+    float sum = 0.0f;
+    for (int i = lane; i < E; i += 32) sum += expf(z[i] - top);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    if (r.keep < r.groups) {
+        const int size = E / r.groups;
+        for (int g = lane; g < r.groups; g += 32) {
+            float m = -INFINITY;
+            for (int i = 0; i < size; ++i) m = fmaxf(m, z[g * size + i]);
+            gs[g] = m;
+        }
+        __syncwarp();
+        for (int k = 0; k < r.keep; ++k) {
+            float v;
+            const int g = warp_argmax(gs, r.groups, &v);
+            __syncwarp();
+            if (lane == 0 && g < r.groups) gs[g] = -INFINITY;        // taken
+            __syncwarp();
+        }
+        for (int i = lane; i < E; i += 32)
+            if (gs[i / size] != -INFINITY) z[i] = -INFINITY;         // not among the best
+        __syncwarp();
+    }
+    for (int k = 0; k < r.top; ++k) {
+        float v;
+        int e = warp_argmax(z, E, &v);
+        if (e >= E) e = 0;                                           // only where logits are not numbers
+        __syncwarp();
+        if (lane == 0) { z[e] = -INFINITY; emit(k, e, expf(v - top) / sum); }
+        __syncwarp();
+    }
+}
+}  // namespace
+
+__global__ void __launch_bounds__(NT) route_rows_kernel(const RouteRows p) {
+    extern __shared__ __align__(16) float sm[];              // x [TOK][KC] | z [TOK][experts] | groups [TOK][groups]
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, E = p.r.experts, t0 = blockIdx.x * TOK, nt = min(TOK, p.M - t0);
+    float* xs = sm;
+    float* z = sm + TOK * KC;
+    float* gs = z + TOK * E;
+    for (int i = tid; i < TOK * E; i += NT) z[i] = 0.0f;
+    for (int k0 = 0; k0 < p.r.ld; k0 += KC) {
+        __syncthreads();
+        for (int i = tid; i < TOK * KC; i += NT) {
+            const int t = i / KC, k = i - t * KC;
+            xs[t * KC + spot(k)] = t < nt && k0 + k < p.d ? p.x[(size_t)(t0 + t) * p.d + k0 + k] : 0.0f;
+        }
+        __syncthreads();
+        for (int e0 = warp * EPW; e0 < E; e0 += NT / 32 * EPW) {
+            float s[EPW][TOK] = {};
+#pragma unroll
+            for (int c = 0; c < KC; c += 256) {
+                const int k = k0 + c + lane * 8;
+                uint4 w[EPW];
+#pragma unroll
+                for (int y = 0; y < EPW; ++y)
+                    w[y] = e0 + y < E && k < p.r.ld ? __ldg((const uint4*)(p.r.w + (size_t)(e0 + y) * p.r.ld + k)) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+                for (int t = 0; t < TOK; ++t) {
+                    const float4 u = *(const float4*)(xs + t * KC + c + lane * 4), v = *(const float4*)(xs + t * KC + c + lane * 4 + 128);
+#pragma unroll
+                    for (int y = 0; y < EPW; ++y) dot8(w[y], u, v, s[y][t]);
+                }
+            }
+#pragma unroll
+            for (int y = 0; y < EPW; ++y)
+#pragma unroll
+                for (int t = 0; t < TOK; ++t) {
+                    float v = s[y][t];
+#pragma unroll
+                    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+                    if (lane == 0 && e0 + y < E) z[t * E + e0 + y] += v;
+                }
+        }
+    }
+    __syncthreads();
+    const int t = warp;
+    if (t < nt)
+        choose(z + t * E, gs + t * p.r.groups, p.r, [&](int k, int e, float w) {
+            const size_t at = (size_t)(t0 + t) * p.r.top + k;
+            p.expert[at] = e;
+            p.weight[at] = w;
+            p.index[at] = atomicAdd(p.counts + e, 1);
+        });
+}
+
+__global__ void __launch_bounds__(NT) gather_rows_kernel(const RouteRows p, const unsigned char* __restrict__ plane, int row16) {
+    extern __shared__ int off[];                             // first row of every expert's run
+    __shared__ int place[64];
+    const int tid = threadIdx.x, lane = tid & 31, E = p.r.experts, m = blockIdx.x, top = p.r.top;
+    const int per = (E + 31) / 32;
+    if (tid < 32) {                                          // a lane sums `per` neighbouring experts
+        int n = 0;
+        for (int i = lane * per; i < min(E, (lane + 1) * per); ++i) n += p.counts[i];
+        int at = n;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int x = __shfl_up_sync(0xffffffffu, at, o);
+            if (lane >= o) at += x;
+        }
+        at -= n;
+        for (int i = lane * per; i < min(E, (lane + 1) * per); ++i) { off[i] = at; at += p.counts[i]; }
+    }
+    __syncthreads();
+    if (m == 0 && tid < 32) {
+        int n = 0;
+        for (int i = lane * per; i < min(E, (lane + 1) * per); ++i) n += (p.counts[i] + p.tile_rows - 1) / p.tile_rows;
+        int at = n;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int x = __shfl_up_sync(0xffffffffu, at, o);
+            if (lane >= o) at += x;
+        }
+        if (lane == 31) *p.n_table = at;
+        at -= n;
+        for (int i = lane * per; i < min(E, (lane + 1) * per); ++i)
+            for (int r = 0; r < p.counts[i]; r += p.tile_rows) p.table[at++] = make_int4(off[i] + r, min(p.tile_rows, p.counts[i] - r), i, 0);
+    }
+    for (int s = tid; s < top; s += NT) {
+        const size_t at = (size_t)m * top + s;
+        const int row = off[p.expert[at]] + p.index[at];
+        p.index[at] = row;
+        place[s] = row;
+    }
+    __syncthreads();
+    const uint4* src = (const uint4*)(plane + (size_t)m * row16 * 16);
+    uint4* dst = (uint4*)p.rows;
+    for (int i = tid; i < row16; i += NT) {
+        const uint4 v = src[i];
+        for (int s = 0; s < top; ++s) dst[(size_t)place[s] * row16 + i] = v;
+    }
+}
+
+int max_row_tiles(const Router& r, int M, int tile_rows) {
+    const long long rows = (long long)M * r.top;
+    return (int)std::min<long long>(rows, rows / tile_rows + r.experts);
+}
+int launch_route_rows(const RouteRows& p, const void* plane, bool f32_rows, cudaStream_t st) {
+    const Router& r = p.r;
+    if (r.experts > kMaxExperts || r.groups > kMaxGroups || r.top > 64) return fail(FC_E_SHAPE, "%d experts in %d groups, %d chosen", r.experts, r.groups, r.top);
+    const size_t smem = (size_t)TOK * (KC + r.experts + r.groups) * sizeof(float);
+    if (smem > 47 * 1024) FC_CUDA(cudaFuncSetAttribute(route_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
+    route_rows_kernel<<<(p.M + TOK - 1) / TOK, NT, smem, st>>>(p);
+    FC_LAUNCHED();
+    gather_rows_kernel<<<p.M, NT, (size_t)r.experts * sizeof(int), st>>>(p, (const unsigned char*)plane, p.ld * (f32_rows ? 4 : 2) / 16);
+    FC_LAUNCHED();
+    return FC_OK;
+}
+
+// ------------------------------------------------------------------------------------------------ one token
+__global__ void __launch_bounds__(NT) route_step_kernel(const __grid_constant__ RouteStep p) {
+    extern __shared__ __align__(16) float sm[];              // x [ld up to 256s] | z [experts] | groups
+    __shared__ float red[NT / 32];
+    __shared__ bool is_last;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, d = p.d, E = p.r.experts, ld = p.r.ld, cap = (ld + 255) / 256 * 256;
+    float* xs = sm;
+    float* z = sm + cap;
+    float* gs = z + E;
+    const int e = blockIdx.x * (NT / 32) + warp;
+    const uint16_t* w = p.r.w + (size_t)min(e, E - 1) * ld;
+    uint4 pre[8];
+#pragma unroll
+    for (int c = 0; c < 8; ++c) pre[c] = c * 256 + lane * 8 < ld ? __ldg((const uint4*)(w + c * 256 + lane * 8)) : make_uint4(0, 0, 0, 0);
+    pdl_wait();
+    pdl_trigger();
+    if (p.state->done | p.state->error) return;
+    float yy = 0.0f;
+    for (int c = tid; c < cap; c += NT) {
+        const float y = c < d ? post_norm_sum(p.post, 0, c, d) : 0.0f;
+        xs[spot(c)] = y;
+        yy = fmaf(y, y, yy);
+    }
+    const float inv = 1.0f / sqrtf(block_sum_of<NT>(yy, red) / (float)d + p.eps);
+    for (int c = tid; c < d; c += NT) {
+        const float x = fmaf(xs[spot(c)] * inv, p.post.norm_w[c], p.x_in[c]);
+        xs[spot(c)] = x;
+        if (blockIdx.x == 0) p.x_out[c] = x;
+    }
+    __syncthreads();
+    float s = 0.0f;
+#pragma unroll
+    for (int c = 0; c < 8; ++c)
+        if (c * 256 < ld) dot8(pre[c], *(const float4*)(xs + c * 256 + lane * 4), *(const float4*)(xs + c * 256 + lane * 4 + 128), s);
+    for (int c = 8; c * 256 < ld; ++c)
+        if (c * 256 + lane * 8 < ld)
+            dot8(__ldg((const uint4*)(w + c * 256 + lane * 8)), *(const float4*)(xs + c * 256 + lane * 4), *(const float4*)(xs + c * 256 + lane * 4 + 128), s);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    if (lane == 0 && e < E) p.z[e] = s;
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) is_last = atomicAdd(p.counter, 1u) == gridDim.x - 1;
+    __syncthreads();
+    if (!is_last) return;
+    __threadfence();
+    if (tid == 0) *p.counter = 0;
+    for (int i = tid; i < E; i += NT) z[i] = __ldcg(p.z + i);
+    __syncthreads();
+    if (warp == 0)
+        choose(z, gs, p.r, [&](int k, int x, float v) {
+            p.expert[k] = x;
+            p.weight[k] = v;
+        });
+}
+int launch_route_step(const RouteStep& p, cudaStream_t st) {
+    const Router& r = p.r;
+    if (r.experts > kMaxExperts || r.groups > kMaxGroups) return fail(FC_E_SHAPE, "%d experts in %d groups", r.experts, r.groups);
+    const size_t smem = (size_t)((r.ld + 255) / 256 * 256 + r.experts + r.groups) * sizeof(float);
+    if (smem > 200 * 1024) return fail(FC_E_SHAPE, "rows of %d values exceed the router's staging", p.d);
+    if (smem > 47 * 1024) FC_CUDA(cudaFuncSetAttribute(route_step_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    FC_CUDA(launch_pdl(route_step_kernel, dim3((r.experts + NT / 32 - 1) / (NT / 32)), dim3(NT), smem, st, p));
+    ++g_launches;
+    return FC_OK;
+}
+
+}  // namespace fc

@@ -1,18 +1,19 @@
-// The attention of talk_attn.cu on the tcgen05 tensor cores, for portions of a prompt: queries already mixed (bf16,
-// scale, temperature and log2(e) inside), keys and values straight from the bf16 cache.
+// Attention of a portion's rows over cached keys on the tcgen05 tensor cores: bf16 queries (scale and log2(e) inside), keys
+// and values, fp32 scores, softmax and sums.
 //
-// One CTA owns 128 query rows of one head; key tiles of 64.
+// One CTA owns 128 query rows of one head; key tiles of 64, from the first the window of its rows reaches.
 //   warp 8      TMA: the query tile once (k-chunks of 64 columns; a tile too wide to stay travels again with every key
-//               tile), then per key tile the chunks of the wide key row through a ring, and the value tile of the head's
-//               key/value head (two buffers)
-//   warp 9      tcgen05.mma: S = q' K^T into one of two score buffers, one tile ahead; O += P V (V consumed MN-major),
+//               tile), then per key tile the chunks of the key row (the head's own part, then the part all heads share)
+//               through a ring, and the value tile of the head's key/value head (two buffers)
+//   warp 9      tcgen05.mma: S = q K^T into one of two score buffers, one tile ahead; O += P V (V consumed MN-major),
 //               P as bf16 hi + lo so that the weights keep 16 bits
-//   warps 0-7   two threads per query row, 32 keys each: score + bias[distance] (a 191-entry slice of the head's table per
-//               tile, -inf for keys ahead of the query), online softmax in base 2 that starts from the sink (max = sink,
-//               sum = 1), P to shared memory. O stays in TMEM; it is rescaled only when a row's maximum has grown by more than 8.
+//   warps 0-7   two threads per query row, 32 keys each: score + a 191-entry slice per tile of the distance's bias (0 without
+//               one), -inf for keys ahead of the query or behind its window; online softmax in base 2 that starts from the
+//               sink (max = sink, sum = 1) or from nothing, P to shared memory. O stays in TMEM; it is rescaled only when a
+//               row's maximum has grown by more than 8. Tiles that no edge crosses skip the slice when there is no bias.
 // Every mbarrier wait is bounded; on a timeout the status word is raised and the CTA leaves.
 //
-// Bound: tensor pipe / special-function unit. Per (query, key) pair and head KV * dim + 2 vdim multiply-adds executed.
+// Bound: tensor pipe / special-function unit. Per (query, key) pair and head w0 + w1 + 2 vdim multiply-adds executed.
 #include <algorithm>
 
 #include "bf16_ops.cuh"
@@ -41,9 +42,12 @@ struct Bars {
     float half[2][2][QT];            // per buffer, half of the tile's keys: a row's largest score; at the end its sums
 };
 struct Args {
-    int M, pos0, kd, nkc, ks, nv, H, KV, vdim, vp, far, ldo;
+    int M, pos0, kq, nkc, ks, nv, H, KV, vdim, far, ldo, window;
+    int nc0, w0, last0, last1;       // chunks and columns of the head's own key part; MMA steps of either part's last chunk
+    int k0_col, k0_head, k0_base, k1_col, k1_base, v_col, v_head, v_base;
+    int has_sink;
     int q_stream;        // the query tile is too wide to stay in shared memory: its chunks travel with the key chunks
-    const float *bias, *sink;
+    const float *bias, *sink;        // bias null: none; has_sink with sink null: a score of 0
     uint16_t* out;
     int* status;
     long long wait_cycles;
@@ -66,8 +70,8 @@ int plan_stages(int nkc, int nv, bool q_stream) {
 }  // namespace
 
 __global__ void __launch_bounds__(THREADS, 1)
-talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv,
-                       const Args a) {
+flash_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk0, const __grid_constant__ CUtensorMap mk1,
+                const __grid_constant__ CUtensorMap mv, const Args a) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char* smem = (unsigned char*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     unsigned char* sk = smem + (a.q_stream ? a.ks : a.nkc) * Q_CHUNK;
@@ -77,7 +81,8 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int q0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * QT, h = blockIdx.x, kv = h / (a.H / a.KV);
     const int last = a.pos0 + min(a.M, q0 + QT) - 1;       // the last key any row of the tile sees
-    const int n_kt = last / KT + 1;
+    const int kt0 = max(0, a.pos0 + q0 - a.window + 1) / KT;    // the first tile any of them sees
+    const int n_kt = last / KT + 1 - kt0;                  // tiles are counted from there
 
     if (threadIdx.x == 0) {
         mbar_init(&bars->q_full, 1);
@@ -101,7 +106,8 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
     if (warp == TMA_WARP) {
         if (lane == 0 && !a.withhold) {
             if (!a.q_stream) mbar_expect_tx(&bars->q_full, a.nkc * Q_CHUNK);
-            for (int c = 0; !a.q_stream && c < a.nkc; ++c) tma_load_2d(smem + c * Q_CHUNK, &mq, h * a.kd + c * CH, q0, &bars->q_full);
+            auto q_x = [&](int c) { return h * a.kq + (c < a.nc0 ? c * CH : a.w0 + (c - a.nc0) * CH); };
+            for (int c = 0; !a.q_stream && c < a.nkc; ++c) tma_load_2d(smem + c * Q_CHUNK, &mq, q_x(c), q0, &bars->q_full);
             int s = 0, issued = 0, nvt = 0;               // ring stage, key chunks and value tiles asked for
             uint32_t ph = 1;                              // parity of k_empty: a fresh ring is empty
             bool ok = true;
@@ -110,8 +116,9 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
                     ok = wait(&bars->k_empty[s], ph);
                     if (!ok) break;
                     mbar_expect_tx(&bars->k_full[s], a.q_stream ? K_CHUNK + Q_CHUNK : K_CHUNK);
-                    if (a.q_stream) tma_load_2d(smem + s * Q_CHUNK, &mq, h * a.kd + c * CH, q0, &bars->k_full[s]);
-                    tma_load_2d(sk + s * K_CHUNK, &mk, c * CH, kt * KT, &bars->k_full[s]);
+                    if (a.q_stream) tma_load_2d(smem + s * Q_CHUNK, &mq, q_x(c), q0, &bars->k_full[s]);
+                    if (c < a.nc0) tma_load_2d(sk + s * K_CHUNK, &mk0, a.k0_col + kv * a.k0_head + c * CH, (kt0 + kt) * KT - a.k0_base, &bars->k_full[s]);
+                    else tma_load_2d(sk + s * K_CHUNK, &mk1, a.k1_col + (c - a.nc0) * CH, (kt0 + kt) * KT - a.k1_base, &bars->k_full[s]);
                     ++issued;
                     if (++s == a.ks) { s = 0; ph ^= 1; }
                 }
@@ -119,7 +126,7 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
                 ok = ok && wait(&bars->v_empty[b], ((kt >> 1) & 1) ^ 1);
                 if (!ok) break;
                 mbar_expect_tx(&bars->v_full[b], a.nv * K_CHUNK);
-                for (int c = 0; c < a.nv; ++c) tma_load_2d(sv_ + (b * a.nv + c) * K_CHUNK, &mv, kv * a.vp + c * CH, kt * KT, &bars->v_full[b]);
+                for (int c = 0; c < a.nv; ++c) tma_load_2d(sv_ + (b * a.nv + c) * K_CHUNK, &mv, a.v_col + kv * a.v_head + c * CH, (kt0 + kt) * KT - a.v_base, &bars->v_full[b]);
                 ++nvt;
             }
             if (bars->abort) {                            // leaving early: no copy may still be on its way into this CTA
@@ -146,9 +153,11 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
                 for (int c = 0; c < a.nkc; ++c) {
                     if (!wait(&bars->k_full[s], kph)) return false;
                     fence_after();
+                    const int steps = c + 1 == a.nc0 ? a.last0 : (c + 1 == a.nkc ? a.last1 : CH / 16);
                     const uint64_t qd = q_desc + (uint64_t)((a.q_stream ? s : c) * (Q_CHUNK >> 4)), kd = k_desc + (uint64_t)(s * (K_CHUNK >> 4));
 #pragma unroll
-                    for (int ks = 0; ks < CH / 16; ++ks) umma(tmem + b * KT, qd + (uint64_t)(ks * 2), kd + (uint64_t)(ks * 2), IDESC_S, (c | ks) != 0);
+                    for (int ks = 0; ks < CH / 16; ++ks)
+                        if (ks < steps) umma(tmem + b * KT, qd + (uint64_t)(ks * 2), kd + (uint64_t)(ks * 2), IDESC_S, (c | ks) != 0);
                     umma_commit(&bars->k_empty[s]);
                     if (++s == a.ks) { s = 0; kph ^= 1; }
                 }
@@ -177,22 +186,29 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
     } else {
         // two threads a query row, each with half of the tile's keys (and of the output's columns)
         const int hf = warp >> 2, r = (warp & 3) * 32 + lane, tid = threadIdx.x;
-        const float* bias = a.bias + (size_t)h * (a.far + 1);
-        float m = a.sink[h] * kLog2e, l = hf == 0 ? 1.0f : 0.0f;
+        const float* bias = a.bias ? a.bias + (size_t)h * (a.far + 1) : nullptr;
+        // without a sink the maximum starts below every score, and what precedes the first visible key is scaled away
+        float m = a.has_sink ? (a.sink ? a.sink[h] * kLog2e : 0.0f) : -1e30f, l = a.has_sink && hf == 0 ? 1.0f : 0.0f;
         unsigned char* ph = sp + r * 128;
         unsigned char* pl = ph + P_BYTES;
         const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
         constexpr int HK = KT / 2;
         auto bias_at = [&](int kt) -> float {              // entry tid of tile kt's slice of the table
-            const int n = a.pos0 + q0 - kt * KT - (KT - 1) + tid;
-            return n < 0 ? -INFINITY : __ldg(bias + min(n, a.far)) * kLog2e;
+            const int n = a.pos0 + q0 - (kt0 + kt) * KT - (KT - 1) + tid;
+            if (n < 0 || n >= a.window) return -INFINITY;
+            return bias ? __ldg(bias + min(n, a.far)) * kLog2e : 0.0f;
+        };
+        auto edges = [&](int kt) -> bool {                 // does any pair of tile kt need the slice?
+            const int n = a.pos0 + q0 - (kt0 + kt) * KT;   // distance of the first row to the first key
+            return bias || n < KT - 1 || n + QT - 1 >= a.window;
         };
         float next_bias = bias_at(0);
         bool ok = true;
         for (int kt = 0; kt < n_kt; ++kt) {
             const int b = kt & 1;
             float* bt = bars->bias[b];
-            if (tid < QT + KT - 1) bt[tid] = next_bias;
+            const bool slice = edges(kt);
+            if (slice && tid < QT + KT - 1) bt[tid] = next_bias;
             if (kt + 1 < n_kt) next_bias = bias_at(kt + 1);
             ok = __all_sync(0xffffffffu, wait(&bars->s_full[b], (kt >> 1) & 1));
             uint32_t sr[HK];
@@ -206,14 +222,15 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
             }
             // one warp's timeout must not leave the others at a named barrier: everybody goes on to them, tile by tile, with
             // waits that the abort flag ends at once
-            asm volatile("bar.sync 1, 256;" ::: "memory");
+            // (a slice's buffer is written again two tiles on, after o_done of this tile, which every warp's P precedes)
+            if (slice) asm volatile("bar.sync 1, 256;" ::: "memory");
             if (ok) {
+                if (slice) {
 #pragma unroll
-                for (int j = 0; j < HK; ++j) {
-                    const float s = __uint_as_float(sr[j]) + bt[r + (KT - 1) - hf * HK - j];
-                    sr[j] = __float_as_uint(s);
-                    mx = fmaxf(mx, s);
+                    for (int j = 0; j < HK; ++j) sr[j] = __float_as_uint(__uint_as_float(sr[j]) + bt[r + (KT - 1) - hf * HK - j]);
                 }
+#pragma unroll
+                for (int j = 0; j < HK; ++j) mx = fmaxf(mx, __uint_as_float(sr[j]));
                 bars->half[b][hf][r] = mx;
             }
             // the two warps of these 32 rows
@@ -301,30 +318,41 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_cons
     }
 }
 
-int launch_talk_prefill_tc(const TalkAttn& t, const void* qm, const void* kc, const void* vc, int M, int pos0, int ctx, void* out, int ldo,
-                           int* status, cudaStream_t st) {
+int launch_flash_tc(const Flash& f, const void* q, int M, int pos0, void* out, int ldo, int* status, cudaStream_t st) {
+    const int w0 = f.k0.width, w1 = f.k1.p ? f.k1.width : 0;
+    if (f.vdim > 256) return fail(FC_E_SHAPE, "value heads of %d do not fit the tensor-core attention", f.vdim);
+    if (w0 <= 0 || w0 % 16 || w1 % 16 || f.k0.col % 16 || f.k0.head_stride % 16 || f.k1.col % 16 || f.v.head_stride % 16 || f.v.width % 16)
+        return fail(FC_E_SHAPE, "tensor-core attention: key parts of %d and %d columns", w0, w1);
     Args a = {};
-    a.nkc = (t.kd + CH - 1) / CH;
-    a.nv = (t.vp + CH - 1) / CH;
-    if (t.vdim > 256) return fail(FC_E_SHAPE, "value heads of %d do not fit the tensor-core attention", t.vdim);
+    a.nc0 = (w0 + CH - 1) / CH;
+    const int nc1 = (w1 + CH - 1) / CH;
+    a.nkc = a.nc0 + nc1;
+    a.last0 = (w0 - (a.nc0 - 1) * CH) / 16;
+    a.last1 = nc1 ? (w1 - (nc1 - 1) * CH) / 16 : a.last0;
+    a.nv = (f.v.width + CH - 1) / CH;
     a.ks = plan_stages(a.nkc, a.nv, false);
     if (!a.ks) { a.q_stream = 1; a.ks = plan_stages(a.nkc, a.nv, true); }
     static bool attr_set[64] = {};
     int dev = 0;
     FC_CUDA(cudaGetDevice(&dev));
     if (dev < 64 && !attr_set[dev]) {
-        FC_CUDA(cudaFuncSetAttribute(talk_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+        FC_CUDA(cudaFuncSetAttribute(flash_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
         attr_set[dev] = true;
     }
-    CUtensorMap mq, mk, mv;
-    FC_TRY(encode_bf16(&mq, qm, M, (size_t)t.H * t.kd, (size_t)t.H * t.kd, QT));
-    FC_TRY(encode_bf16(&mk, kc, ctx, t.kd, t.kd, KT));
-    FC_TRY(encode_bf16(&mv, vc, ctx, (size_t)t.KV * t.vp, (size_t)t.KV * t.vp, KT));
-    a.M = M; a.pos0 = pos0; a.kd = t.kd; a.H = t.H; a.KV = t.KV; a.vdim = t.vdim; a.vp = t.vp; a.far = t.far; a.ldo = ldo;
-    a.bias = t.bias; a.sink = t.sink; a.out = (uint16_t*)out; a.status = status;
+    CUtensorMap mq, mk0, mk1, mv;
+    a.kq = w0 + w1;
+    FC_TRY(encode_bf16(&mq, q, M, (size_t)f.H * a.kq, (size_t)f.H * a.kq, QT));
+    FC_TRY(encode_bf16(&mk0, f.k0.p, f.k0.rows, f.k0.ld, f.k0.ld, KT));
+    mk1 = mk0;
+    if (w1) FC_TRY(encode_bf16(&mk1, f.k1.p, f.k1.rows, f.k1.ld, f.k1.ld, KT));
+    FC_TRY(encode_bf16(&mv, f.v.p, f.v.rows, f.v.ld, f.v.ld, KT));
+    a.M = M; a.pos0 = pos0; a.H = f.H; a.KV = f.KV; a.vdim = f.vdim; a.far = f.far; a.ldo = ldo; a.window = f.window; a.w0 = w0;
+    a.k0_col = f.k0.col; a.k0_head = f.k0.head_stride; a.k0_base = f.k0.pos0; a.k1_col = f.k1.col; a.k1_base = f.k1.pos0;
+    a.v_col = f.v.col; a.v_head = f.v.head_stride; a.v_base = f.v.pos0;
+    a.bias = f.bias; a.has_sink = f.has_sink; a.sink = f.sink; a.out = (uint16_t*)out; a.status = status;
     a.wait_cycles = g_debug.wait_cycles; a.withhold = g_debug.withhold;
     a.tmem_cols = a.nv <= 2 ? 256 : 512;
-    talk_prefill_tc_kernel<<<dim3(t.H, (M + QT - 1) / QT), THREADS, smem_bytes(a.nkc, a.ks, a.nv, a.q_stream), st>>>(mq, mk, mv, a);
+    flash_tc_kernel<<<dim3(f.H, (M + QT - 1) / QT), THREADS, smem_bytes(a.nkc, a.ks, a.nv, a.q_stream), st>>>(mq, mk0, mk1, mv, a);
     FC_LAUNCHED();
     return FC_OK;
 }

@@ -33,15 +33,23 @@ struct Bars {
 };
 constexpr int SMEM_BYTES = STAGES * STAGE_BYTES + 1024 + (int)sizeof(Bars);
 
-struct Tile { int seg, m0, n0; };
+// Rows [m0, m_end) of the operand plane (and of the output), columns from n0 on, weight rows from b0 on.
+struct Tile { int seg, m0, m_end, n0, b0; };
+template <bool RAGGED>
 __device__ __forceinline__ Tile locate(const GemmGroup& g, int tile) {
+    if constexpr (RAGGED) {
+        const int e = tile / g.seg[0].tiles_n;
+        const int4 t = __ldg(g.ragged.table + e);
+        return {0, t.x, t.x + t.y, (tile - e * g.seg[0].tiles_n) * BN, g.seg[0].b_row0 + t.z * g.ragged.b_step};
+    }
     int s = 0;
     while (s + 1 < g.n_seg && tile >= g.seg[s + 1].tile0) ++s;
     const int local = tile - g.seg[s].tile0;
-    return {s, (local / g.seg[s].tiles_n) * BM, (local % g.seg[s].tiles_n) * BN};
+    return {s, (local / g.seg[s].tiles_n) * BM, g.M, (local % g.seg[s].tiles_n) * BN, g.seg[s].b_row0};
 }
 }  // namespace
 
+template <bool RAGGED>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_bf16_group_kernel(const __grid_constant__ GemmMaps maps, const __grid_constant__ GemmGroup g) {
     extern __shared__ unsigned char smem_raw[];
@@ -49,6 +57,7 @@ gemm_bf16_group_kernel(const __grid_constant__ GemmMaps maps, const __grid_const
     Bars* bars = (Bars*)(smem + STAGES * STAGE_BYTES);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
+    const int n_tiles = RAGGED ? *g.ragged.n * g.seg[0].tiles_n : g.n_tiles;
     if (threadIdx.x == 0) {
         for (int s = 0; s < STAGES; ++s) { mbar_init(&bars->full[s], 1); mbar_init(&bars->empty[s], 1); }
         for (int b = 0; b < 2; ++b) { mbar_init(&bars->acc_full[b], 1); mbar_init(&bars->acc_empty[b], EPI_WARPS); }
@@ -64,21 +73,21 @@ gemm_bf16_group_kernel(const __grid_constant__ GemmMaps maps, const __grid_const
     if (warp == TMA_WARP) {
         if (lane == 0 && !g.withhold) {
             int it = 0;
-            for (int tile = blockIdx.x; tile < g.n_tiles; tile += gridDim.x) {
-                const Tile t = locate(g, tile);
+            for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x) {
+                const Tile t = locate<RAGGED>(g, tile);
                 const GemmSeg& s = g.seg[t.seg];
-                const bool two = t.m0 + 128 < g.M;
+                const bool two = t.m0 + 128 < t.m_end;
                 const CUtensorMap* ma = &maps.a[s.a_map];
                 const CUtensorMap* mb = &maps.b[s.b_map];
                 for (int kb = 0; kb < s.kb; ++kb, ++it) {
                     const int st = it % STAGES;
-                    if (!wait_bar(&bars->abort, &bars->empty[st], ((it / STAGES) & 1) ^ 1, g.status, g.wait_cycles)) { tile = g.n_tiles; break; }
+                    if (!wait_bar(&bars->abort, &bars->empty[st], ((it / STAGES) & 1) ^ 1, g.status, g.wait_cycles)) { tile = n_tiles; break; }
                     unsigned char* p = smem + st * STAGE_BYTES;
                     mbar_expect_tx(&bars->full[st], (two ? 3 : 2) * TILE_BYTES);
                     const int x = (s.kb0 + kb) * BK;
                     tma_load_2d(p, ma, x, s.a_row0 + t.m0, &bars->full[st]);
                     if (two) tma_load_2d(p + TILE_BYTES, ma, x, s.a_row0 + t.m0 + 128, &bars->full[st]);
-                    tma_load_2d(p + 2 * TILE_BYTES, mb, x, s.b_row0 + t.n0, &bars->full[st]);
+                    tma_load_2d(p + 2 * TILE_BYTES, mb, x, t.b0 + t.n0, &bars->full[st]);
                 }
             }
             if (bars->abort)                              // leaving early: no copy may still be on its way into this CTA
@@ -91,9 +100,9 @@ gemm_bf16_group_kernel(const __grid_constant__ GemmMaps maps, const __grid_const
         if (lane == 0) {
             int it = 0, ti = 0;
             bool ok = true;
-            for (int tile = blockIdx.x; tile < g.n_tiles && ok; tile += gridDim.x, ++ti) {
-                const Tile t = locate(g, tile);
-                const int nkb = g.seg[t.seg].kb, halves = t.m0 + 128 < g.M ? 2 : 1, buf = ti & 1;
+            for (int tile = blockIdx.x; tile < n_tiles && ok; tile += gridDim.x, ++ti) {
+                const Tile t = locate<RAGGED>(g, tile);
+                const int nkb = g.seg[t.seg].kb, halves = t.m0 + 128 < t.m_end ? 2 : 1, buf = ti & 1;
                 ok = wait_bar(&bars->abort, &bars->acc_empty[buf], ((ti >> 1) & 1) ^ 1, g.status, g.wait_cycles);
                 if (!ok) break;
                 fence_after();
@@ -118,8 +127,8 @@ gemm_bf16_group_kernel(const __grid_constant__ GemmMaps maps, const __grid_const
     } else {
         int ti = 0;
         const int hm = warp >> 2, quarter = warp & 3;
-        for (int tile = blockIdx.x; tile < g.n_tiles; tile += gridDim.x, ++ti) {
-            const Tile t = locate(g, tile);
+        for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x, ++ti) {
+            const Tile t = locate<RAGGED>(g, tile);
             const GemmSeg& s = g.seg[t.seg];
             const int buf = ti & 1;
             if (!wait_bar(&bars->abort, &bars->acc_full[buf], (ti >> 1) & 1, g.status, g.wait_cycles)) break;
@@ -137,10 +146,13 @@ gemm_bf16_group_kernel(const __grid_constant__ GemmMaps maps, const __grid_const
                     if (lane == 0) mbar_arrive(&bars->acc_empty[buf]);
                 }
                 const int nb = t.n0 + c * 32;
-                if (m < g.M && nb < s.n) {
+                if (m < t.m_end && nb < s.n) {
                     if (s.epi == ROW_XIELU) {
 #pragma unroll
                         for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(xielu_f(__uint_as_float(r[i]), s.c0, s.c1));
+                    } else if (s.epi == ROW_GELU) {
+#pragma unroll
+                        for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(gelu_erf_f(__uint_as_float(r[i])));
                     }
                     const bool full = nb + 32 <= s.n;
                     const size_t off = (size_t)m * s.ldy + nb;
@@ -177,15 +189,22 @@ gemm_bf16_group_kernel(const __grid_constant__ GemmMaps maps, const __grid_const
     }
 }
 
-int launch_gemm_bf16_group(const GemmMaps& maps, GemmGroup g, int M, int* status, cudaStream_t st) {
+static int prepare(int* sms_out) {
     static int sms[64] = {};
     int dev = 0;
     FC_CUDA(cudaGetDevice(&dev));
     if (dev >= 64) return fail(FC_E_ARG, "device %d out of range", dev);
     if (!sms[dev]) {
-        FC_CUDA(cudaFuncSetAttribute(gemm_bf16_group_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
+        FC_CUDA(cudaFuncSetAttribute(gemm_bf16_group_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
+        FC_CUDA(cudaFuncSetAttribute(gemm_bf16_group_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
         FC_CUDA(cudaDeviceGetAttribute(&sms[dev], cudaDevAttrMultiProcessorCount, dev));
     }
+    *sms_out = sms[dev];
+    return FC_OK;
+}
+int launch_gemm_bf16_group(const GemmMaps& maps, GemmGroup g, int M, int* status, cudaStream_t st) {
+    int sms = 0;
+    FC_TRY(prepare(&sms));
     if (M <= 0 || g.n_seg <= 0 || g.n_seg > kGemmSegs) return fail(FC_E_SHAPE, "grouped GEMM: M = %d, %d segments", M, g.n_seg);
     const int tiles_m = (M + BM - 1) / BM;
     int tiles = 0;
@@ -196,7 +215,20 @@ int launch_gemm_bf16_group(const GemmMaps& maps, GemmGroup g, int M, int* status
     }
     g.M = M; g.n_tiles = tiles; g.status = status;
     g.wait_cycles = g_debug.wait_cycles; g.withhold = g_debug.withhold;
-    gemm_bf16_group_kernel<<<std::min(tiles, sms[dev]), THREADS, SMEM_BYTES, st>>>(maps, g);
+    gemm_bf16_group_kernel<false><<<std::min(tiles, sms), THREADS, SMEM_BYTES, st>>>(maps, g);
+    FC_LAUNCHED();
+    return FC_OK;
+}
+int launch_gemm_bf16_ragged(const GemmMaps& maps, const GemmSeg& seg, const Ragged& r, int max_entries, int* status, cudaStream_t st) {
+    static_assert(kRaggedRows == BM, "a table entry is a tile's rows");
+    int sms = 0;
+    FC_TRY(prepare(&sms));
+    GemmGroup g = {};
+    g.seg[0] = seg; g.n_seg = 1; g.ragged = r; g.status = status;
+    g.seg[0].tiles_n = (seg.n + BN - 1) / BN;
+    g.wait_cycles = g_debug.wait_cycles; g.withhold = g_debug.withhold;
+    if (max_entries <= 0 || seg.n <= 0) return fail(FC_E_SHAPE, "product over runs: %d entries, n = %d", max_entries, seg.n);
+    gemm_bf16_group_kernel<true><<<(int)std::min<long long>((long long)max_entries * g.seg[0].tiles_n, sms), THREADS, SMEM_BYTES, st>>>(maps, g);
     FC_LAUNCHED();
     return FC_OK;
 }
@@ -206,9 +238,17 @@ int launch_gemm_bf16_group(const GemmMaps& maps, GemmGroup g, int M, int* status
 namespace {
 constexpr int FM = 64, FN = 64, FK = 32;
 }
-__global__ void __launch_bounds__(256) gemm_bf16w_f32_kernel(const uint16_t* __restrict__ w, int K_pad, int n, const GemmF32 p, int M) {
+__global__ void __launch_bounds__(256) gemm_bf16w_f32_kernel(const uint16_t* __restrict__ w, int K_pad, int n, const GemmF32 p, int M,
+                                                             const Ragged runs) {
     __shared__ __align__(16) float As[FK][FM + 4], Bs[FK][FN + 4];
-    const int t = threadIdx.x, m0 = blockIdx.y * FM, n0 = blockIdx.x * FN;
+    const int t = threadIdx.x, n0 = blockIdx.x * FN;
+    int m0 = blockIdx.y * FM;
+    if (runs.table) {                                     // rows m0 .. M - 1 of one run, with its weights
+        if ((int)blockIdx.y >= *runs.n) return;
+        const int4 e = __ldg(runs.table + blockIdx.y);
+        m0 = e.x; M = e.x + e.y;
+        w += (size_t)e.z * runs.b_step * K_pad;
+    }
     const int row = t >> 2, k8 = (t & 3) * 8;             // this thread loads 8 consecutive k of one row
     const bool va = m0 + row < M, vb = n0 + row < n;
     const float* ap = p.a + (size_t)(va ? m0 + row : 0) * p.lda + k8;
@@ -262,6 +302,7 @@ __global__ void __launch_bounds__(256) gemm_bf16w_f32_kernel(const uint16_t* __r
             if (c >= n) continue;
             float v = acc[i][j];
             if (p.epi == ROW_XIELU) v = xielu_f(v, p.c0, p.c1);
+            else if (p.epi == ROW_GELU) v = gelu_erf_f(v);
             else if (p.epi == ROW_DECAY) v = expf(-expf(v + p.vec[c]));
             if (p.y) p.y[(size_t)m * p.ldy + c] = v;
             else p.yb[(size_t)m * p.ldy + c] = __bfloat16_as_ushort(__float2bfloat16_rn(v));
@@ -270,7 +311,14 @@ __global__ void __launch_bounds__(256) gemm_bf16w_f32_kernel(const uint16_t* __r
 }
 int launch_gemm_bf16w_f32(const BMat& w, int row0, int n, const GemmF32& p, int M, cudaStream_t st) {
     if (M <= 0 || n <= 0 || p.lda % 4 || ((uintptr_t)p.a & 15)) return fail(FC_E_SHAPE, "f32 product: M = %d, n = %d, lda = %d", M, n, p.lda);
-    gemm_bf16w_f32_kernel<<<dim3((n + FN - 1) / FN, (M + FM - 1) / FM), 256, 0, st>>>(w.w + (size_t)row0 * w.K_pad, w.K_pad, n, p, M);
+    gemm_bf16w_f32_kernel<<<dim3((n + FN - 1) / FN, (M + FM - 1) / FM), 256, 0, st>>>(w.w + (size_t)row0 * w.K_pad, w.K_pad, n, p, M, Ragged{});
+    FC_LAUNCHED();
+    return FC_OK;
+}
+int launch_gemm_bf16w_f32_ragged(const BMat& w, int n, const GemmF32& p, const Ragged& r, int max_entries, cudaStream_t st) {
+    static_assert(kRaggedRowsF32 == FM, "a table entry is a tile's rows");
+    if (max_entries <= 0 || n <= 0 || p.lda % 4 || ((uintptr_t)p.a & 15)) return fail(FC_E_SHAPE, "f32 product over runs: %d entries, n = %d, lda = %d", max_entries, n, p.lda);
+    gemm_bf16w_f32_kernel<<<dim3((n + FN - 1) / FN, max_entries), 256, 0, st>>>(w.w, w.K_pad, n, p, 0, r);
     FC_LAUNCHED();
     return FC_OK;
 }

@@ -1,12 +1,13 @@
 // Several products of one activation row in one launch, on bf16 weights: the decode counterpart of the grouped GEMM.
 //
 // The rows of all segments form one list that is cut into equal shares of bytes, one persistent CTA of 16 warps per SM.
-// A warp takes a row (or a K slice given as a segment of its own) at a time: 16-byte loads, up to 2048 weights of the row
-// in registers at once, two such pieces in flight; activations are f32 in shared memory, sums are f32.
+// A warp takes pieces of 2048 weights, two in flight: a row (or a K slice given as a segment of its own) that is longer takes
+// several, of rows of at most 1024, 512 or 256 weights a piece holds 2, 4 or 8. 16-byte loads, activations f32 in shared
+// memory, f32 sums. A segment's rows may begin at an index read from the device (an expert chosen there).
 // Launched as a programmatic dependent: the first two pieces of every warp are requested before the wait on the kernel
 // ahead, since weights never change.
 //
-// Prologues: plain inputs; or the residual update of the layer before, the norm and the token-shift mixes of the row
+// Prologues: plain inputs; the residual of layers that norm what they add (and a norm of it); or the residual update of the layer before, the norm and the token-shift mixes of the row
 // (every CTA computes them for itself, CTA 0 stores the residual and the token-shift row); or residual and norm alone
 // (the head). The residual alternates between two buffers and the token-shift row between two slots (by the position's
 // parity), so that no CTA overwrites what another still reads.
@@ -75,21 +76,29 @@ __global__ void __launch_bounds__(NT, 1) gemv_bf16_group_kernel(const __grid_con
         if (row < end) break;
     }
     const uint16_t* base = nullptr;
-    int ldw = 0, K_pad = 0, pieces = 1, items = 0;
+    int ldw = 0, K_pad = 0, pieces = 1, lc = 3, items = 0;    // a piece holds 8 >> lc rows of 1 << lc loads of 256 weights
+    bool ready = false;                            // past the wait: indices may be read
     auto open = [&]() {
-        if (seg >= g.n_seg) { items = 0; return; }
-        ldw = g.seg[seg].ldw;
-        base = g.seg[seg].w + (size_t)row * ldw;
-        K_pad = g.seg[seg].K_pad;
+        items = 0;
+        if (seg >= g.n_seg) return;
+        const GemvSeg& s = g.seg[seg];
+        ldw = s.ldw;
+        K_pad = s.K_pad;
         pieces = (K_pad + PIECE - 1) / PIECE;
-        const int mine = end - row - warp;
-        items = mine > 0 ? (mine + NW - 1) / NW * pieces : 0;
+        lc = K_pad > 1024 ? 3 : (K_pad > 512 ? 2 : (K_pad > 256 ? 1 : 0));
+        const int rp = 8 >> lc, mine = end - row - warp * rp;
+        if (s.index && !ready) return;             // loaded after the wait
+        base = s.w + (size_t)row * ldw;
+        if (s.index) base += (size_t)*s.index * s.w_step;
+        items = mine > 0 ? (mine + NW * rp - 1) / (NW * rp) * pieces : 0;
     };
-    auto load = [&](Piece& p, int i) {             // item i: piece i % pieces of row warp + (i / pieces) NW
-        const int ri = i / pieces, k0 = (i - ri * pieces) * PIECE + lane * 8;
-        const uint16_t* src = base + (size_t)(warp + ri * NW) * ldw;
+    auto load = [&](Piece& p, int i) {             // item i: piece i % pieces of the rows from (warp + (i / pieces) NW) rp on
+        const int ri = i / pieces, k0 = (i - ri * pieces) * PIECE + lane * 8, rp = 8 >> lc, r0 = (warp + ri * NW) * rp;
 #pragma unroll
-        for (int c = 0; c < 8; ++c) p.w[c] = i < items && k0 + c * 256 < K_pad ? ld_stream(src + k0 + c * 256) : make_uint4(0, 0, 0, 0);
+        for (int c = 0; c < 8; ++c) {
+            const int r = r0 + (c >> lc), k = k0 + (c & ((1 << lc) - 1)) * 256;
+            p.w[c] = i < items && r < end - row && k < K_pad ? ld_stream(base + (size_t)r * ldw + k) : make_uint4(0, 0, 0, 0);
+        }
     };
     Piece pa, pb;
     open();
@@ -98,10 +107,28 @@ __global__ void __launch_bounds__(NT, 1) gemv_bf16_group_kernel(const __grid_con
     pdl_wait();
     pdl_trigger();
     if (g.state->done | g.state->error) return;
+    ready = true;
+    if (seg < g.n_seg && g.seg[seg].index) { open(); load(pa, 0); load(pb, 1); }
 
     if (g.mode != 0) {
         const int pos = g.state->pos;
         float ss = 0.0f;
+        const bool post = g.mode >= 3;
+        if (post && g.post.y) {
+            float yy = 0.0f;
+            for (int c = tid; c < d; c += NT) {
+                const float y = post_norm_sum(g.post, 0, c, d);
+                hs[c] = y;
+                yy = fmaf(y, y, yy);
+            }
+            const float iy = 1.0f / sqrtf(block_sum2(yy, 0.0f, red).x / (float)d + g.eps);
+            for (int c = tid; c < d; c += NT) {
+                const float x = fmaf(hs[c] * iy, g.post.norm_w[c], g.x_in[c]);
+                if (blockIdx.x == 0 && g.x_out) g.x_out[c] = x;
+                hs[c] = x;
+                ss = fmaf(x, x, ss);
+            }
+        } else
         if (g.prev.outs) {
             const float* lo = g.prev.outs;
             const float* ro = lo + g.prev.stride;
@@ -127,17 +154,27 @@ __global__ void __launch_bounds__(NT, 1) gemv_bf16_group_kernel(const __grid_con
             const uint16_t* e = g.embed.table + (size_t)id * g.embed.ld;
             for (int c = tid; c < d; c += NT) {
                 const float x = __uint_as_float((uint32_t)e[c] << 16) * g.embed.scale;
-                if (blockIdx.x == 0 && g.x_out) g.x_out[c] = x;
+                if (!post && blockIdx.x == 0 && g.x_out) g.x_out[c] = x;
                 hs[c] = x;
                 ss = fmaf(x, x, ss);
+            }
+            if (post) {                             // the normed embedding is the residual's first value
+                const float ie = 1.0f / sqrtf(block_sum2(ss, 0.0f, red).x / (float)d + g.eps);
+                ss = 0.0f;
+                for (int c = tid; c < d; c += NT) {
+                    const float x = hs[c] * ie * g.post.norm_w[c];
+                    if (blockIdx.x == 0 && g.x_out) g.x_out[c] = x;
+                    hs[c] = x;
+                    ss = fmaf(x, x, ss);
+                }
             }
         } else {
             for (int c = tid; c < d; c += NT) { const float x = g.x_in[c]; hs[c] = x; ss = fmaf(x, x, ss); }
         }
-        const float inv = 1.0f / sqrtf(block_sum2(ss, 0.0f, red).x / (float)d + g.eps);
+        const float inv = g.mode == 3 ? 1.0f : 1.0f / sqrtf(block_sum2(ss, 0.0f, red).x / (float)d + g.eps);
         const float* before = g.mode == 1 ? g.shift + (size_t)(pos & 1) * g.shift_slot : nullptr;
         float* after = g.mode == 1 ? g.shift + (size_t)((pos + 1) & 1) * g.shift_slot : nullptr;
-        for (int c = tid; c < d; c += NT) {
+        for (int c = tid; g.mode != 3 && c < d; c += NT) {
             const float h = hs[c] * inv * g.norm_w[c];
             hs[c] = h;
             if (before) {
@@ -150,7 +187,7 @@ __global__ void __launch_bounds__(NT, 1) gemv_bf16_group_kernel(const __grid_con
     while (seg < g.n_seg) {
         const GemvSeg& s = g.seg[seg];
         __syncthreads();                            // hs is complete / the last segment's input has been read
-        const int kr = pieces * PIECE;
+        const int kr = pieces > 1 ? pieces * PIECE : 256 << lc;
         if (g.mode == 0) {
             const float* x = g.x[s.src];
             for (int k = tid; k < kr; k += NT) xs[spot(k)] = k < s.K ? x[k] : 0.0f;
@@ -163,29 +200,35 @@ __global__ void __launch_bounds__(NT, 1) gemv_bf16_group_kernel(const __grid_con
         __syncthreads();
         float acc = 0.0f;
         auto work = [&](const Piece& p, int i) {
-            const int ri = i / pieces, pc = i - ri * pieces;
+            const int ri = i / pieces, pc = i - ri * pieces, mask = (1 << lc) - 1, r0 = (warp + ri * NW) * (8 >> lc);
             const float* x = xs + pc * PIECE + lane * 4;
             float a0 = 0.0f, a1 = 0.0f;
 #pragma unroll
             for (int c = 0; c < 8; ++c) {
-                if (pc * PIECE + c * 256 < K_pad) {                     // uniform
-                    const float4 u = *(const float4*)(x + c * 256), v = *(const float4*)(x + c * 256 + 128);
+                const int kc = (c & mask) * 256;
+                if (pc * PIECE + kc < K_pad) {                          // uniform
+                    const float4 u = *(const float4*)(x + kc), v = *(const float4*)(x + kc + 128);
                     const uint4 w = p.w[c];
                     a0 = fmaf(__uint_as_float(w.x << 16), u.x, a0); a1 = fmaf(__uint_as_float(w.x & 0xffff0000u), u.y, a1);
                     a0 = fmaf(__uint_as_float(w.y << 16), u.z, a0); a1 = fmaf(__uint_as_float(w.y & 0xffff0000u), u.w, a1);
                     a0 = fmaf(__uint_as_float(w.z << 16), v.x, a0); a1 = fmaf(__uint_as_float(w.z & 0xffff0000u), v.y, a1);
                     a0 = fmaf(__uint_as_float(w.w << 16), v.z, a0); a1 = fmaf(__uint_as_float(w.w & 0xffff0000u), v.w, a1);
                 }
-            }
-            acc += a0 + a1;
-            if (pc + 1 == pieces) {
-                float v = acc;
-                acc = 0.0f;
+                if ((c & mask) == mask) {                               // uniform: the end of a row of this piece
+                    acc += a0 + a1;
+                    a0 = a1 = 0.0f;
+                    if (pc + 1 == pieces) {
+                        float v = acc;
+                        acc = 0.0f;
 #pragma unroll
-                for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-                if (lane == 0) {
-                    if (s.epi == ROW_XIELU) v = xielu_f(v, s.c0, s.c1);
-                    s.y[row + warp + ri * NW] = v;
+                        for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+                        const int r = r0 + (c >> lc);
+                        if (lane == 0 && r < end - row) {
+                            if (s.epi == ROW_XIELU) v = xielu_f(v, s.c0, s.c1);
+                            else if (s.epi == ROW_GELU) v = gelu_erf_f(v);
+                            s.y[row + r] = v;
+                        }
+                    }
                 }
             }
         };

@@ -1,30 +1,22 @@
-// C ABI of the Nurinex decoder: a stack of layers in which attention (mixed heads, distance bias, sink) and a
+// The Nurinex decoder: a stack of layers in which attention (mixed heads, distance bias, sink) and a
 // linear-attention recurrence stand side by side on one norm, next to a feed-forward on the same norm. Everything that
 // differs between models of the design is read from the folder's config.json; a layer may use another layer's tensors
 // with a cache and state of its own.
 //
-// Loading, the forward of a portion of tokens (prefill kernels), the decode step (captured in a CUDA graph), generation
-// and scoring. Kernels: bf16_ops.cuh.
+// Configuration, tensors, cache contents, the forward of a portion of tokens (prefill kernels) and the decode step; the
+// rest is decoder.cu's. Kernels: bf16_ops.cuh.
 #include <algorithm>
 #include <cmath>
-#include <cstring>
 #include <memory>
-#include <string>
-#include <vector>
 
-#include "bf16_ops.cuh"
-#include "decode_loop.cuh"
-#include "llama_ops.cuh"
-#include "model_dir.h"
+#include "decoder.h"
 #include "tc_common.cuh"
 
 using namespace fc;
 
 namespace {
 
-constexpr int kMaxPortion = 2048;       // tokens of one forward pass; longer portions are cut
 constexpr int kFfSplits = 4;            // most partial sums of the feed-forward's second product
-constexpr int kMaxSplits = 64;          // attention splits of a decode step
 
 // The entries of config.json for one layer.
 struct LayerCfg {
@@ -35,30 +27,11 @@ struct LayerCfg {
     int ff = 0;                         // 0: no feed-forward
 };
 struct Config {
-    int vocab = 0, width = 0;
     double eps = 0, emb_scale = 1;
     std::vector<LayerCfg> layers;
 };
 
-int want_int(const Json* o, const char* key, const std::string& where, int* out) {
-    const Json* v = o ? o->find(key) : nullptr;
-    if (!v || v->kind != Json::Number || v->num != std::floor(v->num) || v->num < 1 || v->num > 1e9)
-        return fail(FC_E_FORMAT, "config.json: %s.%s must be a positive whole number", where.c_str(), key);
-    *out = (int)v->num;
-    return FC_OK;
-}
-int want_num(const Json* o, const char* key, const std::string& where, double* out) {
-    const Json* v = o ? o->find(key) : nullptr;
-    if (!v || v->kind != Json::Number || !std::isfinite(v->num)) return fail(FC_E_FORMAT, "config.json: %s.%s must be a number", where.c_str(), key);
-    *out = v->num;
-    return FC_OK;
-}
-
 int parse_config(const Json& j, Config* c) {
-    const Json* arch = j.find("architecture");
-    if (!arch || arch->str != "Nurinex") return fail(FC_E_FORMAT, "config.json: architecture is not Nurinex");
-    FC_TRY(want_int(&j, "vocab", "config", &c->vocab));
-    FC_TRY(want_int(&j, "width", "config", &c->width));
     FC_TRY(want_num(j.find("norm"), "eps", "norm", &c->eps));
     if (j.has("embedding") && j.find("embedding")->has("scale")) FC_TRY(want_num(j.find("embedding"), "scale", "embedding", &c->emb_scale));
     const Json* layers = j.find("layers");
@@ -122,33 +95,6 @@ int distance_bucket(int n, int rows, double bias_max) {
     return (int)std::min<double>(rows - 1, half + std::floor(f + 1e-10));
 }
 
-// A tensor of the file with the shape it must have.
-int find_tensor(const ModelDir& md, const std::string& name, std::initializer_list<int64_t> shape, const TensorView** out) {
-    const TensorView* t = md.tensor(name);
-    if (!t) return fail(FC_E_FORMAT, "tensor %s is missing", name.c_str());
-    if (t->shape.size() != shape.size() || !std::equal(shape.begin(), shape.end(), t->shape.begin()))
-        return fail(FC_E_DIM, "tensor %s does not have the shape the configuration asks for", name.c_str());
-    if (t->dtype != "BF16" && t->dtype != "F32") return fail(FC_E_FORMAT, "tensor %s: type %s is not read here", name.c_str(), t->dtype.c_str());
-    *out = t;
-    return FC_OK;
-}
-float bf16_value(uint16_t b) {
-    const uint32_t u = (uint32_t)b << 16;
-    float f;
-    std::memcpy(&f, &u, 4);
-    return f;
-}
-void to_f32(const TensorView& t, std::vector<float>* out) {
-    const size_t n = t.dtype == "F32" ? t.nbytes / 4 : t.nbytes / 2;
-    out->resize(n);
-    if (t.dtype == "F32") { std::memcpy(out->data(), t.data, t.nbytes); return; }
-    for (size_t i = 0; i < n; ++i) {
-        uint16_t b;
-        std::memcpy(&b, t.data + 2 * i, 2);
-        (*out)[i] = bf16_value(b);
-    }
-}
-
 }  // namespace
 
 // The tensors of one layer on the device.
@@ -165,87 +111,57 @@ struct NxWeights {
     CUtensorMap a_planes, a_att, a_ro, a_hid;          // operand maps into the workspace
 };
 
-struct fc_nurinex {
+namespace {
+struct Nurinex : fc_decoder {
     Config cfg;
-    int device = 0, mode = 0, ctx = 0;
-    bool f32 = false;
-    cudaStream_t st = nullptr, side = nullptr;
-    cudaEvent_t fork = nullptr, join = nullptr, ev0 = nullptr, ev1 = nullptr;
-    Arena arena, ws_arena;
-    BMat embed, head;
-    float* final_norm = nullptr;
+    cudaStream_t side = nullptr;
+    cudaEvent_t fork = nullptr, join = nullptr;
     std::vector<std::unique_ptr<NxWeights>> own;       // by layer index; null where another layer's are used
     std::vector<const NxWeights*> run;                 // by layer
     int max_proj = 0, max_att = 0, max_ro = 0, max_hid = 0, max_qm = 0, max_rd = 0, max_qo = 0;
-    int64_t weight_bytes = 0;                          // matrices a decode step reads
-    CUtensorMap m_head, a_head;
     // workspace of a portion of ws_rows tokens
-    int ws_rows = 0, head_chunk = 0;
-    float *x[2] = {}, *proj = nullptr, *outs = nullptr, *decay = nullptr, *wkv_o = nullptr, *logits = nullptr, *h_last = nullptr, *wkv_scratch = nullptr;
-    void *planes = nullptr, *att = nullptr, *ro = nullptr, *hid = nullptr, *qm = nullptr;
-    int *ids_d = nullptr, *rows_d = nullptr, *targets_d = nullptr, *status = nullptr;     // status: [0] timeout, [1] bad id
-    double* lp_d = nullptr;
-    uint8_t* gr_d = nullptr;
-    float last_forward_ms = 0.0f;
-};
+    float *x[2] = {}, *proj = nullptr, *outs = nullptr, *decay = nullptr, *wkv_o = nullptr, *h_last = nullptr, *wkv_scratch = nullptr;
+    void *att = nullptr, *ro = nullptr, *hid = nullptr, *qm = nullptr;
+    MixRows tail;                                      // final norm of the last portion, but for the rows
 
-struct fc_nurinex_cache {
-    fc_nurinex* m = nullptr;
-    int device = 0;
-    Arena arena;
+    ~Nurinex() override {
+        for (cudaEvent_t e : {fork, join}) if (e) cudaEventDestroy(e);
+        if (side) cudaStreamDestroy(side);
+    }
+    int parse(const Json& config) override;
+    int tensors(const ModelDir& md, bool upload) override;
+    int n_planes() const override { return 1 + kMixes; }
+    int workspace(int rows) override;
+    fc_decoder_cache* make_cache() override;
+    int portion(fc_decoder_cache* s, int M, float* layers_out) override;
+    int final_rows(const int* rows, int n) override;
+    int step(fc_decoder_cache* s, bool with_head) override;
+};
+const DecoderDesign design("Nurinex", []() -> fc_decoder* { return new Nurinex(); });
+
+struct NurinexCache : fc_decoder_cache {
     std::vector<void*> kc, vc;                 // per layer: [ctx][kd], [ctx][KV][vp]
     std::vector<float*> wkv;                   // per layer: [rH][rdim][rdim]
     float* shift = nullptr;                    // [2][layers][width]: h of the token before, by the parity of the position
     float* state_block = nullptr;              // recurrence states and `shift`, one block
     size_t state_floats = 0;
-    float *x[2] = {}, *proj = nullptr, *outs = nullptr, *hid = nullptr, *att = nullptr, *ro = nullptr, *logits = nullptr;
+    float *x[2] = {}, *proj = nullptr, *outs = nullptr, *hid = nullptr, *att = nullptr, *ro = nullptr;
     float *part = nullptr, *part_ml = nullptr;
     unsigned int* counter = nullptr;
     int max_splits = 1;
-    int* queue = nullptr;
-    int queue_cap = 0;
-    StepState* state = nullptr;
-    unsigned long long* rng_d = nullptr;
-    int host_pos = 0;
-    cudaGraphExec_t graph[2] = {nullptr, nullptr};
-    int graph_nodes[2] = {0, 0};
-    cudaEvent_t ev0 = nullptr, ev1 = nullptr;
-    float last_decode_ms = 0.0f;
+    int create() override;
+    int clear() override {
+        FC_CUDA(cudaMemsetAsync(state_block, 0, state_floats * 4, m->st));
+        return FC_OK;
+    }
 };
 
-namespace {
-
 // ------------------------------------------------------------------------------------ loading
-struct Part { const TensorView* t; int rows; };
-// Rows of several matrices with the same row length into one padded device matrix; every part starts at its row0.
-int upload_rows(Arena& ar, const std::vector<std::pair<int, Part>>& parts, int rows_total, int K, const char* what, BMat* out, cudaStream_t st) {
-    const int K_pad = pad_to(K, 64), N_pad = pad_to(rows_total, 128);
-    std::vector<uint16_t> buf((size_t)N_pad * K_pad, 0);
-    for (auto& p : parts) {
-        if (p.second.t->dtype != "BF16") return fail(FC_E_FORMAT, "%s: matrices must be stored as BF16", what);
-        for (int r = 0; r < p.second.rows; ++r)
-            std::memcpy(buf.data() + (size_t)(p.first + r) * K_pad, p.second.t->data + (size_t)r * K * 2, (size_t)K * 2);
-    }
-    uint16_t* d = nullptr;
-    FC_TRY(ar.alloc_n(&d, buf.size()));
-    FC_CUDA(cudaMemcpyAsync(d, buf.data(), buf.size() * 2, cudaMemcpyHostToDevice, st));
-    FC_CUDA(cudaStreamSynchronize(st));
-    out->w = d; out->N = rows_total; out->K = K; out->N_pad = N_pad; out->K_pad = K_pad;
-    return FC_OK;
-}
-int upload_vec(Arena& ar, const TensorView& t, float** out, cudaStream_t st) {
-    std::vector<float> v;
-    to_f32(t, &v);
-    FC_TRY(upload_f32(ar, v.data(), v.size(), out, st));
-    FC_CUDA(cudaStreamSynchronize(st));
-    return FC_OK;
-}
-int map_of(const BMat& w, CUtensorMap* m) { return tc::encode_bf16(m, w.w, w.N_pad, w.K_pad, w.K_pad, kGemmBoxRows); }
-
 // Looks up and checks every tensor of a layer; with `w` uploads them.
-int load_layer(const ModelDir& md, const Config& c, int i, fc_nurinex* m, NxWeights* w) {
+int load_layer(const ModelDir& md, int i, Nurinex* m, NxWeights* w) {
+    const Config& c = m->cfg;
     const LayerCfg& L = c.layers[i];
-    const int d = c.width, rd = L.rH * L.rdim;
+    const int d = m->width, rd = L.rH * L.rdim;
     const std::string p = "l" + std::to_string(i) + ".";
     const TensorView *q, *k, *v, *rel, *talk, *sink, *lo, *mu[kMixes], *r, *rk, *rv, *rg, *w1, *w2, *w0, *u, *rn, *ro, *lout, *rout, *n1;
     const TensorView *up = nullptr, *down = nullptr, *act = nullptr;
@@ -358,77 +274,6 @@ int load_layer(const ModelDir& md, const Config& c, int i, fc_nurinex* m, NxWeig
     return FC_OK;
 }
 
-size_t el(const fc_nurinex* m) { return m->f32 ? 4 : 2; }
-
-int ensure_workspace(fc_nurinex* m, int rows) {
-    if (rows <= m->ws_rows) return FC_OK;
-    int R = 128;
-    while (R < rows) R *= 2;
-    FC_CUDA(cudaStreamSynchronize(m->st));
-    m->ws_arena.release();
-    m->ws_rows = 0;
-    const int d = m->cfg.width, dp = m->head.K_pad;
-    const size_t RR = R, e = el(m);
-    Arena& a = m->ws_arena;
-    // padding columns must hold finite values (they meet zero weights): everything starts as zero
-    auto get = [&](void** p, size_t bytes) -> int {
-        FC_TRY(a.alloc(p, bytes));
-        FC_CUDA(cudaMemsetAsync(*p, 0, bytes ? bytes : 16, m->st));
-        return FC_OK;
-    };
-    FC_TRY(get((void**)&m->x[0], RR * d * 4));
-    FC_TRY(get((void**)&m->x[1], RR * d * 4));
-    FC_TRY(get((void**)&m->proj, RR * m->max_proj * 4));
-    FC_TRY(get((void**)&m->outs, (2 + kFfSplits) * RR * d * 4));
-    FC_TRY(get((void**)&m->decay, RR * m->max_rd * 4));
-    FC_TRY(get((void**)&m->wkv_o, RR * m->max_rd * 4));
-    size_t scratch = 0;
-    for (const NxWeights* w : m->run) scratch = std::max(scratch, wkv_scratch_floats(w->rH, w->rdim));
-    FC_TRY(get((void**)&m->wkv_scratch, scratch * 4));
-    FC_TRY(get((void**)&m->h_last, (size_t)m->cfg.layers.size() * d * 4));
-    FC_TRY(get(&m->planes, (1 + kMixes) * RR * dp * e));
-    FC_TRY(get(&m->att, RR * m->max_att * e));
-    FC_TRY(get(&m->ro, RR * m->max_ro * e));
-    FC_TRY(get(&m->hid, RR * m->max_hid * e));
-    FC_TRY(get(&m->qm, RR * m->max_qm * e));
-    m->head_chunk = (int)std::max<size_t>(1, std::min<size_t>(RR, ((size_t)1 << 27) / m->head.N_pad));
-    FC_TRY(get((void**)&m->logits, (size_t)m->head_chunk * m->head.N_pad * 4));
-    FC_TRY(get((void**)&m->ids_d, RR * 4));
-    FC_TRY(get((void**)&m->rows_d, RR * 4));
-    FC_TRY(get((void**)&m->targets_d, RR * 4));
-    FC_TRY(get((void**)&m->lp_d, RR * 8));
-    FC_TRY(get((void**)&m->gr_d, RR));
-    FC_TRY(get((void**)&m->status, 8));
-    if (!m->f32) {
-        for (auto& w : m->own) {
-            if (!w) continue;
-            FC_TRY(tc::encode_bf16(&w->a_planes, m->planes, (1 + kMixes) * RR, dp, dp, kGemmBoxRows));
-            FC_TRY(tc::encode_bf16(&w->a_att, m->att, RR, w->lo.K_pad, w->lo.K_pad, kGemmBoxRows));
-            FC_TRY(tc::encode_bf16(&w->a_ro, m->ro, RR, w->ro.K_pad, w->ro.K_pad, kGemmBoxRows));
-            w->a_hid = w->a_ro;
-            if (w->ff) FC_TRY(tc::encode_bf16(&w->a_hid, m->hid, RR, w->down.K_pad, w->down.K_pad, kGemmBoxRows));
-        }
-        FC_TRY(tc::encode_bf16(&m->a_head, m->planes, RR, dp, dp, kGemmBoxRows));
-    }
-    m->ws_rows = R;
-    return FC_OK;
-}
-
-int check_ids(const fc_nurinex* m, const int32_t* ids, size_t n) {
-    for (size_t i = 0; i < n; ++i)
-        if (ids[i] < 0 || ids[i] >= m->cfg.vocab) return fail(FC_E_DIM, "token %d ≥ vocab_size %d", ids[i], m->cfg.vocab);
-    return FC_OK;
-}
-int check_status(fc_nurinex* m) {
-    int s[2] = {0, 0};
-    FC_CUDA(cudaMemcpyAsync(s, m->status, 8, cudaMemcpyDeviceToHost, m->st));
-    FC_CUDA(cudaStreamSynchronize(m->st));
-    if (s[0] || s[1]) cudaMemsetAsync(m->status, 0, 8, m->st);
-    if (s[0]) return fail(FC_E_TIMEOUT, "a bounded wait inside a tensor-core kernel ran out (status %d)", s[0]);
-    if (s[1]) return fail(s[1], "a token id was rejected on the device");
-    return FC_OK;
-}
-
 // ---------------------------------------------------------------------- a portion of tokens
 // How many partial sums the feed-forward's second product is cut into. The tiles of the three output products go round
 // robin over the SMs, the longest first; with few tiles the feed-forward's long K decides, so the number is the one whose
@@ -458,10 +303,10 @@ SideOutputs outputs_of(const NxWeights& w, const float* outs, size_t stride, int
 }
 
 // One layer's products and mixers for M rows whose norm and mixes are in the planes; positions pos0...
-int layer_forward(fc_nurinex* m, fc_nurinex_cache* s, int l, int M, int pos0, int* n_ff) {
+int layer_forward(Nurinex* m, NurinexCache* s, int l, int M, int pos0, int* n_ff) {
     const NxWeights& w = *m->run[l];
     cudaStream_t st = m->st;
-    const int R = m->ws_rows, dp = m->head.K_pad, d = m->cfg.width, rd = w.rH * w.rdim;
+    const int R = m->ws_rows, dp = m->head.K_pad, d = m->width, rd = w.rH * w.rdim;
     const int ldp = w.proj;
     struct In { int plane, row, n, off; };
     const In in[6] = {{0, 0, w.n_qkv, 0}, {1, w.row_r, rd, w.off_r}, {2, w.row_k, rd, w.off_k}, {3, w.row_v, rd, w.off_v},
@@ -506,8 +351,9 @@ int layer_forward(fc_nurinex* m, fc_nurinex_cache* s, int l, int M, int pos0, in
     }
     FC_CUDA(cudaEventRecord(m->join, m->side));
     FC_TRY(launch_talk_prep(w.t, m->proj, ldp, M, pos0, m->f32 ? 1.0f : kLog2e, m->qm, s->kc[l], s->vc[l], m->f32, st));
-    if (m->f32) FC_TRY(launch_talk_prefill_f32(w.t, (const float*)m->qm, (const float*)s->kc[l], (const float*)s->vc[l], M, pos0, (float*)m->att, w.lo.K_pad, st));
-    else FC_TRY(launch_talk_prefill_tc(w.t, m->qm, s->kc[l], s->vc[l], M, pos0, m->ctx, m->att, w.lo.K_pad, m->status, st));
+    const Flash f = talk_flash(w.t, s->kc[l], s->vc[l], m->ctx);
+    if (m->f32) FC_TRY(launch_flash_f32(f, (const float*)m->qm, M, pos0, (float*)m->att, w.lo.K_pad, st));
+    else FC_TRY(launch_flash_tc(f, m->qm, M, pos0, m->att, w.lo.K_pad, m->status, st));
     FC_CUDA(cudaStreamWaitEvent(st, m->join, 0));
     const size_t stride = (size_t)R * d;
     if (m->f32) {
@@ -540,15 +386,15 @@ int layer_forward(fc_nurinex* m, fc_nurinex_cache* s, int l, int M, int pos0, in
     return launch_gemm_bf16_group(maps, g, M, m->status, st);
 }
 
-// M tokens whose ids are in m->ids_d through all layers, from the cache's position on. Afterwards `tail` runs the rows
-// it wants through the final norm (finish_rows). layers_out (host, may be null): residual stream after every layer.
-struct Tail { MixRows rows; };
-int portion_forward(fc_nurinex* m, fc_nurinex_cache* s, int M, float* layers_out, Tail* tail) {
+}  // namespace
+
+int Nurinex::portion(fc_decoder_cache* sc, int M, float* layers_out) {
+    Nurinex* m = this;
+    auto* s = static_cast<NurinexCache*>(sc);
     const Config& c = m->cfg;
-    const int d = c.width, L = (int)c.layers.size(), R = m->ws_rows, dp = m->head.K_pad, pos0 = s->host_pos;
-    cudaStream_t st = m->st;
+    const int d = width, L = (int)c.layers.size(), R = m->ws_rows, dp = m->head.K_pad, pos0 = s->host_pos;
     MixRows p = {};
-    p.embed.table = m->embed.w; p.embed.vocab = c.vocab; p.embed.ld = m->embed.K_pad; p.embed.scale = (float)c.emb_scale;
+    p.embed.table = m->embed.w; p.embed.vocab = vocab; p.embed.ld = m->embed.K_pad; p.embed.scale = (float)c.emb_scale;
     p.ids = m->ids_d; p.eps = (float)c.eps; p.M = M; p.d = d; p.ld = dp; p.planes = m->planes; p.plane_stride = (size_t)R * dp;
     p.error_flag = m->status + 1;
     int n_ff = 0;
@@ -579,36 +425,23 @@ int portion_forward(fc_nurinex* m, fc_nurinex_cache* s, int M, float* layers_out
         p.x_out = nullptr;
     }
     p.norm_w = m->final_norm;
-    tail->rows = p;
-    s->host_pos += M;
-    return launch_step_set(s->state, s->host_pos, s->host_pos, s->host_pos, st);
+    tail = p;
+    return FC_OK;
 }
 
-// Final norm and head for n rows of the portion (their indices on the device in m->rows_d + at); logits [n][ldl].
-int head_rows(fc_nurinex* m, const Tail& tail, int at, int n, float* logits, int ldl) {
-    MixRows p = tail.rows;
-    p.row_idx = m->rows_d + at;
+int Nurinex::final_rows(const int* rows, int n) {
+    MixRows p = tail;
+    p.row_idx = rows;
     p.M = n;
-    FC_TRY(launch_mix_rows(p, m->f32, m->st));
-    if (m->f32) {
-        GemmF32 q = {};
-        q.a = (const float*)m->planes; q.lda = m->head.K_pad; q.y = logits; q.ldy = ldl;
-        return launch_gemm_bf16w_f32(m->head, 0, m->cfg.vocab, q, n, m->st);
-    }
-    GemmMaps maps;
-    for (int i = 0; i < 3; ++i) { maps.a[i] = m->a_head; maps.b[i] = m->m_head; }
-    GemmGroup g = {};
-    GemmSeg& q = g.seg[g.n_seg++];
-    q.kb = m->head.K_pad / 64; q.n = m->cfg.vocab; q.y = logits; q.ldy = ldl;
-    return launch_gemm_bf16_group(maps, g, n, m->status, m->st);
+    return launch_mix_rows(p, f32, st);
 }
 
 // ------------------------------------------------------------------------------ decode step
-int launch_step(fc_nurinex_cache* s, int with_head) {
-    fc_nurinex* m = s->m;
-    const Config& c = m->cfg;
-    const int d = c.width, L = (int)c.layers.size();
-    cudaStream_t st = m->st;
+int Nurinex::step(fc_decoder_cache* sc, bool with_head) {
+    Nurinex* m = this;
+    auto* s = static_cast<NurinexCache*>(sc);
+    const Config& c = cfg;
+    const int d = width, L = (int)c.layers.size();
     GemvGroup base = {};
     base.eps = (float)c.eps; base.d = d; base.state = s->state; base.ctx = m->ctx;
     base.shift_slot = (size_t)L * d;
@@ -620,7 +453,7 @@ int launch_step(fc_nurinex_cache* s, int with_head) {
         g.mode = 1;
         g.prev = prev;
         if (!l) {
-            g.embed.table = m->embed.w; g.embed.vocab = c.vocab; g.embed.ld = m->embed.K_pad; g.embed.scale = (float)c.emb_scale;
+            g.embed.table = m->embed.w; g.embed.vocab = vocab; g.embed.ld = m->embed.K_pad; g.embed.scale = (float)c.emb_scale;
             g.queue = s->queue;
         }
         g.x_in = s->x[l & 1]; g.x_out = s->x[(l + 1) & 1];
@@ -682,416 +515,111 @@ int launch_step(fc_nurinex_cache* s, int with_head) {
         g.x_in = s->x[L & 1];
         g.norm_w = m->final_norm;
         GemvSeg& q = g.seg[g.n_seg++];
-        q.w = m->head.w; q.n = c.vocab; q.ldw = q.K_pad = m->head.K_pad; q.K = d; q.y = s->logits;
+        q.w = m->head.w; q.n = vocab; q.ldw = q.K_pad = m->head.K_pad; q.K = d; q.y = s->logits;
         FC_TRY(launch_gemv_bf16_group(g, st));
     }
-    return launch_step_advance_pdl(s->state, st);
-}
-
-int run_step(fc_nurinex_cache* s, int with_head) {
-    if (!s->graph[with_head]) {
-        cudaStream_t st = s->m->st;
-        cudaGraph_t g = nullptr;
-        const int64_t before = g_launches;
-        FC_CUDA(cudaStreamBeginCapture(st, cudaStreamCaptureModeThreadLocal));
-        const int rc = launch_step(s, with_head);
-        const cudaError_t e = cudaStreamEndCapture(st, &g);
-        s->graph_nodes[with_head] = (int)(g_launches - before);
-        g_launches = before;
-        if (rc != FC_OK) { if (g) cudaGraphDestroy(g); return rc; }
-        FC_CUDA(e);
-        const cudaError_t ei = cudaGraphInstantiate(&s->graph[with_head], g, 0);
-        cudaGraphDestroy(g);
-        FC_CUDA(ei);
-    }
-    FC_CUDA(cudaGraphLaunch(s->graph[with_head], s->m->st));
-    g_launches += s->graph_nodes[with_head];
     return FC_OK;
 }
 
-int read_state(fc_nurinex_cache* s, StepState* out) {
-    FC_CUDA(cudaMemcpyAsync(out, s->state, sizeof(StepState), cudaMemcpyDeviceToHost, s->m->st));
-    FC_CUDA(cudaStreamSynchronize(s->m->st));
+
+int Nurinex::parse(const Json& j) {
+    FC_TRY(parse_config(j, &cfg));
+    n_layers = (int)cfg.layers.size();
+    for (int i = 0; i < n_layers; ++i) n_own_layers += cfg.layers[i].owner == i;
     return FC_OK;
 }
 
-int check_room(const fc_nurinex_cache* s, int n) {
-    if (n > s->m->ctx - s->host_pos)
-        return fail(FC_E_DIM, "%d more tokens do not fit the %d-token context (position %d)", n, s->m->ctx, s->host_pos);
-    return FC_OK;
-}
-
-// Puts the next `n` ids on the device for a portion (and into the queue, the ids so far).
-int stage_ids(fc_nurinex_cache* s, const int32_t* ids, int n) {
-    FC_CUDA(cudaMemcpyAsync(s->m->ids_d, ids, (size_t)n * 4, cudaMemcpyHostToDevice, s->m->st));
-    FC_CUDA(cudaMemcpyAsync(s->queue + s->host_pos, ids, (size_t)n * 4, cudaMemcpyHostToDevice, s->m->st));
-    return FC_OK;
-}
-
-// One token through the decode step; logits stay in s->logits.
-int feed_one(fc_nurinex_cache* s, int32_t id, int with_head) {
-    FC_CUDA(cudaMemcpyAsync(s->queue + s->host_pos, &id, 4, cudaMemcpyHostToDevice, s->m->st));
-    FC_TRY(launch_step_set(s->state, s->host_pos, s->host_pos, s->host_pos + 1, s->m->st));
-    FC_TRY(run_step(s, with_head));
-    s->host_pos += 1;
-    StepState hs;
-    FC_TRY(read_state(s, &hs));
-    if (hs.error) { s->host_pos -= 1; return fail(hs.error, "the decode step rejected a token or position on the device"); }
-    return FC_OK;
-}
-
-// A prompt of n ids; the logits of its last token in s->logits.
-int feed_prompt(fc_nurinex_cache* s, const int32_t* ids, int n) {
-    fc_nurinex* m = s->m;
-    for (int at = 0; at < n;) {
-        const int M = std::min(kMaxPortion, n - at);
-        if (M == 1) {
-            FC_TRY(feed_one(s, ids[at], at + 1 == n));
-        } else {
-            FC_TRY(ensure_workspace(m, M));
-            FC_TRY(stage_ids(s, ids + at, M));
-            Tail tail;
-            FC_TRY(portion_forward(m, s, M, nullptr, &tail));
-            if (at + M == n) {
-                const int32_t last = M - 1;
-                FC_CUDA(cudaMemcpyAsync(m->rows_d, &last, 4, cudaMemcpyHostToDevice, m->st));
-                FC_TRY(head_rows(m, tail, 0, 1, s->logits, m->head.N_pad));
-            }
-            FC_TRY(check_status(m));
-        }
-        at += M;
-    }
-    return FC_OK;
-}
-
-}  // namespace
-
-extern "C" {
-
-static int probe_dir(const char* dir, ModelDir* md, Config* c) {
-    FC_TRY(md->open(dir));
-    FC_TRY(parse_config(md->config, c));
-    const TensorView* t;
-    FC_TRY(find_tensor(*md, "embed", {c->vocab, c->width}, &t));
-    FC_TRY(find_tensor(*md, "head", {c->vocab, c->width}, &t));
-    FC_TRY(find_tensor(*md, "final.norm", {c->width}, &t));
-    for (size_t i = 0; i < c->layers.size(); ++i)
-        if (c->layers[i].owner == (int)i) FC_TRY(load_layer(*md, *c, (int)i, nullptr, nullptr));
-    return FC_OK;
-}
-static void fill_info(const Config& c, int ctx, int64_t weight_bytes, fc_nurinex_info* out) {
-    out->vocab = c.vocab; out->width = c.width; out->n_layers = (int)c.layers.size(); out->ctx = ctx;
-    out->n_own_layers = 0;
-    for (size_t i = 0; i < c.layers.size(); ++i) out->n_own_layers += c.layers[i].owner == (int)i;
-    out->weight_bytes = weight_bytes;
-}
-
-int fc_nurinex_probe(const char* dir, fc_nurinex_info* out) {
-    if (!dir || !out) return fail(FC_E_ARG, "fc_nurinex_probe: null argument");
-    ModelDir md;
-    Config c;
-    FC_TRY(probe_dir(dir, &md, &c));
-    fill_info(c, 0, 0, out);
-    return FC_OK;
-}
-
-int fc_nurinex_load(const char* dir, int device, int math_mode, int ctx, fc_nurinex** out) {
-    if (!dir || !out) return fail(FC_E_ARG, "fc_nurinex_load: null argument");
-    *out = nullptr;
-    if (math_mode != FC_MATH_FP32 && math_mode != FC_MATH_BF16) return fail(FC_E_ARG, "math_mode %d: this decoder runs in f32 or bf16", math_mode);
-    if (ctx <= 0) return fail(FC_E_SHAPE, "fc_nurinex_load: ctx = %d", ctx);
-    ModelDir md;
-    auto* m = new fc_nurinex();
-    auto build = [&]() -> int {
-        FC_TRY(probe_dir(dir, &md, &m->cfg));
-        FC_TRY(select_device(device));
-        m->device = device; m->mode = math_mode; m->f32 = math_mode == FC_MATH_FP32; m->ctx = ctx;
-        FC_CUDA(cudaStreamCreateWithFlags(&m->st, cudaStreamNonBlocking));
-        FC_CUDA(cudaStreamCreateWithFlags(&m->side, cudaStreamNonBlocking));
-        FC_CUDA(cudaEventCreateWithFlags(&m->fork, cudaEventDisableTiming));
-        FC_CUDA(cudaEventCreateWithFlags(&m->join, cudaEventDisableTiming));
-        FC_CUDA(cudaEventCreate(&m->ev0));
-        FC_CUDA(cudaEventCreate(&m->ev1));
-        const Config& c = m->cfg;
-        const TensorView* t;
-        FC_TRY(find_tensor(md, "embed", {c.vocab, c.width}, &t));
-        FC_TRY(upload_rows(m->arena, {{0, {t, c.vocab}}}, c.vocab, c.width, "embed", &m->embed, m->st));
-        FC_TRY(find_tensor(md, "head", {c.vocab, c.width}, &t));
-        FC_TRY(upload_rows(m->arena, {{0, {t, c.vocab}}}, c.vocab, c.width, "head", &m->head, m->st));
-        FC_TRY(map_of(m->head, &m->m_head));
-        FC_TRY(find_tensor(md, "final.norm", {c.width}, &t));
-        FC_TRY(upload_vec(m->arena, *t, &m->final_norm, m->st));
-        m->own.resize(c.layers.size());
-        for (size_t i = 0; i < c.layers.size(); ++i) {
-            if (c.layers[i].owner != (int)i) continue;
-            m->own[i] = std::make_unique<NxWeights>();
-            FC_TRY(load_layer(md, c, (int)i, m, m->own[i].get()));
-        }
-        for (size_t i = 0; i < c.layers.size(); ++i) m->run.push_back(m->own[c.layers[i].owner].get());
-        m->weight_bytes = (int64_t)m->head.N * m->head.K * 2;
-        for (const NxWeights* w : m->run) {
-            const int rd = w->rH * w->rdim;
-            m->max_proj = std::max(m->max_proj, w->proj);
-            m->max_att = std::max(m->max_att, w->lo.K_pad);
-            m->max_ro = std::max(m->max_ro, w->ro.K_pad);
-            m->max_hid = std::max(m->max_hid, w->ff ? w->down.K_pad : 64);
-            m->max_qm = std::max(m->max_qm, w->t.H * w->t.kd);
-            m->max_qo = std::max(m->max_qo, w->t.H * w->t.vdim);
-            m->max_rd = std::max(m->max_rd, rd);
-            m->weight_bytes += 2LL * c.width * (w->n_qkv + 2 * w->ff + 5 * rd + w->rank + w->t.H * w->t.vdim) + 2LL * rd * w->rank;
-        }
+int Nurinex::tensors(const ModelDir& md, bool upload) {
+    if (!upload) {
+        for (int i = 0; i < n_layers; ++i)
+            if (cfg.layers[i].owner == i) FC_TRY(load_layer(md, i, this, nullptr));
         return FC_OK;
-    };
-    const int rc = build();
-    if (rc != FC_OK) { fc_nurinex_free(m); return rc; }
-    *out = m;
-    return FC_OK;
-}
-
-void fc_nurinex_free(fc_nurinex* m) {
-    if (!m) return;
-    if (m->st) {
-        cudaSetDevice(m->device);
-        cudaStreamSynchronize(m->st);
     }
-    m->ws_arena.release();
-    m->arena.release();
-    for (cudaEvent_t e : {m->fork, m->join, m->ev0, m->ev1}) if (e) cudaEventDestroy(e);
-    if (m->side) cudaStreamDestroy(m->side);
-    if (m->st) cudaStreamDestroy(m->st);
-    delete m;
-}
-
-int fc_nurinex_get_info(const fc_nurinex* m, fc_nurinex_info* out) {
-    if (!m || !out) return fail(FC_E_ARG, "fc_nurinex_get_info: null argument");
-    fill_info(m->cfg, m->ctx, m->weight_bytes, out);
-    return FC_OK;
-}
-float fc_nurinex_last_forward_ms(const fc_nurinex* m) { return m ? m->last_forward_ms : 0.0f; }
-
-int fc_nurinex_cache_create(fc_nurinex* m, fc_nurinex_cache** out) {
-    if (!m || !out) return fail(FC_E_ARG, "fc_nurinex_cache_create: null argument");
-    *out = nullptr;
-    FC_CUDA(cudaSetDevice(m->device));
-    const Config& c = m->cfg;
-    const int L = (int)c.layers.size(), d = c.width;
-    auto* s = new fc_nurinex_cache();
-    s->m = m;
-    s->device = m->device;
-    auto build = [&]() -> int {
-        Arena& a = s->arena;
-        // rows a kernel may touch before they are written must hold finite values: the caches start as zero
-        auto zero = [&](void** p, size_t bytes) -> int {
-            FC_TRY(a.alloc(p, bytes));
-            FC_CUDA(cudaMemsetAsync(*p, 0, bytes, m->st));
-            return FC_OK;
-        };
-        s->state_floats = (size_t)2 * L * d;
-        for (const NxWeights* w : m->run) {
-            void *k = nullptr, *v = nullptr;
-            FC_TRY(zero(&k, (size_t)m->ctx * w->t.kd * el(m)));
-            s->kc.push_back(k);
-            FC_TRY(zero(&v, (size_t)m->ctx * w->t.KV * w->t.vp * el(m)));
-            s->vc.push_back(v);
-            s->state_floats += (size_t)w->rH * w->rdim * w->rdim;
-        }
-        FC_TRY(a.alloc_n(&s->state_block, s->state_floats));
-        s->shift = s->state_block;
-        float* at = s->state_block + (size_t)2 * L * d;
-        for (const NxWeights* w : m->run) { s->wkv.push_back(at); at += (size_t)w->rH * w->rdim * w->rdim; }
-        s->max_splits = std::max(1, std::min(kMaxSplits, (m->ctx + 63) / 64));
-        FC_TRY(a.alloc_n(&s->x[0], (size_t)d));
-        FC_TRY(a.alloc_n(&s->x[1], (size_t)d));
-        FC_TRY(a.alloc_n(&s->proj, (size_t)m->max_proj));
-        FC_TRY(a.alloc_n(&s->outs, (size_t)(2 + kFfSplits) * d));
-        FC_TRY(a.alloc_n(&s->hid, (size_t)m->max_hid));
-        FC_TRY(a.alloc_n(&s->att, (size_t)m->max_qo));
-        FC_TRY(a.alloc_n(&s->ro, (size_t)m->max_rd));
-        FC_TRY(a.alloc_n(&s->logits, (size_t)m->head.N_pad));
-        FC_TRY(a.alloc_n(&s->part, (size_t)s->max_splits * m->max_qo));
-        int heads = 1;
-        for (const NxWeights* w : m->run) heads = std::max(heads, w->t.H);
-        FC_TRY(a.alloc_n(&s->part_ml, (size_t)s->max_splits * heads * 2));
-        FC_TRY(zero((void**)&s->counter, 4));
-        s->queue_cap = m->ctx + 1;
-        FC_TRY(a.alloc_n(&s->queue, (size_t)s->queue_cap));
-        FC_TRY(a.alloc_n(&s->state, 1));
-        FC_TRY(a.alloc_n(&s->rng_d, 1));
-        FC_CUDA(cudaEventCreate(&s->ev0));
-        FC_CUDA(cudaEventCreate(&s->ev1));
-        return fc_nurinex_cache_clear(s);
-    };
-    const int rc = build();
-    if (rc != FC_OK) { fc_nurinex_cache_free(s); return rc; }
-    *out = s;
-    return FC_OK;
-}
-
-void fc_nurinex_cache_free(fc_nurinex_cache* s) {
-    if (!s) return;
-    cudaSetDevice(s->device);
-    cudaDeviceSynchronize();              // the model (and its streams) may already be gone
-    for (auto& g : s->graph) if (g) cudaGraphExecDestroy(g);
-    if (s->ev0) cudaEventDestroy(s->ev0);
-    if (s->ev1) cudaEventDestroy(s->ev1);
-    s->arena.release();
-    delete s;
-}
-
-int fc_nurinex_cache_clear(fc_nurinex_cache* s) {
-    if (!s) return fail(FC_E_ARG, "fc_nurinex_cache_clear: null cache");
-    FC_CUDA(cudaSetDevice(s->device));
-    FC_CUDA(cudaMemsetAsync(s->state_block, 0, s->state_floats * 4, s->m->st));
-    FC_TRY(launch_step_set(s->state, 0, 0, 0, s->m->st));
-    s->host_pos = 0;
-    return FC_OK;
-}
-int fc_nurinex_cache_pos(const fc_nurinex_cache* s) { return s ? s->host_pos : 0; }
-
-int fc_nurinex_feed(fc_nurinex_cache* s, const int32_t* ids, int n, const int32_t* want, int n_want, float* logits) {
-    if (!s || !ids || (n_want > 0 && (!want || !logits))) return fail(FC_E_ARG, "fc_nurinex_feed: null argument");
-    if (n <= 0 || n_want < 0) return fail(FC_E_SHAPE, "fc_nurinex_feed: n = %d, n_want = %d", n, n_want);
-    fc_nurinex* m = s->m;
-    FC_CUDA(cudaSetDevice(m->device));
-    FC_TRY(check_ids(m, ids, (size_t)n));
-    FC_TRY(check_room(s, n));
-    for (int k = 0; k < n_want; ++k)
-        if (want[k] < 0 || want[k] >= n) return fail(FC_E_DIM, "wanted place %d is not among the %d tokens", want[k], n);
-    const int V = m->cfg.vocab, ldl = m->head.N_pad;
-    m->last_forward_ms = 0.0f;
-    std::vector<int32_t> rows, dst;
-    for (int at = 0; at < n;) {
-        const int M = std::min(kMaxPortion, n - at);
-        rows.clear(); dst.clear();
-        for (int k = 0; k < n_want; ++k)
-            if (want[k] >= at && want[k] < at + M) { rows.push_back(want[k] - at); dst.push_back(k); }
-        if (M == 1) {
-            FC_TRY(feed_one(s, ids[at], !rows.empty()));
-            for (int32_t k : dst) FC_CUDA(cudaMemcpyAsync(logits + (size_t)k * V, s->logits, (size_t)V * 4, cudaMemcpyDeviceToHost, m->st));
-            FC_CUDA(cudaStreamSynchronize(m->st));
-        } else {
-            FC_TRY(ensure_workspace(m, M));
-            FC_TRY(stage_ids(s, ids + at, M));
-            FC_CUDA(cudaEventRecord(m->ev0, m->st));
-            Tail tail;
-            FC_TRY(portion_forward(m, s, M, nullptr, &tail));
-            for (size_t k = 0; k < rows.size();) {
-                const int c = (int)std::min<size_t>(std::min(m->head_chunk, m->ws_rows), rows.size() - k);
-                FC_CUDA(cudaMemcpyAsync(m->rows_d, rows.data() + k, (size_t)c * 4, cudaMemcpyHostToDevice, m->st));
-                FC_TRY(head_rows(m, tail, 0, c, m->logits, ldl));
-                for (int i = 0; i < c;) {                  // runs of neighbouring places in one copy
-                    int e = i + 1;
-                    while (e < c && dst[k + e] == dst[k + e - 1] + 1) ++e;
-                    FC_CUDA(cudaMemcpy2DAsync(logits + (size_t)dst[k + i] * V, (size_t)V * 4, m->logits + (size_t)i * ldl, (size_t)ldl * 4, (size_t)V * 4,
-                                              e - i, cudaMemcpyDeviceToHost, m->st));
-                    i = e;
-                }
-                k += c;
-            }
-            FC_CUDA(cudaEventRecord(m->ev1, m->st));
-            FC_TRY(check_status(m));
-            float ms = 0.0f;
-            FC_CUDA(cudaEventElapsedTime(&ms, m->ev0, m->ev1));
-            m->last_forward_ms += ms;
-        }
-        at += M;
+    FC_CUDA(cudaStreamCreateWithFlags(&side, cudaStreamNonBlocking));
+    FC_CUDA(cudaEventCreateWithFlags(&fork, cudaEventDisableTiming));
+    FC_CUDA(cudaEventCreateWithFlags(&join, cudaEventDisableTiming));
+    own.resize(n_layers);
+    for (int i = 0; i < n_layers; ++i) {
+        if (cfg.layers[i].owner != i) continue;
+        own[i] = std::make_unique<NxWeights>();
+        FC_TRY(load_layer(md, i, this, own[i].get()));
+    }
+    for (int i = 0; i < n_layers; ++i) run.push_back(own[cfg.layers[i].owner].get());
+    for (const NxWeights* w : run) {
+        const int rd = w->rH * w->rdim;
+        max_proj = std::max(max_proj, w->proj);
+        max_att = std::max(max_att, w->lo.K_pad);
+        max_ro = std::max(max_ro, w->ro.K_pad);
+        max_hid = std::max(max_hid, w->ff ? w->down.K_pad : 64);
+        max_qm = std::max(max_qm, w->t.H * w->t.kd);
+        max_qo = std::max(max_qo, w->t.H * w->t.vdim);
+        max_rd = std::max(max_rd, rd);
+        weight_bytes += 2LL * width * (w->n_qkv + 2 * w->ff + 5 * rd + w->rank + w->t.H * w->t.vdim) + 2LL * rd * w->rank;
     }
     return FC_OK;
 }
 
-int fc_nurinex_feed_layers(fc_nurinex_cache* s, const int32_t* ids, int n, float* layers) {
-    if (!s || !ids || !layers) return fail(FC_E_ARG, "fc_nurinex_feed_layers: null argument");
-    if (n <= 0 || n > kMaxPortion) return fail(FC_E_SHAPE, "fc_nurinex_feed_layers: n = %d, at most %d", n, kMaxPortion);
-    fc_nurinex* m = s->m;
-    FC_CUDA(cudaSetDevice(m->device));
-    FC_TRY(check_ids(m, ids, (size_t)n));
-    FC_TRY(check_room(s, n));
-    FC_TRY(ensure_workspace(m, n));
-    FC_TRY(stage_ids(s, ids, n));
-    Tail tail;
-    FC_TRY(portion_forward(m, s, n, layers, &tail));
-    return check_status(m);
-}
-
-int fc_nurinex_score(fc_nurinex_cache* s, const int32_t* ids, int n, int from, fc_score* score, float* lp, uint8_t* is_greedy) {
-    if (!s || !ids || !score) return fail(FC_E_ARG, "fc_nurinex_score: null argument");
-    if (n < 0 || from < 0) return fail(FC_E_SHAPE, "fc_nurinex_score: n = %d, from = %d", n, from);
-    fc_nurinex* m = s->m;
-    FC_CUDA(cudaSetDevice(m->device));
-    FC_TRY(check_ids(m, ids, (size_t)n));
-    score->logprob = 0.0; score->n_tokens = 0; score->greedy = 1;
-    if (lp) std::fill(lp, lp + std::max(n - 1, 0), 0.0f);
-    if (is_greedy) std::fill(is_greedy, is_greedy + std::max(n - 1, 0), (uint8_t)0);
-    const int first = std::max(from, 1) - 1, feed = n - 1;       // row t predicts id t + 1
-    if (first >= feed) return FC_OK;
-    FC_TRY(fc_nurinex_cache_clear(s));
-    FC_TRY(check_room(s, feed));
-    m->last_forward_ms = 0.0f;
-    std::vector<int32_t> rows, targets;
-    std::vector<double> lps;
-    std::vector<uint8_t> grs;
-    for (int at = 0; at < feed;) {
-        const int M = std::min(kMaxPortion, feed - at);
-        FC_TRY(ensure_workspace(m, M));
-        FC_TRY(stage_ids(s, ids + at, M));
-        FC_CUDA(cudaEventRecord(m->ev0, m->st));
-        Tail tail;
-        FC_TRY(portion_forward(m, s, M, nullptr, &tail));
-        rows.clear(); targets.clear();
-        for (int t = std::max(first, at); t < at + M; ++t) { rows.push_back(t - at); targets.push_back(ids[t + 1]); }
-        const int R = (int)rows.size();
-        if (R) {
-            FC_CUDA(cudaMemcpyAsync(m->rows_d, rows.data(), (size_t)R * 4, cudaMemcpyHostToDevice, m->st));
-            FC_CUDA(cudaMemcpyAsync(m->targets_d, targets.data(), (size_t)R * 4, cudaMemcpyHostToDevice, m->st));
-            for (int k = 0; k < R; k += m->head_chunk) {
-                const int c = std::min(m->head_chunk, R - k);
-                FC_TRY(head_rows(m, tail, k, c, m->logits, m->head.N_pad));
-                FC_TRY(launch_llama_score_rows(m->logits, m->head.N_pad, m->cfg.vocab, m->targets_d + k, c, m->lp_d + k, m->gr_d + k, m->st));
-            }
-        }
-        FC_CUDA(cudaEventRecord(m->ev1, m->st));
-        lps.resize(R); grs.resize(R);
-        if (R) {
-            FC_CUDA(cudaMemcpyAsync(lps.data(), m->lp_d, (size_t)R * 8, cudaMemcpyDeviceToHost, m->st));
-            FC_CUDA(cudaMemcpyAsync(grs.data(), m->gr_d, (size_t)R, cudaMemcpyDeviceToHost, m->st));
-        }
-        FC_TRY(check_status(m));
-        float ms = 0.0f;
-        FC_CUDA(cudaEventElapsedTime(&ms, m->ev0, m->ev1));
-        m->last_forward_ms += ms;
-        for (int i = 0; i < R; ++i) {
-            const int t = at + rows[i];
-            score->logprob += lps[i];
-            score->n_tokens += 1;
-            if (!grs[i]) score->greedy = 0;
-            if (lp) lp[t] = (float)lps[i];
-            if (is_greedy) is_greedy[t] = grs[i];
-        }
-        at += M;
+int Nurinex::workspace(int rows) {
+    const int d = width, dp = head.K_pad;
+    const size_t RR = rows, e = el();
+    Arena& a = ws_arena;
+    FC_TRY(zeroed_n(a, &x[0], RR * d));
+    FC_TRY(zeroed_n(a, &x[1], RR * d));
+    FC_TRY(zeroed_n(a, &proj, RR * max_proj));
+    FC_TRY(zeroed_n(a, &outs, (2 + kFfSplits) * RR * d));
+    FC_TRY(zeroed_n(a, &decay, RR * max_rd));
+    FC_TRY(zeroed_n(a, &wkv_o, RR * max_rd));
+    size_t scratch = 0;
+    for (const NxWeights* w : run) scratch = std::max(scratch, wkv_scratch_floats(w->rH, w->rdim));
+    FC_TRY(zeroed_n(a, &wkv_scratch, scratch));
+    FC_TRY(zeroed_n(a, &h_last, (size_t)n_layers * d));
+    FC_TRY(zeroed(a, &att, RR * max_att * e));
+    FC_TRY(zeroed(a, &ro, RR * max_ro * e));
+    FC_TRY(zeroed(a, &hid, RR * max_hid * e));
+    FC_TRY(zeroed(a, &qm, RR * max_qm * e));
+    if (f32) return FC_OK;
+    for (auto& w : own) {
+        if (!w) continue;
+        FC_TRY(tc::encode_bf16(&w->a_planes, planes, (1 + kMixes) * RR, dp, dp, kGemmBoxRows));
+        FC_TRY(tc::encode_bf16(&w->a_att, att, RR, w->lo.K_pad, w->lo.K_pad, kGemmBoxRows));
+        FC_TRY(tc::encode_bf16(&w->a_ro, ro, RR, w->ro.K_pad, w->ro.K_pad, kGemmBoxRows));
+        w->a_hid = w->a_ro;
+        if (w->ff) FC_TRY(tc::encode_bf16(&w->a_hid, hid, RR, w->down.K_pad, w->down.K_pad, kGemmBoxRows));
     }
     return FC_OK;
 }
 
-int fc_nurinex_generate(fc_nurinex_cache* s, const int32_t* prompt, int n, int max_new, const fc_sampling* params, const int32_t* stops,
-                        int n_stops, uint64_t* rng_state, const volatile int32_t* cancel, int32_t* out, int* n_out) {
-    if (!s || !prompt || !params || !rng_state || !n_out || (max_new > 0 && !out) || (n_stops > 0 && !stops))
-        return fail(FC_E_ARG, "fc_nurinex_generate: null argument");
-    *n_out = 0;
-    if (n <= 0) return fail(FC_E_DIM, "prompt must be non-empty");
-    if (max_new < 0 || n_stops < 0) return fail(FC_E_SHAPE, "fc_nurinex_generate: max_new = %d, n_stops = %d", max_new, n_stops);
-    fc_nurinex* m = s->m;
-    FC_CUDA(cudaSetDevice(m->device));
-    FC_TRY(check_ids(m, prompt, (size_t)n));
-    if (n >= m->ctx) return fail(FC_E_DIM, "prompt of %d tokens does not fit the %d-token context", n, m->ctx);
-    max_new = std::min(max_new, m->ctx - n);
-    if (cancel && *cancel) return FC_OK;
-    FC_TRY(fc_nurinex_cache_clear(s));
-    FC_CUDA(cudaMemcpyAsync(s->rng_d, rng_state, 8, cudaMemcpyHostToDevice, m->st));
-    FC_TRY(feed_prompt(s, prompt, n));
-    const GenCtx g = {m->st, s->logits, m->cfg.vocab, s->queue, s->queue_cap, s->state, s->rng_d, s->ev0, s->ev1, &s->host_pos, &s->last_decode_ms};
-    return generate_tokens(g, n, max_new, params, stops, n_stops, rng_state, cancel, out, n_out, [&] { return run_step(s, 1); },
-                           [&](StepState* hs) { return read_state(s, hs); });
-}
-float fc_nurinex_last_decode_ms(const fc_nurinex_cache* s) { return s ? s->last_decode_ms : 0.0f; }
+fc_decoder_cache* Nurinex::make_cache() { return new NurinexCache(); }
 
-}  // extern "C"
+int NurinexCache::create() {
+    auto* n = static_cast<Nurinex*>(m);
+    Arena& a = arena;
+    const int L = n->n_layers, d = n->width;
+    // rows a kernel may touch before they are written must hold finite values: the caches start as zero
+    state_floats = (size_t)2 * L * d;
+    for (const NxWeights* w : n->run) {
+        void *k = nullptr, *v = nullptr;
+        FC_TRY(n->zeroed(a, &k, (size_t)n->ctx * w->t.kd * n->el()));
+        kc.push_back(k);
+        FC_TRY(n->zeroed(a, &v, (size_t)n->ctx * w->t.KV * w->t.vp * n->el()));
+        vc.push_back(v);
+        state_floats += (size_t)w->rH * w->rdim * w->rdim;
+    }
+    FC_TRY(a.alloc_n(&state_block, state_floats));
+    shift = state_block;
+    float* at = state_block + (size_t)2 * L * d;
+    for (const NxWeights* w : n->run) { wkv.push_back(at); at += (size_t)w->rH * w->rdim * w->rdim; }
+    max_splits = std::max(1, std::min(kMaxSplits, (n->ctx + 63) / 64));
+    FC_TRY(a.alloc_n(&x[0], (size_t)d));
+    FC_TRY(a.alloc_n(&x[1], (size_t)d));
+    FC_TRY(a.alloc_n(&proj, (size_t)n->max_proj));
+    FC_TRY(a.alloc_n(&outs, (size_t)(2 + kFfSplits) * d));
+    FC_TRY(a.alloc_n(&hid, (size_t)n->max_hid));
+    FC_TRY(a.alloc_n(&att, (size_t)n->max_qo));
+    FC_TRY(a.alloc_n(&ro, (size_t)n->max_rd));
+    FC_TRY(a.alloc_n(&part, (size_t)max_splits * n->max_qo));
+    int heads = 1;
+    for (const NxWeights* w : n->run) heads = std::max(heads, w->t.H);
+    FC_TRY(a.alloc_n(&part_ml, (size_t)max_splits * heads * 2));
+    return n->zeroed_n(a, &counter, 1);
+}

@@ -5,9 +5,8 @@
 // q'_h = [sum_{g in group 0} talk[h][g] q_g | sum_{g in group 1} ... ], plus a per-head table of the distance whose
 // heads are mixed once at load. So after `talk_prep_kernel` this is ordinary attention with one wide shared key head.
 //
-//   talk_prep_kernel          one CTA per token: mixed queries out, key row and normed value row into the cache
-//   talk_prefill_f32_kernel   16 query rows x one head per CTA, CUDA cores, online softmax over key tiles of 32
-// Bound: prep HBM / L2; prefill fp32 FMA (the tcgen05 form is talk_attn_tc.cu).
+//   talk_prep_kernel   one CTA per token: mixed queries out, key row and normed value row into the cache
+// The attention itself: flash_tc.cu, flash_f32.cu. Bound: HBM / L2.
 #include <algorithm>
 
 #include "bf16_ops.cuh"
@@ -115,97 +114,14 @@ int launch_talk_prep(const TalkAttn& t, const float* proj, int ldp, int M, int p
     return f32 ? prep<float>(t, proj, ldp, M, pos0, factor, qm, kc, vc, st) : prep<uint16_t>(t, proj, ldp, M, pos0, factor, qm, kc, vc, st);
 }
 
-namespace {
-constexpr int QR = 16, KT = 32, KC = 64, PNT = 128, VCOLS = 2;     // value columns per thread: heads of at most 256
-}
-__global__ void __launch_bounds__(PNT) talk_prefill_f32_kernel(const TalkAttn t, const float* __restrict__ qm, const float* __restrict__ kc,
-                                                               const float* __restrict__ vc, int M, int pos0, float* __restrict__ out, int ldo) {
-    __shared__ float Qs[QR][KC + 1], Ks[KT][KC + 1], P[QR][KT + 1];
-    __shared__ float corr_s[QR], l_s[QR];
-    const int tid = threadIdx.x, h = blockIdx.y, row0 = (gridDim.x - 1 - blockIdx.x) * QR, kv = h / (t.H / t.KV);
-    const int rows = min(QR, M - row0), last = pos0 + row0 + rows - 1;
-    const int qi = tid >> 3, k8 = tid & 7, qpos = pos0 + row0 + qi;
-    const float* bias = t.bias + (size_t)h * (t.far + 1);
-    float m = t.sink[h], l = 1.0f;                 // the sink: weight exp(sink - m) = 1 so far, no key, no value
-    float acc[VCOLS][QR];
-#pragma unroll
-    for (int c = 0; c < VCOLS; ++c)
-#pragma unroll
-        for (int r = 0; r < QR; ++r) acc[c][r] = 0.0f;
-    for (int k0 = 0; k0 <= last; k0 += KT) {
-        float s[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-        for (int e0 = 0; e0 < t.kd; e0 += KC) {
-            __syncthreads();
-            for (int i = tid; i < QR * KC; i += PNT) {
-                const int r = i / KC, e = i - r * KC;
-                Qs[r][e] = r < rows && e0 + e < t.kd ? qm[((size_t)(row0 + r) * t.H + h) * t.kd + e0 + e] : 0.0f;
-            }
-            for (int i = tid; i < KT * KC; i += PNT) {
-                const int r = i / KC, e = i - r * KC;
-                Ks[r][e] = k0 + r <= last && e0 + e < t.kd ? kc[(size_t)(k0 + r) * t.kd + e0 + e] : 0.0f;
-            }
-            __syncthreads();
-#pragma unroll 8
-            for (int e = 0; e < KC; ++e) {
-                const float q = Qs[qi][e];
-#pragma unroll
-                for (int x = 0; x < 4; ++x) s[x] = fmaf(q, Ks[k8 + 8 * x][e], s[x]);
-            }
-        }
-        float mx = -INFINITY;
-#pragma unroll
-        for (int x = 0; x < 4; ++x) {
-            const int n = qpos - (k0 + k8 + 8 * x);
-            s[x] = n >= 0 ? s[x] + bias[min(n, t.far)] : -INFINITY;
-            mx = fmaxf(mx, s[x]);
-        }
-#pragma unroll
-        for (int o = 4; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-        const float mn = fmaxf(m, mx), corr = expf(m - mn);
-        float ps = 0.0f;
-#pragma unroll
-        for (int x = 0; x < 4; ++x) {
-            const float p = expf(s[x] - mn);
-            P[qi][k8 + 8 * x] = p;
-            ps += p;
-        }
-#pragma unroll
-        for (int o = 4; o > 0; o >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
-        l = fmaf(l, corr, ps);
-        m = mn;
-        if (k8 == 0) { corr_s[qi] = corr; l_s[qi] = l; }
-        __syncthreads();
-        const int nk = min(KT, last - k0 + 1);
-#pragma unroll
-        for (int c = 0; c < VCOLS; ++c) {
-            const int col = tid + c * PNT;
-            if (col >= t.vdim) continue;
-#pragma unroll
-            for (int r = 0; r < QR; ++r) acc[c][r] *= corr_s[r];
-            const float* v = vc + ((size_t)k0 * t.KV + kv) * t.vp + col;
-            for (int j = 0; j < nk; ++j) {
-                const float x = v[(size_t)j * t.KV * t.vp];
-#pragma unroll
-                for (int r = 0; r < QR; ++r) acc[c][r] = fmaf(P[r][j], x, acc[c][r]);
-            }
-        }
-    }
-    __syncthreads();
-#pragma unroll
-    for (int c = 0; c < VCOLS; ++c) {
-        const int col = tid + c * PNT;
-        if (col >= t.vdim) continue;
-#pragma unroll
-        for (int r = 0; r < QR; ++r)
-            if (r < rows) out[(size_t)(row0 + r) * ldo + (size_t)h * t.vdim + col] = acc[c][r] / l_s[r];
-    }
-}
-int launch_talk_prefill_f32(const TalkAttn& t, const float* qm, const float* kc, const float* vc, int M, int pos0, float* out, int ldo,
-                            cudaStream_t st) {
-    if (t.vdim > VCOLS * PNT) return fail(FC_E_SHAPE, "value heads of %d: at most %d", t.vdim, VCOLS * PNT);
-    talk_prefill_f32_kernel<<<dim3((M + QR - 1) / QR, t.H), PNT, 0, st>>>(t, qm, kc, vc, M, pos0, out, ldo);
-    FC_LAUNCHED();
-    return FC_OK;
+// What the attention of a portion reads: one wide key all heads share, values by key/value head, the bias, the sink.
+Flash talk_flash(const TalkAttn& t, const void* kc, const void* vc, int ctx) {
+    Flash f;
+    f.H = t.H; f.KV = t.KV; f.vdim = t.vdim;
+    f.k0.p = kc; f.k0.rows = ctx; f.k0.ld = t.kd; f.k0.width = t.kd;
+    f.v.p = vc; f.v.rows = ctx; f.v.ld = t.KV * t.vp; f.v.head_stride = t.vp; f.v.width = t.vp;
+    f.bias = t.bias; f.far = t.far; f.sink = t.sink; f.has_sink = true;
+    return f;
 }
 
 }  // namespace fc

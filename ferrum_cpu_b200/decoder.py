@@ -1,7 +1,7 @@
-"""Python face of the Nurinex part of the C ABI. Token ids in, logits / scores / token ids out; every
-method is a thin ctypes call into the library.
+"""Python face of the decoders whose model is a folder (fc_decoder*): one class for every design. Token ids in,
+logits / scores / token ids out; every method is a thin ctypes call into the library.
 
-CudaNurinex has the calls of CudaLlama (caches of one's own) and, on a cache it keeps itself, the three
+CudaDecoder has the calls of CudaLlama (caches of one's own) and, on a cache it keeps itself, the three
 calls CudaBackend makes of a model: generate_tokens, generate_sampled and score_requests.
 """
 import ctypes as C
@@ -18,23 +18,23 @@ DEFAULT_CTX = 4096
 
 def probe(path):
     """Sizes of a model folder; validates configuration and tensors without a GPU."""
-    info = _lib.FcNurinexInfo()
-    check(_lib.lib().fc_nurinex_probe(str(path).encode(), C.byref(info)))
+    info = _lib.FcDecoderInfo()
+    check(_lib.lib().fc_decoder_probe(str(path).encode(), C.byref(info)))
     return info
 
 
-class NurinexCache:
-    """What one sequence holds: key / value rows, recurrence states, token-shift rows and the position."""
+class DecoderCache:
+    """What one sequence holds: cached rows and states of every layer, and the position."""
 
     def __init__(self, model):
         self.model = model
         self._h = C.c_void_p()
-        check(_lib.lib().fc_nurinex_cache_create(model._h, C.byref(self._h)))
+        check(_lib.lib().fc_decoder_cache_create(model._h, C.byref(self._h)))
         model._caches.append(weakref.ref(self))
 
     def close(self):
         if self._h:
-            _lib.lib().fc_nurinex_cache_free(self._h)
+            _lib.lib().fc_decoder_cache_free(self._h)
             self._h = C.c_void_p()
 
     def __del__(self):
@@ -44,26 +44,37 @@ class NurinexCache:
             pass
 
     def clear(self):
-        check(_lib.lib().fc_nurinex_cache_clear(self._h))
+        check(_lib.lib().fc_decoder_cache_clear(self._h))
 
     def pos(self):
-        return _lib.lib().fc_nurinex_cache_pos(self._h)
+        return _lib.lib().fc_decoder_cache_pos(self._h)
 
     @property
     def last_decode_ms(self):
-        return _lib.lib().fc_nurinex_last_decode_ms(self._h)
+        return _lib.lib().fc_decoder_last_decode_ms(self._h)
 
 
-class CudaNurinex:
-    """A Nurinex model folder on one GPU. math_mode: FC_MATH_BF16 or FC_MATH_FP32; ctx: positions a cache holds."""
+def dir_architecture(path):
+    """Architecture of a model folder, read by the library."""
+    buf = C.create_string_buffer(256)
+    check(_lib.lib().fc_model_dir_architecture(str(path).encode(), buf, len(buf)))
+    return buf.value.decode()
+
+
+class CudaDecoder:
+    """A model folder on one GPU. math_mode: FC_MATH_BF16 or FC_MATH_FP32; ctx: positions a cache holds."""
+
+    architecture = None        # a design's class takes folders of that design only
 
     def __init__(self, path, device=0, math_mode=_lib.FC_MATH_BF16, ctx=DEFAULT_CTX):
         self._h = C.c_void_p()
         self._caches = []
         self._own = None
-        check(_lib.lib().fc_nurinex_load(str(path).encode(), device, math_mode, ctx, C.byref(self._h)))
-        self.info = _lib.FcNurinexInfo()
-        check(_lib.lib().fc_nurinex_get_info(self._h, C.byref(self.info)))
+        if self.architecture is not None and dir_architecture(path) != self.architecture:
+            raise FerrumCudaError(_lib.FC_E_FORMAT, f"{path} holds no {self.architecture} model")
+        check(_lib.lib().fc_decoder_load(str(path).encode(), device, math_mode, ctx, C.byref(self._h)))
+        self.info = _lib.FcDecoderInfo()
+        check(_lib.lib().fc_decoder_get_info(self._h, C.byref(self.info)))
 
     def close(self):
         self._own = None
@@ -73,7 +84,7 @@ class CudaNurinex:
                 cache.close()
         self._caches = []
         if self._h:
-            _lib.lib().fc_nurinex_free(self._h)
+            _lib.lib().fc_decoder_free(self._h)
             self._h = C.c_void_p()
 
     def __del__(self):
@@ -83,7 +94,7 @@ class CudaNurinex:
             pass
 
     def new_cache(self):
-        return NurinexCache(self)
+        return DecoderCache(self)
 
     def _cache(self):
         if self._own is None:
@@ -95,7 +106,7 @@ class CudaNurinex:
         """The next tokens of the cache's sequence, any number of them; logits [len(want)][vocab] of the wanted places."""
         ids, want = _ids(ids), _ids(want)
         out = np.empty((want.size, self.info.vocab), dtype=np.float32)
-        check(_lib.lib().fc_nurinex_feed(cache._h, _ptr(ids), ids.size, _ptr(want) if want.size else None, want.size,
+        check(_lib.lib().fc_decoder_feed(cache._h, _ptr(ids), ids.size, _ptr(want) if want.size else None, want.size,
                                          _ptr(out) if want.size else None))
         return out
 
@@ -103,7 +114,7 @@ class CudaNurinex:
         """One portion; the residual stream after every layer [layers][n][width]."""
         ids = _ids(ids)
         out = np.empty((self.info.n_layers, ids.size, self.info.width), dtype=np.float32)
-        check(_lib.lib().fc_nurinex_feed_layers(cache._h, _ptr(ids), ids.size, _ptr(out)))
+        check(_lib.lib().fc_decoder_feed_layers(cache._h, _ptr(ids), ids.size, _ptr(out)))
         return out
 
     def forward_tokens(self, ids):
@@ -118,7 +129,7 @@ class CudaNurinex:
 
     @property
     def last_forward_ms(self):
-        return _lib.lib().fc_nurinex_last_forward_ms(self._h)
+        return _lib.lib().fc_decoder_last_forward_ms(self._h)
 
     # ---- scoring ---------------------------------------------------------------------------
     def score_from(self, ids, start, per_token=False):
@@ -127,7 +138,7 @@ class CudaNurinex:
         sc = _lib.FcScore()
         lp = np.zeros(max(ids.size - 1, 1), dtype=np.float32)
         gr = np.zeros(max(ids.size - 1, 1), dtype=np.uint8)
-        check(_lib.lib().fc_nurinex_score(self._cache()._h, _ptr(ids), ids.size, start, C.byref(sc), _ptr(lp), _ptr(gr)))
+        check(_lib.lib().fc_decoder_score(self._cache()._h, _ptr(ids), ids.size, start, C.byref(sc), _ptr(lp), _ptr(gr)))
         score = Score(sc.logprob, sc.n_tokens, bool(sc.greedy))
         return (score, lp[:max(ids.size - 1, 0)], gr[:max(ids.size - 1, 0)].astype(bool)) if per_token else score
 
@@ -142,7 +153,7 @@ class CudaNurinex:
         out = np.zeros(max(max_new, 1), dtype=np.int32)
         n_out = C.c_int(0)
         state = C.c_uint64(rng_state)
-        rc = _lib.lib().fc_nurinex_generate(cache._h, _ptr(prompt), prompt.size, max_new, C.byref(params),
+        rc = _lib.lib().fc_decoder_generate(cache._h, _ptr(prompt), prompt.size, max_new, C.byref(params),
                                             _ptr(stops_a) if stops_a.size else None, stops_a.size, C.byref(state), cancel_p,
                                             _ptr(out), C.byref(n_out))
         return rc, out[:n_out.value].copy(), state.value
@@ -170,4 +181,14 @@ class CudaNurinex:
         return out, bool(cancel is not None and int(cancel[0]))
 
 
-__all__ = ["CudaNurinex", "NurinexCache", "probe", "FerrumCudaError"]
+class CudaNurinex(CudaDecoder):
+    """Layers of attention with mixed heads, a linear-attention recurrence and a dense feed-forward side by side."""
+    architecture = "Nurinex"
+
+
+class CudaZogevik(CudaDecoder):
+    """Layers of windowed attention (latent, or grouped-query with caches that layers may share) and routed experts."""
+    architecture = "Zogevik"
+
+
+__all__ = ["CudaDecoder", "CudaNurinex", "CudaZogevik", "DecoderCache", "dir_architecture", "probe", "FerrumCudaError"]

@@ -3,19 +3,22 @@
 A folder (config.json + model.safetensors) names its architecture in the configuration; a file is a GGUF,
 whose header says gpt2, llama or qwen2.
 """
-import ctypes as C
 import os
 
 from . import _lib
-from ._lib import FerrumCudaError, check
+from ._lib import FerrumCudaError
 
 DTYPES = {"float32": _lib.FC_MATH_FP32, "bfloat16": _lib.FC_MATH_BF16}
 F32_MODES = (_lib.FC_MATH_FP32, _lib.FC_MATH_BF16X3)
 
 
-def _nurinex(path, device, math_mode, ctx):
-    from .nurinex import DEFAULT_CTX, CudaNurinex
-    return CudaNurinex(path, device=device, math_mode=_lib.FC_MATH_BF16 if math_mode is None else math_mode, ctx=ctx or DEFAULT_CTX)
+def _folder(name):
+    """Loader of the design with that class in decoder.py."""
+    def load_folder(path, device, math_mode, ctx):
+        from . import decoder
+        return getattr(decoder, name)(path, device=device, math_mode=_lib.FC_MATH_BF16 if math_mode is None else math_mode,
+                                      ctx=ctx or decoder.DEFAULT_CTX)
+    return load_folder
 
 
 def _gguf_mode(math_mode):
@@ -40,19 +43,14 @@ ARCHITECTURES = {
     "gpt2": (_gpt2, None),
     "llama": (_llama, None),
     "qwen2": (_llama, None),
-    "Nurinex": (_nurinex, "nurinex"),
+    "Nurinex": (_folder("CudaNurinex"), "nurinex"),
+    "Zogevik": (_folder("CudaZogevik"), "zogevik"),
 }
-
-
-def dir_architecture(path):
-    """Architecture of a model folder, read by the library."""
-    buf = C.create_string_buffer(256)
-    check(_lib.lib().fc_model_dir_architecture(str(path).encode(), buf, len(buf)))
-    return buf.value.decode()
 
 
 def architecture(path):
     if os.path.isdir(path):
+        from .decoder import dir_architecture
         return dir_architecture(path)
     from . import engine, llama
     try:

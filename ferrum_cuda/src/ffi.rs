@@ -96,11 +96,11 @@ pub enum fc_ggml_weight {}
 pub enum fc_llama {}
 pub enum fc_llama_cache {}
 pub enum fc_rowq {}
-pub enum fc_nurinex {}
-pub enum fc_nurinex_cache {}
+pub enum fc_decoder {}
+pub enum fc_decoder_cache {}
 #[repr(C)]
 #[derive(Clone, Copy, Default)]
-pub struct fc_nurinex_info { pub vocab: i32, pub width: i32, pub n_layers: i32, pub n_own_layers: i32, pub ctx: i32, pub pad: i32, pub weight_bytes: i64 }
+pub struct fc_decoder_info { pub vocab: i32, pub width: i32, pub n_layers: i32, pub n_own_layers: i32, pub ctx: i32, pub pad: i32, pub weight_bytes: i64 }
 
 #[link(name = "ferrum_cuda")]
 extern "C" {
@@ -177,20 +177,20 @@ extern "C" {
     pub fn fc_llama_generate(c: *mut fc_llama_cache, prompt: *const i32, n: c_int, max_new: c_int, params: *const fc_sampling, stops: *const i32, n_stops: c_int, rng_state: *mut u64, cancel: *const i32, out: *mut i32, n_out: *mut c_int) -> c_int;
     pub fn fc_llama_last_decode_ms(c: *const fc_llama_cache) -> f32;
     pub fn fc_model_dir_architecture(dir: *const c_char, out: *mut c_char, cap: c_int) -> c_int;
-    pub fn fc_nurinex_probe(dir: *const c_char, out: *mut fc_nurinex_info) -> c_int;
-    pub fn fc_nurinex_load(dir: *const c_char, device: c_int, math_mode: c_int, ctx: c_int, out: *mut *mut fc_nurinex) -> c_int;
-    pub fn fc_nurinex_free(m: *mut fc_nurinex);
-    pub fn fc_nurinex_get_info(m: *const fc_nurinex, out: *mut fc_nurinex_info) -> c_int;
-    pub fn fc_nurinex_cache_create(m: *mut fc_nurinex, out: *mut *mut fc_nurinex_cache) -> c_int;
-    pub fn fc_nurinex_cache_free(c: *mut fc_nurinex_cache);
-    pub fn fc_nurinex_cache_clear(c: *mut fc_nurinex_cache) -> c_int;
-    pub fn fc_nurinex_cache_pos(c: *const fc_nurinex_cache) -> c_int;
-    pub fn fc_nurinex_feed(c: *mut fc_nurinex_cache, ids: *const i32, n: c_int, want: *const i32, n_want: c_int, logits: *mut f32) -> c_int;
-    pub fn fc_nurinex_feed_layers(c: *mut fc_nurinex_cache, ids: *const i32, n: c_int, layers: *mut f32) -> c_int;
-    pub fn fc_nurinex_score(c: *mut fc_nurinex_cache, ids: *const i32, n: c_int, from_: c_int, score: *mut fc_score, lp: *mut f32, is_greedy: *mut u8) -> c_int;
-    pub fn fc_nurinex_generate(c: *mut fc_nurinex_cache, prompt: *const i32, n: c_int, max_new: c_int, params: *const fc_sampling, stops: *const i32, n_stops: c_int, rng_state: *mut u64, cancel: *const i32, out: *mut i32, n_out: *mut c_int) -> c_int;
-    pub fn fc_nurinex_last_forward_ms(m: *const fc_nurinex) -> f32;
-    pub fn fc_nurinex_last_decode_ms(c: *const fc_nurinex_cache) -> f32;
+    pub fn fc_decoder_probe(dir: *const c_char, out: *mut fc_decoder_info) -> c_int;
+    pub fn fc_decoder_load(dir: *const c_char, device: c_int, math_mode: c_int, ctx: c_int, out: *mut *mut fc_decoder) -> c_int;
+    pub fn fc_decoder_free(m: *mut fc_decoder);
+    pub fn fc_decoder_get_info(m: *const fc_decoder, out: *mut fc_decoder_info) -> c_int;
+    pub fn fc_decoder_cache_create(m: *mut fc_decoder, out: *mut *mut fc_decoder_cache) -> c_int;
+    pub fn fc_decoder_cache_free(c: *mut fc_decoder_cache);
+    pub fn fc_decoder_cache_clear(c: *mut fc_decoder_cache) -> c_int;
+    pub fn fc_decoder_cache_pos(c: *const fc_decoder_cache) -> c_int;
+    pub fn fc_decoder_feed(c: *mut fc_decoder_cache, ids: *const i32, n: c_int, want: *const i32, n_want: c_int, logits: *mut f32) -> c_int;
+    pub fn fc_decoder_feed_layers(c: *mut fc_decoder_cache, ids: *const i32, n: c_int, layers: *mut f32) -> c_int;
+    pub fn fc_decoder_score(c: *mut fc_decoder_cache, ids: *const i32, n: c_int, from_: c_int, score: *mut fc_score, lp: *mut f32, is_greedy: *mut u8) -> c_int;
+    pub fn fc_decoder_generate(c: *mut fc_decoder_cache, prompt: *const i32, n: c_int, max_new: c_int, params: *const fc_sampling, stops: *const i32, n_stops: c_int, rng_state: *mut u64, cancel: *const i32, out: *mut i32, n_out: *mut c_int) -> c_int;
+    pub fn fc_decoder_last_forward_ms(m: *const fc_decoder) -> f32;
+    pub fn fc_decoder_last_decode_ms(c: *const fc_decoder_cache) -> f32;
     pub fn fc_rowq_packed_len(rows: c_int, cols: c_int, kind: c_int) -> usize;
     pub fn fc_rowq_from_f32(data: *const f32, rows: c_int, cols: c_int, kind: c_int, scales: *mut f32, q: *mut u8) -> c_int;
     pub fn fc_rowq_to_f32(q: *const u8, scales: *const f32, rows: c_int, cols: c_int, kind: c_int, out: *mut f32) -> c_int;

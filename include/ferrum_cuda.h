@@ -463,35 +463,35 @@ int fc_model_dir_architecture(const char* dir, char* out, int cap);
  * constant comes from the folder's config.json; a layer may use another layer's tensors. Weights are bf16 and stay so.
  * math_mode: FC_MATH_BF16 (bf16 operands and caches; norms, scores, softmax, decays, recurrence and the residual are f32)
  * or FC_MATH_FP32 (f32 everywhere, caches too). ctx: positions a cache holds. */
-typedef struct fc_nurinex fc_nurinex;
-typedef struct fc_nurinex_cache fc_nurinex_cache;   /* key / value rows, recurrence states, token-shift rows, position */
-typedef struct fc_nurinex_info {
+typedef struct fc_decoder fc_decoder;
+typedef struct fc_decoder_cache fc_decoder_cache;   /* key / value rows, recurrence states, token-shift rows, position */
+typedef struct fc_decoder_info {
     int32_t vocab, width, n_layers, n_own_layers, ctx, pad;
     int64_t weight_bytes;   /* bytes of matrices one decoded token reads */
-} fc_nurinex_info;
+} fc_decoder_info;
 /* Validates a folder without a GPU. */
-int fc_nurinex_probe(const char* dir, fc_nurinex_info* out);
-int fc_nurinex_load(const char* dir, int device, int math_mode, int ctx, fc_nurinex** out);
-void fc_nurinex_free(fc_nurinex* m);
-int fc_nurinex_get_info(const fc_nurinex* m, fc_nurinex_info* out);
-int fc_nurinex_cache_create(fc_nurinex* m, fc_nurinex_cache** out);
-void fc_nurinex_cache_free(fc_nurinex_cache* c);
-int fc_nurinex_cache_clear(fc_nurinex_cache* c);
-int fc_nurinex_cache_pos(const fc_nurinex_cache* c);
+int fc_decoder_probe(const char* dir, fc_decoder_info* out);
+int fc_decoder_load(const char* dir, int device, int math_mode, int ctx, fc_decoder** out);
+void fc_decoder_free(fc_decoder* m);
+int fc_decoder_get_info(const fc_decoder* m, fc_decoder_info* out);
+int fc_decoder_cache_create(fc_decoder* m, fc_decoder_cache** out);
+void fc_decoder_cache_free(fc_decoder_cache* c);
+int fc_decoder_cache_clear(fc_decoder_cache* c);
+int fc_decoder_cache_pos(const fc_decoder_cache* c);
 /* The next n tokens of the cache's sequence: one token runs the decode step, more run as a portion of a prompt, cut
  * anywhere. logits [n_want][vocab] (host) of the places want[] among them, in that order; n_want may be 0. */
-int fc_nurinex_feed(fc_nurinex_cache* c, const int32_t* ids, int n, const int32_t* want, int n_want, float* logits);
+int fc_decoder_feed(fc_decoder_cache* c, const int32_t* ids, int n, const int32_t* want, int n_want, float* logits);
 /* The same for one portion (n <= 2048), leaving the residual stream after every layer: layers [n_layers][n][width]. */
-int fc_nurinex_feed_layers(fc_nurinex_cache* c, const int32_t* ids, int n, float* layers);
+int fc_decoder_feed_layers(fc_decoder_cache* c, const int32_t* ids, int n, float* layers);
 /* Clears the cache and scores ids[from..] given what precedes them, as fc_llama_score_from does for one window: ln
  * softmax(logits)[target], no probability floor. The sequence must fit the cache. */
-int fc_nurinex_score(fc_nurinex_cache* c, const int32_t* ids, int n, int from, fc_score* score, float* lp, uint8_t* is_greedy);
+int fc_decoder_score(fc_decoder_cache* c, const int32_t* ids, int n, int from, fc_score* score, float* lp, uint8_t* is_greedy);
 /* fc_llama_generate for this decoder: the same sampling, stops, cancel flag and generator state. */
-int fc_nurinex_generate(fc_nurinex_cache* c, const int32_t* prompt, int n, int max_new, const fc_sampling* params,
+int fc_decoder_generate(fc_decoder_cache* c, const int32_t* prompt, int n, int max_new, const fc_sampling* params,
                         const int32_t* stops, int n_stops, uint64_t* rng_state, const volatile int32_t* cancel,
                         int32_t* out, int* n_out);
-float fc_nurinex_last_forward_ms(const fc_nurinex* m);
-float fc_nurinex_last_decode_ms(const fc_nurinex_cache* c);
+float fc_decoder_last_forward_ms(const fc_decoder* m);
+float fc_decoder_last_decode_ms(const fc_decoder_cache* c);
 
 /* ---- per-row-scale int8 / int4 weights (quant.rs:122-263 QWeight, ops.rs:268-377 qlinear) ---- */
 /* The in-memory quantised weight of the reference: [rows = in_features][cols = out_features]

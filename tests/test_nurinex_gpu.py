@@ -10,9 +10,9 @@ import sys
 import numpy as np
 import pytest
 
-from ferrum_cpu_b200 import FerrumCudaError, _lib, engine, nurinex, registry
+from ferrum_cpu_b200 import FerrumCudaError, _lib, decoder, engine, registry
 from ferrum_cpu_b200.backend import CudaBackend, GenRequest
-from ferrum_cpu_b200.nurinex import CudaNurinex
+from ferrum_cpu_b200.decoder import CudaNurinex
 from tests.nurinex_models import MD, NO, L, build, configs, error, ids, needle
 
 pytestmark = pytest.mark.gpu

@@ -8,7 +8,7 @@ import struct
 import numpy as np
 import pytest
 
-from ferrum_cpu_b200 import FerrumCudaError, _lib, nurinex, registry
+from ferrum_cpu_b200 import FerrumCudaError, _lib, decoder, registry
 from tests.nurinex_models import MD, NO, L, build, configs, ids
 
 
@@ -78,7 +78,7 @@ def test_oracle_is_causal():
 def test_probe_reads_every_configuration(tmp_path, name):
     config, rows, rank = configs()[name]
     path, _ = build(tmp_path, config, bias_rows=rows, rank=rank)
-    info = nurinex.probe(path)
+    info = decoder.probe(path)
     assert (info.vocab, info.width, info.n_layers) == (config["vocab"], config["width"], len(config["layers"]))
     assert info.n_own_layers == sum("weights_of" not in e for e in config["layers"])
     assert registry.architecture(path) == "Nurinex" and "Nurinex" in registry.ARCHITECTURES
@@ -114,7 +114,7 @@ def test_bad_configurations_are_refused_before_a_gpu_is_touched(tmp_path, what):
     change, code = BAD[what]
     _edit_config(path, change)
     with pytest.raises(FerrumCudaError) as e:
-        nurinex.probe(path)
+        decoder.probe(path)
     assert e.value.code == code, str(e.value)
 
 
@@ -129,7 +129,7 @@ def test_bad_tensor_files_are_refused(tmp_path):
     def refused(data):
         open(file, "wb").write(data)
         with pytest.raises(FerrumCudaError) as e:
-            nurinex.probe(path)
+            decoder.probe(path)
         return e.value.code
 
     def with_head(h):
@@ -152,14 +152,14 @@ def test_bad_tensor_files_are_refused(tmp_path):
     h = json.loads(json.dumps(head))
     h["__metadata__"] = {"format": "pt", "note": "escapes \" \\ é \n"}
     open(file, "wb").write(with_head(h))
-    nurinex.probe(path)                                                  # metadata is skipped
+    decoder.probe(path)                                                  # metadata is skipped
 
 
 def test_load_needs_a_gpu_and_a_mode_it_has(tmp_path):
     config, rows, rank = configs()["mixed"]
     path, _ = build(tmp_path, config, bias_rows=rows, rank=rank)
     with pytest.raises(FerrumCudaError) as e:
-        nurinex.CudaNurinex(path, math_mode=_lib.FC_MATH_BF16X3)
+        decoder.CudaNurinex(path, math_mode=_lib.FC_MATH_BF16X3)
     assert e.value.code == _lib.FC_E_ARG
     if _lib.lib().fc_device_count() == 0:
         with pytest.raises(FerrumCudaError) as e:
