@@ -2,7 +2,7 @@
 """Benchmark of the Q8_0 GPT-2 forward path on B200.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--workload ...] [--impl ours|reference]
-    python bench.py --case decode|score|linear|rowq|ggml-linear|streams|llama-*|nurinex-* [...]
+    python bench.py --case decode|score|linear|rowq|ggml-linear|streams|llama-*|nurinex-*|zogevik-* [...]
 
 Workloads (synthetic, seeded; shapes of the reference's configurations):
   decode        : GPT-2-small-shaped Q8_0 model, batch 1, 32-token prompt, 256 greedy tokens with a
@@ -21,6 +21,8 @@ Workloads (synthetic, seeded; shapes of the reference's configurations):
   llama-1b      : the imported Llama-shaped decoder.
   nurinex       : prefill, scoring and batch-1 decode of the Nurinex decoder at a few sizes (bf16, random weights),
                   each beside the Llama-shaped decoder with layers of the same sizes.
+  zogevik       : the same of the Zogevik decoder, each shape beside a Nurinex model of the same width, depth, heads and
+                  active feed-forward.
 
 --case runs one small, self-terminating piece of the same kernels (a few tokens / windows / one
 product) and prints CUDA-event times: these are the command lines the profiler notes under
@@ -289,60 +291,107 @@ def llama_twin(name):
     return (V, d, n, H, G, hd, ff, 2304)
 
 
-def run_nurinex(a, names, prompts=(256, 1024, 2048), with_llama=True):
-    """Prefill (one sequence, logits of the last row), scoring (logits of every row) and greedy decode, device-timed by the
-    library's CUDA events; weights of every shape exceed the L2."""
-    import tempfile
+def zogevik_work(name, T, p_first, n_new):
+    """As nurinex_work for a named Zogevik shape: a token meets its chosen experts only; attention as defined (keys and values of
+    their own per head, windowed), and in decoding the cached rows once and W_uk, W_uv once."""
+    from ferrum_cpu_b200 import model_dir
+    config = model_dir.zogevik_named_config(name)
+    d, V = config["width"], config["vocab"]
+    weights = V * d
+    flop = 0.0
+    cached = 0.0
+    seen = lambda w, p: min(p + 1, w)
+    for layer in config["layers"]:
+        m, r = layer["mixer"], layer["mlp"]["router"]
+        H, w = m["heads"], m["mask"]["size"]
+        pairs = sum(seen(w, p) for p in range(T))
+        row = sum(seen(w, p) for p in range(p_first, p_first + n_new)) / n_new
+        weights += d * (r["experts"] + 2 * r["top"] * layer["mlp"]["expert"]["ff"] + H * m["vdim"])
+        if layer["type"] == "latent_attention":
+            weights += H * (m["dim"] + m["rot_dim"]) * d + (m["kv_rank"] + m["rot_dim"]) * d + H * (m["dim"] + m["vdim"]) * m["kv_rank"]
+            flop += 2.0 * H * (m["dim"] + m["rot_dim"] + m["vdim"]) * pairs
+            cached += row * (m["kv_rank"] + m["rot_dim"]) * 2
+        else:
+            weights += H * m["dim"] * d + (0 if "kv_from" in m else m["kv_heads"] * (m["dim"] + m["vdim"]) * d)
+            flop += 2.0 * H * (m["dim"] + m["vdim"]) * pairs
+            cached += row * m["kv_heads"] * (m["dim"] + m["vdim"]) * 2
+    return weights, flop + 2.0 * weights * T, 2.0 * weights + cached
 
+
+def nurinex_twin(name):
+    """The Nurinex shape with the width, depth, heads and active feed-forward of a named Zogevik shape."""
+    from ferrum_cpu_b200 import model_dir
+    V, d, n, _, (H, G, hd, _), _, (_, top, ff, _, _) = model_dir.ZOGEVIK_SHAPES[name]
+    key = "twin of " + name
+    model_dir.NURINEX_SHAPES[key] = (V, d, n, H, G, hd, d // 64, 64, top * ff, 64)
+    return key
+
+
+def time_folder(a, make, name, V, d, work, prompts, row, prefix=""):
+    """Prefill (one sequence, logits of the last row), scoring (logits of every row) and greedy decode of one model folder,
+    device-timed by the library's CUDA events; fills `row`."""
+    import ferrum_cpu_b200 as fcb
+    from ferrum_cpu_b200 import synth
+    from ferrum_cpu_b200.engine import sampling
+    hbm, tf, _ = peaks()
+    m = make()
+    cache = m.new_cache()
+    fcb.take_launch_count()
+    for T in prompts:
+        ids = synth.token_ids(1, T + 1, V)
+
+        def prefill():
+            cache.clear()
+            m.feed(ids[:T], cache, [T - 1])
+        ms = median_after_warmup(prefill, lambda: m.last_forward_ms, a.steps)
+        _, flop, _ = work(name, T, 0, 1)
+        flop_p = flop - 2.0 * V * d * (T - 1)
+        row[f"{prefix}prefill_{T}"] = {"tokens_per_s": T / ms * 1e3, "ms": ms, "tflops": flop_p / ms / 1e9, "frac": flop_p / ms / 1e9 / tf}
+        ms = median_after_warmup(lambda: m.score_from(ids, 1), lambda: m.last_forward_ms, a.steps)
+        row[f"{prefix}score_{T}"] = {"positions_per_s": T / ms * 1e3, "ms": ms, "tflops": flop / ms / 1e9, "frac": flop / ms / 1e9 / tf}
+    for start in (PROMPT, 1920):
+        prompt = synth.token_ids(0, start, V)
+        ms = median_after_warmup(lambda: m.generate(prompt, NEW_TOKENS, sampling(temperature=0.0), cache=cache), lambda: cache.last_decode_ms, a.steps)
+        _, _, byts = work(name, 1, start, NEW_TOKENS)
+        row[f"{prefix}decode_from_{start}"] = {"tokens_per_s": NEW_TOKENS / ms * 1e3, "us_per_token": ms / NEW_TOKENS * 1e3,
+                                               "gbs": byts * NEW_TOKENS / ms / 1e6, "frac": byts * NEW_TOKENS / ms / 1e6 / hbm}
+    row[prefix + "gpu_launches"] = int(fcb.take_launch_count())
+    m.close()
+
+
+def median_after_warmup(fn, read, reps):
+    for _ in range(3):
+        fn()
+    vals = []
+    for _ in range(reps):
+        fn()
+        vals.append(read())
+    return statistics.median(vals)
+
+
+def folder_of(write, name, cls, **kw):
+    """A model of a named synthetic shape, from a folder that is gone once it is loaded."""
+    import tempfile
+    with tempfile.TemporaryDirectory() as tmp:
+        write(tmp, name, **kw)
+        return cls(tmp, ctx=2304)
+
+
+def run_nurinex(a, names, prompts=(256, 1024, 2048), with_llama=True):
+    """The Nurinex decoder beside the Llama-shaped one of the same layer sizes; weights of every shape exceed the L2."""
     import ferrum_cpu_b200 as fcb
     from ferrum_cpu_b200 import model_dir, synth
+    from ferrum_cpu_b200.decoder import CudaNurinex
     from ferrum_cpu_b200.engine import sampling
     from ferrum_cpu_b200.llama import CudaLlama
-    from ferrum_cpu_b200.decoder import CudaNurinex
     hbm, tf, kind = peaks()
     greedy = sampling(temperature=0.0)
     rows = []
     for name in names:
-        V = model_dir.NURINEX_SHAPES[name][0]
+        V, d = model_dir.NURINEX_SHAPES[name][:2]
         row = {"shape": name, "sizes": dict(zip(("vocab", "width", "layers", "heads", "kv_heads", "dim", "r_heads", "r_dim", "ff", "rank"),
                                                 model_dir.NURINEX_SHAPES[name]))}
-        with tempfile.TemporaryDirectory() as tmp:
-            model_dir.nurinex_named(tmp, name)
-            m = CudaNurinex(tmp, ctx=2304)
-        cache = m.new_cache()
-        fcb.take_launch_count()
-
-        def best(fn, read, reps):
-            fn()
-            fn()
-            fn()
-            vals = []
-            for _ in range(reps):
-                fn()
-                vals.append(read())
-            return statistics.median(vals)
-
-        for T in prompts:
-            ids = synth.token_ids(1, T + 1, V)
-
-            def prefill():
-                cache.clear()
-                m.feed(ids[:T], cache, [T - 1])
-            ms = best(prefill, lambda: m.last_forward_ms, a.steps)
-            _, flop, _ = nurinex_work(name, T, 0, 1)
-            flop_p = flop - 2.0 * V * model_dir.NURINEX_SHAPES[name][1] * (T - 1)
-            row[f"prefill_{T}"] = {"tokens_per_s": T / ms * 1e3, "ms": ms, "tflops": flop_p / ms / 1e9, "frac": flop_p / ms / 1e9 / tf}
-            ms = best(lambda: m.score_from(ids, 1), lambda: m.last_forward_ms, a.steps)
-            row[f"score_{T}"] = {"positions_per_s": T / ms * 1e3, "ms": ms, "tflops": flop / ms / 1e9, "frac": flop / ms / 1e9 / tf}
-        for start in (PROMPT, 1920):
-            prompt = synth.token_ids(0, start, V)
-            n_new = NEW_TOKENS
-            ms = best(lambda: m.generate(prompt, n_new, greedy, cache=cache), lambda: cache.last_decode_ms, a.steps)
-            _, _, byts = nurinex_work(name, 1, start, n_new)
-            row[f"decode_from_{start}"] = {"tokens_per_s": n_new / ms * 1e3, "us_per_token": ms / n_new * 1e3,
-                                           "gbs": byts * n_new / ms / 1e6, "frac": byts * n_new / ms / 1e6 / hbm}
-        row["gpu_launches"] = int(fcb.take_launch_count())
-        m.close()
+        time_folder(a, lambda: folder_of(model_dir.nurinex_named, name, CudaNurinex), name, V, d, nurinex_work, prompts, row)
         if with_llama:
             sml = synth.SynthLlama(*llama_twin(name), math_mode=fcb.FC_MATH_BF16X3)
             gl = CudaLlama.from_synth(sml)
@@ -351,20 +400,40 @@ def run_nurinex(a, names, prompts=(256, 1024, 2048), with_llama=True):
             qd, kvd = c["n_head"] * c["head_dim"], c["n_kv_head"] * c["head_dim"]
             for T in prompts:
                 ids = synth.token_ids(1, T, V).reshape(1, T)
-                ms = best(lambda: gl.score_sequences(ids, batch_windows=1), lambda: gl.last_score_ms, a.steps)
+                ms = median_after_warmup(lambda: gl.score_sequences(ids, batch_windows=1), lambda: gl.last_score_ms, a.steps)
                 flop = 2.0 * sml.q8_weight_bytes * 32 / 34 * T + c["n_layer"] * 4.0 * qd * T * (T + 1) / 2
                 row[f"llama_score_{T}"] = {"positions_per_s": T / ms * 1e3, "ms": ms, "tflops": flop / ms / 1e9, "frac": flop / ms / 1e9 / tf}
             for start in (PROMPT, 1920):
                 prompt = synth.token_ids(0, start, V)
-                ms = best(lambda: gl.generate(prompt, NEW_TOKENS, greedy, cache=lc), lambda: lc.last_decode_ms, a.steps)
+                ms = median_after_warmup(lambda: gl.generate(prompt, NEW_TOKENS, greedy, cache=lc), lambda: lc.last_decode_ms, a.steps)
                 byts = sml.q8_weight_bytes + c["n_layer"] * 2 * (start + NEW_TOKENS / 2) * kvd * 4
                 row[f"llama_decode_from_{start}"] = {"tokens_per_s": NEW_TOKENS / ms * 1e3, "us_per_token": ms / NEW_TOKENS * 1e3,
                                                      "gbs": byts * NEW_TOKENS / ms / 1e6, "frac": byts * NEW_TOKENS / ms / 1e6 / hbm}
             gl.close()
         rows.append(row)
     main_row = rows[len(rows) // 2]
+    print_folder_line(a, "Nurinex", main_row, rows)
+
+
+def run_zogevik(a, names, prompts=(256, 1024, 2048)):
+    """The Zogevik decoder beside the Nurinex one of the same width, depth, heads and active feed-forward."""
+    from ferrum_cpu_b200 import model_dir
+    from ferrum_cpu_b200.decoder import CudaNurinex, CudaZogevik
+    rows = []
+    for name in names:
+        V, d = model_dir.ZOGEVIK_SHAPES[name][:2]
+        row = {"shape": name, "sizes": dict(zip(("vocab", "width", "layers", "latent", "grouped", "window", "experts"), model_dir.ZOGEVIK_SHAPES[name]))}
+        time_folder(a, lambda: folder_of(model_dir.zogevik_named, name, CudaZogevik), name, V, d, zogevik_work, prompts, row)
+        twin = nurinex_twin(name)
+        time_folder(a, lambda: folder_of(model_dir.nurinex_named, twin, CudaNurinex), twin, V, d, nurinex_work, prompts, row, "nurinex_")
+        rows.append(row)
+    print_folder_line(a, "Zogevik", rows[len(rows) // 2], rows)
+
+
+def print_folder_line(a, design, main_row, rows):
+    hbm, tf, kind = peaks()
     print(json.dumps({
-        "metric": "Nurinex batch-1 greedy decode tokens/s (bf16)", "value": main_row[f"decode_from_{PROMPT}"]["tokens_per_s"], "unit": "tokens/s",
+        "metric": design + " batch-1 greedy decode tokens/s (bf16)", "value": main_row[f"decode_from_{PROMPT}"]["tokens_per_s"], "unit": "tokens/s",
         "n_gpus": 1, "steps": a.steps, "warmup": 3, "higher_is_better": True, "scaling": "n/a", "vs_baseline": None, "dtype": "bf16",
         "data": "synthetic", "config": {"workload": "random weights; value is the middle shape; %d-token prompt + %d greedy tokens; weights of every "
                                                     "shape exceed the L2" % (PROMPT, NEW_TOKENS)},
@@ -432,23 +501,23 @@ def run_case(a):
             print(f"ggml type {t} M={a.m} K={a.k} N={a.n}: {ms * 1e3:.1f} us, {byts / ms / 1e6:.1f} GB/s")
         _lib.lib().fc_ggml_weight_free(h)
         return
-    if a.case.startswith("nurinex"):
-        import tempfile
-        from ferrum_cpu_b200 import model_dir
+    if a.case.startswith(("nurinex", "zogevik")):
+        from ferrum_cpu_b200 import decoder, model_dir
         from ferrum_cpu_b200.engine import sampling
-        from ferrum_cpu_b200.decoder import CudaNurinex
-        name = a.model if a.model in model_dir.NURINEX_SHAPES else "nurinex-1b"
-        if a.layers:
-            shape = list(model_dir.NURINEX_SHAPES[name])
-            shape[2] = a.layers
-            model_dir.NURINEX_SHAPES[name] = tuple(shape)
-        with tempfile.TemporaryDirectory() as tmp:
-            model_dir.nurinex_named(tmp, name)
-            m = CudaNurinex(tmp, ctx=2304)
+        if a.case.startswith("zogevik"):
+            name = a.model if a.model in model_dir.ZOGEVIK_SHAPES else "zogevik-1b"
+            m = folder_of(model_dir.zogevik_named, name, decoder.CudaZogevik, layers=a.layers)
+        else:
+            name = nurinex_twin(a.model) if a.model in model_dir.ZOGEVIK_SHAPES else (a.model if a.model in model_dir.NURINEX_SHAPES else "nurinex-1b")
+            if a.layers:
+                shape = list(model_dir.NURINEX_SHAPES[name])
+                shape[2] = a.layers
+                model_dir.NURINEX_SHAPES[name] = tuple(shape)
+            m = folder_of(model_dir.nurinex_named, name, decoder.CudaNurinex)
         cache = m.new_cache()
         ids = synth.token_ids(1, a.prompt, m.info.vocab)
         for _ in range(a.reps):
-            if a.case == "nurinex-prefill":
+            if a.case.endswith("prefill"):
                 cache.clear()
                 m.feed(ids, cache, [a.prompt - 1])
                 print(f"{name} prefill {a.prompt} tokens: device {m.last_forward_ms:.3f} ms, launches {fcb.take_launch_count()}")
@@ -591,17 +660,17 @@ def main():
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=5)
     ap.add_argument("--warmup", type=int, default=3)
-    ap.add_argument("--workload", choices=["decode", "score", "both", "streams-medium", "score-medium", "sweep", "tiny", "llama-1b", "nurinex"],
+    ap.add_argument("--workload", choices=["decode", "score", "both", "streams-medium", "score-medium", "sweep", "tiny", "llama-1b", "nurinex", "zogevik"],
                     default="both", help="see the module docstring")
     ap.add_argument("--case", choices=["decode", "score", "linear", "rowq", "ggml-linear", "streams", "llama-decode", "llama-score",
-                                       "nurinex-decode", "nurinex-prefill"], default=None,
+                                       "nurinex-decode", "nurinex-prefill", "zogevik-decode", "zogevik-prefill"], default=None,
                     help="run one small self-terminating case (for profiler captures) instead of a workload")
     ap.add_argument("--model", default="small")
     ap.add_argument("--tokens", type=int, default=8)
     ap.add_argument("--prompt", type=int, default=32)
     ap.add_argument("--windows", type=int, default=4)
-    ap.add_argument("--layers", type=int, default=0, help="--case nurinex-*: layers of the shape (0: its own number)")
-    ap.add_argument("--shapes", default="nurinex-small,nurinex-1b,nurinex-7b-layers", help="--workload nurinex: which shapes")
+    ap.add_argument("--layers", type=int, default=0, help="--case nurinex-* / zogevik-*: layers of the shape (0: its own number)")
+    ap.add_argument("--shapes", default="", help="--workload nurinex / zogevik: which named shapes (all)")
     ap.add_argument("--streams", type=int, default=8)
     ap.add_argument("--m", type=int, default=1)
     ap.add_argument("--k", type=int, default=768)
@@ -661,9 +730,11 @@ def main():
         return float(t.item())
 
     hbm_peak, tf_peak, peak_kind = peaks()
-    if args.workload == "nurinex":
+    if args.workload in ("nurinex", "zogevik"):
         if rank == 0:
-            run_nurinex(args, args.shapes.split(","))
+            from ferrum_cpu_b200 import model_dir
+            run, shapes = (run_nurinex, model_dir.NURINEX_SHAPES) if args.workload == "nurinex" else (run_zogevik, model_dir.ZOGEVIK_SHAPES)
+            run(args, args.shapes.split(",") if args.shapes else list(shapes))
         if world > 1:
             dist.destroy_process_group()
         return

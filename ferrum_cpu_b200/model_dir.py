@@ -1,4 +1,4 @@
-"""Writer of model folders (config.json + model.safetensors) and synthetic Nurinex models, for tests and
+"""Writer of model folders (config.json + model.safetensors) and synthetic models of the designs, for tests and
 benchmarks. Reading is the library's (csrc/model_dir.cpp)."""
 import json
 import os
@@ -117,6 +117,121 @@ def nurinex_tensors(config, seed=0, bias_rows=12, rank=8):
             put(p + "mlp.up", (ff, d), d ** -0.5)
             put(p + "mlp.down", (d, ff), ff ** -0.5)
             put(p + "mlp.act", (2,), 0.5, 0.3)
+    put("final.norm", (d,), 0.2, 1.0)
+    put("head", (V, d), d ** -0.5)
+    return out
+
+
+def experts_config(experts=8, top=2, ff=64, groups=1, keep=1):
+    """The routed feed-forward of a Zogevik layer."""
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}}}
+
+
+def zogevik_latent(heads=4, dim=32, rot=16, rank=64, vdim=32, window=40, base=10000.0, scale=None, mlp=None):
+    """One entry of `layers`: latent attention. window None: all earlier positions; mlp None: no feed-forward."""
+    mixer = {"heads": heads, "dim": dim, "rot_dim": rot, "kv_rank": rank, "vdim": vdim, "rot": {"base": base, "dims": rot},
+             "scale": (dim + rot) ** -0.5 if scale is None else scale, "mask": None if window is None else {"size": window}}
+    return {"type": "latent_attention", "mixer": mixer, "mlp": mlp}
+
+
+def zogevik_attention(heads=4, kv_heads=2, dim=32, vdim=32, rot=16, window=40, base=10000.0, scale=None, kv_from=None, mlp=None):
+    """One entry of `layers`: grouped-query attention; kv_from: the layer whose keys and values it uses."""
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "rot": {"base": base, "dims": rot},
+             "scale": dim ** -0.5 if scale is None else scale, "mask": None if window is None else {"size": window}}
+    if kv_from is not None:
+        mixer["kv_from"] = kv_from
+    return {"type": "attention", "mixer": mixer, "mlp": mlp}
+
+
+def zogevik_config(vocab, width, layers, eps=1e-5):
+    return {"architecture": "Zogevik", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers}
+
+
+# name -> (vocab, width, layers, latent (heads, dim, rotated, rank, value dim), grouped-query (heads, kv heads, dim, rotated), window,
+# (experts, chosen, ff of one, groups, kept)): layers as those of real models, few of them; every third is grouped-query, and
+# every second of those uses the keys of the one before.
+ZOGEVIK_SHAPES = {
+    "zogevik-small": (32000, 1024, 12, (16, 64, 32, 256, 64), (16, 4, 64, 64), 1024, (32, 8, 512, 4, 2)),
+    "zogevik-1b": (32000, 2048, 8, (16, 128, 64, 512, 128), (32, 8, 64, 64), 1024, (32, 8, 1024, 4, 2)),
+    "zogevik-7b-layers": (32000, 4096, 3, (32, 128, 64, 512, 128), (32, 8, 128, 64), 1024, (16, 8, 1376, 4, 3)),
+}
+
+
+def zogevik_named_config(name, layers=0):
+    V, d, n, (H, dim, rot, rank, vdim), (AH, G, adim, arot), window, (E, top, ff, groups, keep) = ZOGEVIK_SHAPES[name]
+    mlp = experts_config(E, top, ff, groups, keep)
+    out, owner = [], None
+    for i in range(layers or n):
+        if i % 3 != 2:
+            out.append(zogevik_latent(H, dim, rot, rank, vdim, window, 10000.0, mlp=mlp))
+            continue
+        out.append(zogevik_attention(AH, G, adim, adim, arot, window, 10000.0, kv_from=owner, mlp=mlp))
+        owner = i if owner is None else None
+    return zogevik_config(V, d, out)
+
+
+def zogevik_named(path, name, seed=0, layers=0):
+    """Writes a synthetic model of a named shape; returns its configuration."""
+    config = zogevik_named_config(name, layers)
+    write(path, config, zogevik_tensors(config, seed=seed, pool=1 << 22))
+    return config
+
+
+def zogevik_tensors(config, seed=0, code=0, pool=0):
+    """Random bf16 weights of the shapes a configuration asks for: name -> uint16 array. code > 0: the first `code` entries of
+    the residual keep what the embedding put there (the sublayers' norms are 0 on them) and routers read nothing else, so that
+    a token's experts do not hang on the last bits of what came before. pool > 0: large matrices are filled from that many
+    numbers over and over, each from a place of its own (models of gigabytes)."""
+    rng = np.random.default_rng(seed)
+    d, V = config["width"], config["vocab"]
+    out, base = {}, rng.standard_normal(pool, dtype=np.float32) if pool else None
+
+    def put(name, shape, std, mean=0.0):
+        n = int(np.prod(shape))
+        if pool and n * 4 > pool:
+            bits = to_bf16(base * np.float32(std) + np.float32(mean))
+            out[name] = np.resize(np.roll(bits, -int(rng.integers(0, pool))), shape)
+            return
+        out[name] = to_bf16(rng.standard_normal(shape, dtype=np.float32) * np.float32(std) + np.float32(mean))
+
+    def sublayer_norm(name):
+        w = rng.standard_normal(d, dtype=np.float32) * np.float32(0.2) + np.float32(1.0)
+        w[:code] = 0.0
+        out[name] = to_bf16(w)
+
+    put("embed", (V, d), 1.0)
+    put("embed.norm", (d,), 0.2, 1.0)
+    for i, layer in enumerate(config["layers"]):
+        p, m, mlp = f"l{i}.", layer["mixer"], layer.get("mlp")
+        H, dim, vdim = m["heads"], m["dim"], m["vdim"]
+        sublayer_norm(p + "norm1")
+        if layer["type"] == "latent_attention":
+            rank, rot = m["kv_rank"], m["rot_dim"]
+            put(p + "mix.q", (H * (dim + rot), d), d ** -0.5)
+            put(p + "mix.dkv", (rank + rot, d), d ** -0.5)
+            put(p + "mix.dkv.norm", (rank,), 0.2, 1.0)
+            put(p + "mix.uk", (H * dim, rank), rank ** -0.5)
+            put(p + "mix.uv", (H * vdim, rank), rank ** -0.5)
+        else:
+            G = m["kv_heads"]
+            put(p + "mix.q", (H * dim, d), d ** -0.5)
+            put(p + "mix.q.norm", (H * dim,), 0.2, 1.0)
+            if m.get("kv_from") is None:
+                put(p + "mix.k", (G * dim, d), d ** -0.5)
+                put(p + "mix.k.norm", (G * dim,), 0.2, 1.0)
+                put(p + "mix.v", (G * vdim, d), d ** -0.5)
+        put(p + "mix.o", (d, H * vdim), (H * vdim) ** -0.5)
+        if not mlp:
+            continue
+        sublayer_norm(p + "norm2")
+        ff = mlp["expert"]["ff"]
+        for e in range(mlp["router"]["experts"]):
+            put(f"{p}mlp.e{e}.up", (ff, d), d ** -0.5 * 1.5)
+            put(f"{p}mlp.e{e}.down", (d, ff), ff ** -0.5)
+        n = code or d
+        r = np.zeros((mlp["router"]["experts"], d), dtype=np.float32)
+        r[:, :n] = rng.standard_normal((r.shape[0], n), dtype=np.float32) * np.float32(n ** -0.5)
+        out[p + "mlp.router"] = to_bf16(r)
     put("final.norm", (d,), 0.2, 1.0)
     put("head", (V, d), d ** -0.5)
     return out
