@@ -56,7 +56,10 @@ bool plan_of(const AttnDecode& a, int kt, Plan* o) {
     return at <= 200 * 1024;
 }
 int make_plan(const AttnDecode& a, Plan* l) {
-    for (int kt = 64; kt >= 16; kt /= 2)
+    // the smallest tile with which the splits reach every visible row; several tiles a split where that is too large
+    int want = 16;
+    while (want < 64 && want * a.max_splits < a.reach) want *= 2;
+    for (int kt = want; kt >= 16; kt /= 2)
         if (plan_of(a, kt, l)) return FC_OK;
     return fail(FC_E_SHAPE, "decode attention: rows of %d values do not fit shared memory", a.kw);
 }

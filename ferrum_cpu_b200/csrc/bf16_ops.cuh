@@ -195,6 +195,7 @@ struct GemvSeg {
     const uint16_t* w;    // first row; rows ldw apart, K_pad weights of each (a multiple of 64), K inputs
     const int* index;     // not null: the rows begin *index * w_step weights further on (an expert chosen on the device)
     size_t w_step;
+    int early;            // the index was there before the kernel ahead began (its own wait is behind this one's launch)
     int n, ldw, K_pad, src, K;
     float* y;
     int epi;
@@ -276,7 +277,7 @@ struct AttnDecode {
     RotAttn prep;                                    // H 0: q is ready (f32 [H][kw], scaled), the cache row written
     const float* q = nullptr;                        // the projection row q | k | v, or the ready queries
     float *part = nullptr, *part_ml = nullptr;       // [splits][H][vw up to 4s], [splits][H][2]
-    int max_splits = 1;
+    int max_splits = 1, reach = 0;                   // reach: most rows a token can see
     unsigned int* counter = nullptr;                 // one a block of heads; null: the splits stay as they are
     float* out = nullptr;
     const StepState* state = nullptr;

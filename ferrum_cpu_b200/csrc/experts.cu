@@ -1,7 +1,7 @@
 // Routing of feed-forwards that are cut into experts: which experts a token uses and with what weight, and the rows of a
 // portion regrouped so that every expert's products read consecutive rows.
 //
-//   route_rows_kernel    8 tokens a CTA: logits in f32 (rows in shared memory piece by piece, a warp holds four experts), softmax
+//   route_rows_kernel    8 tokens a CTA: logits in f32 (rows in shared memory, a warp holds four experts at a time), softmax
 //                        over all experts, the best groups (a group's score is its largest), the best experts in them; a slot's
 //                        place within its expert from an atomic counter (the order of an expert's rows does not matter)
 //   gather_rows_kernel   a CTA per token: places become rows (prefix sums of the counts), its operand row copied to each; the
@@ -13,12 +13,13 @@
 #include <algorithm>
 
 #include "pdl.cuh"
+#include "post_norm.cuh"
 #include "rot_rows.cuh"
 
 namespace fc {
 
 namespace {
-constexpr int NT = 256, TOK = 8, EPW = 4, KC = 512;      // tokens a CTA, experts a warp holds at once, columns staged at once
+constexpr int NT = 256, TOK = 8, EPW = 4;      // tokens a CTA, experts a warp holds at once
 constexpr int kMaxExperts = 1024, kMaxGroups = 256;
 
 // Place of column k in shared memory: within 256 values, lane l's eight are two float4 at 4 l and 128 + 4 l.
@@ -49,10 +50,22 @@ __device__ __forceinline__ int warp_argmax(const float* z, int n, float* best) {
     return at;
 }
 // One warp chooses from logits z (overwritten) of a token; gs: room for the groups' scores. emit(slot, expert, weight) runs in
-// lane 0. Softmax keeps the logits' order, so they are compared in its place.
+// one lane per slot. Softmax keeps the logits' order, so they are compared in its place; of equals the first counts as larger.
+// Few entries are ranked by counting those ahead of each, more are taken one by one.
+constexpr int kRankBy = 128;
+__device__ __forceinline__ int rank_of(const float* z, int n, int i) {
+    const float v = z[i];
+    int ahead = 0;
+#pragma unroll 8
+    for (int k = 0; k < n; ++k) ahead += z[k] > v || (z[k] == v && k < i);
+    return ahead;
+}
 template <class F>
 __device__ void choose(float* z, float* gs, const Router& r, F emit) {
     const int lane = threadIdx.x & 31, E = r.experts;
+    for (int i = lane; i < E; i += 32)
+        if (z[i] != z[i]) z[i] = -INFINITY;                          // what is not a number comes last: every slot gets an expert
+    __syncwarp();
     float top;
     warp_argmax(z, E, &top);
     float sum = 0.0f;
@@ -67,16 +80,16 @@ __device__ void choose(float* z, float* gs, const Router& r, F emit) {
             gs[g] = m;
         }
         __syncwarp();
-        for (int k = 0; k < r.keep; ++k) {
-            float v;
-            const int g = warp_argmax(gs, r.groups, &v);
-            __syncwarp();
-            if (lane == 0 && g < r.groups) gs[g] = -INFINITY;        // taken
-            __syncwarp();
-        }
         for (int i = lane; i < E; i += 32)
-            if (gs[i / size] != -INFINITY) z[i] = -INFINITY;         // not among the best
+            if (rank_of(gs, r.groups, i / size) >= r.keep) z[i] = -INFINITY;
         __syncwarp();
+    }
+    if (E <= kRankBy) {
+        for (int i = lane; i < E; i += 32) {
+            const int k = rank_of(z, E, i);
+            if (k < r.top) emit(k, i, expf(z[i] - top) / sum);
+        }
+        return;
     }
     for (int k = 0; k < r.top; ++k) {
         float v;
@@ -87,26 +100,47 @@ __device__ void choose(float* z, float* gs, const Router& r, F emit) {
         __syncwarp();
     }
 }
+// Sums over the warp of 32 values a lane holds: lane i receives value i's.
+__device__ __forceinline__ float warp_sums32(float (&v)[32]) {
+    const int lane = threadIdx.x & 31;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const bool up = lane & o;
+#pragma unroll
+        for (int i = 0; i < o; ++i) {
+            const float mine = up ? v[i + o] : v[i], other = up ? v[i] : v[i + o];
+            v[i] = mine + __shfl_xor_sync(0xffffffffu, other, o);
+        }
+    }
+    return v[0];
+}
 }  // namespace
 
-__global__ void __launch_bounds__(NT) route_rows_kernel(const RouteRows p) {
-    extern __shared__ __align__(16) float sm[];              // x [TOK][KC] | z [TOK][experts] | groups [TOK][groups]
+__global__ void __launch_bounds__(NT) route_rows_kernel(const RouteRows p, int kc) {
+    extern __shared__ __align__(16) float sm[];              // x [TOK][kc] | z [TOK][experts] | groups [TOK][groups]
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, E = p.r.experts, t0 = blockIdx.x * TOK, nt = min(TOK, p.M - t0);
     float* xs = sm;
-    float* z = sm + TOK * KC;
+    float* z = sm + TOK * kc;
     float* gs = z + TOK * E;
     for (int i = tid; i < TOK * E; i += NT) z[i] = 0.0f;
-    for (int k0 = 0; k0 < p.r.ld; k0 += KC) {
+    const bool vec = p.d % 4 == 0;
+    for (int k0 = 0; k0 < p.r.ld; k0 += kc) {                // all columns at once where they fit
         __syncthreads();
-        for (int i = tid; i < TOK * KC; i += NT) {
-            const int t = i / KC, k = i - t * KC;
-            xs[t * KC + spot(k)] = t < nt && k0 + k < p.d ? p.x[(size_t)(t0 + t) * p.d + k0 + k] : 0.0f;
+        for (int t = 0; t < TOK; ++t) {
+            const float* x = p.x + (size_t)(t0 + t) * p.d;
+            if (vec) {
+#pragma unroll 4
+                for (int k = tid * 4; k < kc; k += NT * 4)
+                    *(float4*)(xs + t * kc + spot(k)) = t < nt && k0 + k < p.d ? *(const float4*)(x + k0 + k) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            } else {
+                for (int k = tid; k < kc; k += NT) xs[t * kc + spot(k)] = t < nt && k0 + k < p.d ? x[k0 + k] : 0.0f;
+            }
         }
         __syncthreads();
         for (int e0 = warp * EPW; e0 < E; e0 += NT / 32 * EPW) {
-            float s[EPW][TOK] = {};
-#pragma unroll
-            for (int c = 0; c < KC; c += 256) {
+            float s[EPW * TOK] = {};
+#pragma unroll 2
+            for (int c = 0; c < kc; c += 256) {
                 const int k = k0 + c + lane * 8;
                 uint4 w[EPW];
 #pragma unroll
@@ -114,20 +148,14 @@ __global__ void __launch_bounds__(NT) route_rows_kernel(const RouteRows p) {
                     w[y] = e0 + y < E && k < p.r.ld ? __ldg((const uint4*)(p.r.w + (size_t)(e0 + y) * p.r.ld + k)) : make_uint4(0, 0, 0, 0);
 #pragma unroll
                 for (int t = 0; t < TOK; ++t) {
-                    const float4 u = *(const float4*)(xs + t * KC + c + lane * 4), v = *(const float4*)(xs + t * KC + c + lane * 4 + 128);
+                    const float4 u = *(const float4*)(xs + t * kc + c + lane * 4), v = *(const float4*)(xs + t * kc + c + lane * 4 + 128);
 #pragma unroll
-                    for (int y = 0; y < EPW; ++y) dot8(w[y], u, v, s[y][t]);
+                    for (int y = 0; y < EPW; ++y) dot8(w[y], u, v, s[y * TOK + t]);
                 }
             }
-#pragma unroll
-            for (int y = 0; y < EPW; ++y)
-#pragma unroll
-                for (int t = 0; t < TOK; ++t) {
-                    float v = s[y][t];
-#pragma unroll
-                    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-                    if (lane == 0 && e0 + y < E) z[t * E + e0 + y] += v;
-                }
+            static_assert(EPW * TOK == 32, "a sum a lane");
+            const float v = warp_sums32(s);
+            if (e0 + lane / TOK < E) z[(lane % TOK) * E + e0 + lane / TOK] += v;
         }
     }
     __syncthreads();
@@ -195,9 +223,10 @@ int max_row_tiles(const Router& r, int M, int tile_rows) {
 int launch_route_rows(const RouteRows& p, const void* plane, bool f32_rows, cudaStream_t st) {
     const Router& r = p.r;
     if (r.experts > kMaxExperts || r.groups > kMaxGroups || r.top > 64) return fail(FC_E_SHAPE, "%d experts in %d groups, %d chosen", r.experts, r.groups, r.top);
-    const size_t smem = (size_t)TOK * (KC + r.experts + r.groups) * sizeof(float);
-    if (smem > 47 * 1024) FC_CUDA(cudaFuncSetAttribute(route_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
-    route_rows_kernel<<<(p.M + TOK - 1) / TOK, NT, smem, st>>>(p);
+    const int rest = TOK * (r.experts + r.groups) * 4, kc = std::min(pad_to(r.ld, 256), (200 * 1024 - rest) / (TOK * 4) / 256 * 256);
+    const size_t smem = (size_t)TOK * kc * 4 + rest;
+    if (smem > 47 * 1024) FC_CUDA(cudaFuncSetAttribute(route_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+    route_rows_kernel<<<(p.M + TOK - 1) / TOK, NT, smem, st>>>(p, kc);
     FC_LAUNCHED();
     gather_rows_kernel<<<p.M, NT, (size_t)r.experts * sizeof(int), st>>>(p, (const unsigned char*)plane, p.ld * (f32_rows ? 4 : 2) / 16);
     FC_LAUNCHED();
@@ -218,21 +247,16 @@ __global__ void __launch_bounds__(NT) route_step_kernel(const __grid_constant__ 
     uint4 pre[8];
 #pragma unroll
     for (int c = 0; c < 8; ++c) pre[c] = c * 256 + lane * 8 < ld ? __ldg((const uint4*)(w + c * 256 + lane * 8)) : make_uint4(0, 0, 0, 0);
+    PostRow<NT, 4> row;
+    row.load(p.post.norm_w, d);
+    for (int c = d + tid; c < cap; c += NT) xs[spot(c)] = 0.0f;
     pdl_wait();
     pdl_trigger();
     if (p.state->done | p.state->error) return;
-    float yy = 0.0f;
-    for (int c = tid; c < cap; c += NT) {
-        const float y = c < d ? post_norm_sum(p.post, 0, c, d) : 0.0f;
-        xs[spot(c)] = y;
-        yy = fmaf(y, y, yy);
-    }
-    const float inv = 1.0f / sqrtf(block_sum_of<NT>(yy, red) / (float)d + p.eps);
-    for (int c = tid; c < d; c += NT) {
-        const float x = fmaf(xs[spot(c)] * inv, p.post.norm_w[c], p.x_in[c]);
+    row.run(p.post, p.x_in, d, p.eps, [&](int c, float x) {
         xs[spot(c)] = x;
         if (blockIdx.x == 0) p.x_out[c] = x;
-    }
+    }, [&](float v) { return block_sum_of<NT>(v, red); }, [&](int c) -> float& { return xs[spot(c)]; });
     __syncthreads();
     float s = 0.0f;
 #pragma unroll

@@ -17,6 +17,7 @@
 
 #include "bf16_ops.cuh"
 #include "pdl.cuh"
+#include "post_norm.cuh"
 #include "tc_common.cuh"
 
 namespace fc {
@@ -87,7 +88,7 @@ __global__ void __launch_bounds__(NT, 1) gemv_bf16_group_kernel(const __grid_con
         pieces = (K_pad + PIECE - 1) / PIECE;
         lc = K_pad > 1024 ? 3 : (K_pad > 512 ? 2 : (K_pad > 256 ? 1 : 0));
         const int rp = 8 >> lc, mine = end - row - warp * rp;
-        if (s.index && !ready) return;             // loaded after the wait
+        if (s.index && !s.early && !ready) return;             // loaded after the wait
         base = s.w + (size_t)row * ldw;
         if (s.index) base += (size_t)*s.index * s.w_step;
         items = mine > 0 ? (mine + NW * rp - 1) / (NW * rp) * pieces : 0;
@@ -104,30 +105,23 @@ __global__ void __launch_bounds__(NT, 1) gemv_bf16_group_kernel(const __grid_con
     open();
     load(pa, 0);
     load(pb, 1);
+    PostRow<NT, 2> post_row;
+    if (g.mode >= 3) post_row.load(g.post.norm_w, d);
     pdl_wait();
     pdl_trigger();
     if (g.state->done | g.state->error) return;
     ready = true;
-    if (seg < g.n_seg && g.seg[seg].index) { open(); load(pa, 0); load(pb, 1); }
+    if (seg < g.n_seg && g.seg[seg].index && !g.seg[seg].early) { open(); load(pa, 0); load(pb, 1); }
 
     if (g.mode != 0) {
         const int pos = g.state->pos;
         float ss = 0.0f;
         const bool post = g.mode >= 3;
         if (post && g.post.y) {
-            float yy = 0.0f;
-            for (int c = tid; c < d; c += NT) {
-                const float y = post_norm_sum(g.post, 0, c, d);
-                hs[c] = y;
-                yy = fmaf(y, y, yy);
-            }
-            const float iy = 1.0f / sqrtf(block_sum2(yy, 0.0f, red).x / (float)d + g.eps);
-            for (int c = tid; c < d; c += NT) {
-                const float x = fmaf(hs[c] * iy, g.post.norm_w[c], g.x_in[c]);
+            ss = post_row.run(g.post, g.x_in, d, g.eps, [&](int c, float x) {
                 if (blockIdx.x == 0 && g.x_out) g.x_out[c] = x;
                 hs[c] = x;
-                ss = fmaf(x, x, ss);
-            }
+            }, [&](float v) { return block_sum2(v, 0.0f, red).x; }, [&](int c) -> float& { return hs[c]; });
         } else
         if (g.prev.outs) {
             const float* lo = g.prev.outs;

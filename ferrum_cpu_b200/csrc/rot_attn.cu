@@ -37,13 +37,14 @@ __global__ void __launch_bounds__(NT) rot_prep_kernel(const RotAttn t, const flo
     __syncthreads();
     qi *= t.scale * factor;
     auto head = [&](const float* x, const float* w, float inv, int width, T* out) {      // two elements a thread
-        const int units = t.kp / 2;
-        for (int i = tid; i < width * units; i += NT) {
-            const int h = i / units, e = 2 * (i - h * units);
+        for (int h = tid >> 5; h < width; h += NT / 32) {
             auto at = [&](int k) { return x[h * dim + k] * (w ? w[h * dim + k] : 1.0f); };
-            const float a = e < dim ? rotated(t.rot.neighbours, t.rot.dims, cs, e, at) * inv : 0.0f;
-            const float b = e + 1 < dim ? rotated(t.rot.neighbours, t.rot.dims, cs, e + 1, at) * inv : 0.0f;
-            put_pair(out + (size_t)h * t.kp + e, a, b);
+#pragma unroll 2
+            for (int e = (tid & 31) * 2; e < t.kp; e += 64) {
+                const float a = e < dim ? rotated(t.rot.neighbours, t.rot.dims, cs, e, at) * inv : 0.0f;
+                const float b = e + 1 < dim ? rotated(t.rot.neighbours, t.rot.dims, cs, e + 1, at) * inv : 0.0f;
+                put_pair(out + (size_t)h * t.kp + e, a, b);
+            }
         }
     };
     head(src, t.q_norm, qi, t.H, q + (size_t)row * t.H * t.kp);
@@ -87,9 +88,9 @@ __global__ void __launch_bounds__(NT) latent_prep_kernel(const LatentAttn t, con
     const float inv = 1.0f / sqrtf(block_sum_of<NT>(s, red) / (float)t.rank + t.eps);      // also the barrier behind cs
     const float qs = t.scale * factor;
     T* out = q + (size_t)row * t.H * wq;
-    const int units = wq / 2;
-    for (int i = tid; i < t.H * units; i += NT) {
-        const int h = i / units, e0 = 2 * (i - h * units);
+    for (int h = tid >> 5; h < t.H; h += NT / 32)
+#pragma unroll 2
+    for (int e0 = (tid & 31) * 2; e0 < wq; e0 += 64) {
         const float* x = src + (size_t)h * hq;
         float v[2];
 #pragma unroll

@@ -451,7 +451,7 @@ fc_decoder_cache* Zogevik::make_cache() { return new ZogevikCache(); }
 AttnDecode ZogevikCache::attend(int l) const {
     const Layer& w = layer(l);
     AttnDecode a;
-    a.H = w.H(); a.f32 = m->f32; a.window = w.window(); a.max_splits = max_splits;
+    a.H = w.H(); a.f32 = m->f32; a.window = w.window(); a.max_splits = max_splits; a.reach = std::min(w.window(), m->ctx);
     a.part = part; a.part_ml = part_ml; a.state = state;
     a.k_ld = w.row;
     if (w.latent) {
@@ -557,7 +557,7 @@ int Zogevik::step(fc_decoder_cache* sc, bool with_head) {
             u.epi = ROW_GELU; u.index = s->expert + k; u.w_step = (size_t)w.ff * w.up.K_pad;
             down.x[k] = s->hid + (size_t)k * w.down.K_pad;
             GemvSeg& v = add(down, w.down.w, w.down.K_pad, d, w.ff, k, s->y + (size_t)k * d);
-            v.index = s->expert + k; v.w_step = (size_t)d * w.down.K_pad;
+            v.index = s->expert + k; v.w_step = (size_t)d * w.down.K_pad; v.early = 1;
         }
         FC_TRY(launch_gemv_bf16_group(up, st));
         FC_TRY(launch_gemv_bf16_group(down, st));
