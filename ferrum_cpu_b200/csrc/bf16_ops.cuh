@@ -193,20 +193,24 @@ int launch_wkv_finish(const float* o, int ldo, const float* gate, int ldg, const
 // prologue, or x[src]).
 struct GemvSeg {
     const uint16_t* w;    // first row; rows ldw apart, K_pad weights of each (a multiple of 64), K inputs
-    const int* index;     // not null: the rows begin *index * w_step weights further on (an expert chosen on the device)
-    size_t w_step;
-    int early;            // the index was there before the kernel ahead began (its own wait is behind this one's launch)
     int n, ldw, K_pad, src, K;
     float* y;
     int epi;
     float c0, c1;
-    long long cost0;      // filled by the launcher
+    // the product again with other weights (experts chosen on the device): rep r reads the rows index[r] * w_step weights further on
+    // and the input x_step * r values further on (mode 0), and writes y_step * r values further on
+    int reps;             // 0 or 1: once
+    const int* index;
+    size_t w_step;
+    int x_step, y_step;
+    int early;            // the indices were there before the kernel ahead began (its own wait is behind this one's launch)
+    int cost0, cost;      // filled by the launcher
 };
-constexpr int kGemvSegs = 32, kGemvInputs = 32;
+constexpr int kGemvSegs = 16;
 struct GemvGroup {
     GemvSeg seg[kGemvSegs];
     int n_seg;
-    const float* x[kGemvInputs];       // plain inputs (mode 0)
+    const float* x[8];                 // plain inputs (mode 0)
     int mode;                          // 0: plain inputs; 1: residual + norm + mixes of the row; 2: residual + norm;
                                        // 3: residual of PostNorm; 4: the same and a norm (norm_w)
     PostNorm post;                     // modes 3 and 4 (x_in, x_out, queue and embed as in the others)
@@ -218,7 +222,7 @@ struct GemvGroup {
     float* shift; size_t shift_slot;   // two slots of h, read at position parity, written at the other
     int d;
     StepState* state;
-    long long total_cost;
+    int share, rest;      // filled by the launcher: cost of a CTA, and what the division leaves
 };
 int launch_gemv_bf16_group(GemvGroup g, cudaStream_t st);
 

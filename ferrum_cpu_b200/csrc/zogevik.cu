@@ -16,7 +16,7 @@ using namespace fc;
 namespace {
 
 constexpr int kOutSplits = 4;           // most partial sums of the mixer's output product
-constexpr int kMaxTop = 24;             // most experts a token uses (segments of one decode product)
+constexpr int kMaxTop = 64;             // most experts a token uses
 
 // The entries of config.json for one layer.
 struct LayerCfg {
@@ -552,13 +552,11 @@ int Zogevik::step(fc_decoder_cache* sc, bool with_head) {
         FC_TRY(launch_route_step(r, st));
         GemvGroup up = base, down = base;
         up.x[0] = s->x[cur];
-        for (int k = 0; k < w.router.top; ++k) {
-            GemvSeg& u = add(up, w.up.w, w.up.K_pad, w.ff, d, 0, s->hid + (size_t)k * w.down.K_pad);
-            u.epi = ROW_GELU; u.index = s->expert + k; u.w_step = (size_t)w.ff * w.up.K_pad;
-            down.x[k] = s->hid + (size_t)k * w.down.K_pad;
-            GemvSeg& v = add(down, w.down.w, w.down.K_pad, d, w.ff, k, s->y + (size_t)k * d);
-            v.index = s->expert + k; v.w_step = (size_t)d * w.down.K_pad; v.early = 1;
-        }
+        down.x[0] = s->hid;
+        GemvSeg& u = add(up, w.up.w, w.up.K_pad, w.ff, d, 0, s->hid);
+        u.epi = ROW_GELU; u.reps = w.router.top; u.index = s->expert; u.w_step = (size_t)w.ff * w.up.K_pad; u.y_step = w.down.K_pad;
+        GemvSeg& v = add(down, w.down.w, w.down.K_pad, d, w.ff, 0, s->y);
+        v.reps = w.router.top; v.index = s->expert; v.w_step = (size_t)d * w.down.K_pad; v.x_step = w.down.K_pad; v.y_step = d; v.early = 1;
         FC_TRY(launch_gemv_bf16_group(up, st));
         FC_TRY(launch_gemv_bf16_group(down, st));
         prev = PostNorm();
