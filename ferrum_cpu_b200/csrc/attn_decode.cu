@@ -13,6 +13,8 @@
 // of earlier tokens and weights are asked for before the wait.
 //
 // Bound: HBM / latency (cached rows once per block of heads, W_uk and W_uv once).
+#include <cooperative_groups.h>
+
 #include <algorithm>
 
 #include "pdl.cuh"
@@ -145,7 +147,6 @@ __global__ void __launch_bounds__(NT) attn_decode_kernel(const __grid_constant__
         }
     };
     if (live) stage(r.begin, r.begin, min(min(r.end, r.begin + l.kt), pos));
-    for (int i = tid; i < l.nkp * l.hb4 * l.vw4; i += NT) acc[i] = 0.0f;
     for (int i = tid; i < l.hb4; i += NT) { ml[3 * i] = -1e30f; ml[3 * i + 1] = 0.0f; ml[3 * i + 2] = 0.0f; }
     for (int i = tid; i < t.rot.dims / 2; i += NT) cs[i] = rot_cs(pos, t.rot.freq[i]);
     pdl_wait();
@@ -162,11 +163,12 @@ __global__ void __launch_bounds__(NT) attn_decode_kernel(const __grid_constant__
             inv = t.scale / sqrtf(block_sum_of<NT>(s, red) / (float)qn + t.eps);
         }
         __syncthreads();                           // cs
-        for (int i = tid; i < l.hb4 * kw; i += NT) {
-            const int h = i / kw, e = i - h * kw;
+        for (int h = warp; h < l.hb4; h += NT / 32) {
             const float* x = a.q + (size_t)(h0 + h) * t.dim;
             const float* w = t.q_norm + (size_t)(h0 + h) * t.dim;
-            q[i] = h < nh && e < t.dim ? rotated(t.rot.neighbours, t.rot.dims, cs, e, [&](int k) { return x[k] * (t.q_norm ? w[k] : 1.0f); }) * inv : 0.0f;
+#pragma unroll 4
+            for (int e = lane; e < kw; e += 32)
+                q[h * kw + e] = h < nh && e < t.dim ? rotated(t.rot.neighbours, t.rot.dims, cs, e, [&](int k) { return x[k] * (t.q_norm ? w[k] : 1.0f); }) * inv : 0.0f;
         }
         if (own && t.own_kv) {
             float ki = 1.0f;
@@ -191,10 +193,14 @@ __global__ void __launch_bounds__(NT) attn_decode_kernel(const __grid_constant__
             }
         }
     } else {
-        for (int i = tid; i < l.hb4 * kw; i += NT) { const int h = i / kw; q[i] = h < nh ? a.q[(size_t)h0 * kw + i] : 0.0f; }
+        const float4* src = (const float4*)(a.q + (size_t)h0 * kw);      // kw is a multiple of 8
+#pragma unroll 4
+        for (int i = tid; i < l.hb4 * kw / 4; i += NT) ((float4*)q)[i] = i < nh * kw / 4 ? src[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     }
     const bool self = own && t.H && t.own_kv;      // the own row does not come from the cache when one tile holds the split
     const int ng = l.hb4 / PER, pst = l.hb4 + 4;
+    // one tile, one piece of its rows, and splits to be merged: the values go from the registers to where they are merged
+    const bool straight = r.end - r.begin <= l.kt && l.nkp == 1 && !(a.counter && r.splits == 1);
     for (int k0 = r.begin; k0 < r.end; k0 += l.kt) {
         const int nk = min(l.kt, r.end - k0);
         if (k0 > r.begin) {
@@ -297,9 +303,17 @@ __global__ void __launch_bounds__(NT) attn_decode_kernel(const __grid_constant__
 #pragma unroll
             for (int y = 0; y < PER; ++y) {
                 const int h = g * PER + y;
-                const float corr = ml[3 * h + 2];
+                if (straight) {
+                    if (h < nh) *(float2*)(a.part + ((size_t)blockIdx.x * a.H + h0 + h) * l.vw4 + 2 * u) = make_float2(o[y][0], o[y][1]);
+                    continue;
+                }
                 float2* to = (float2*)(acc + ((size_t)s * l.hb4 + h) * l.vw4 + 2 * u);
-                *to = make_float2(fmaf(to->x, corr, o[y][0]), fmaf(to->y, corr, o[y][1]));
+                if (k0 == r.begin) {
+                    *to = make_float2(o[y][0], o[y][1]);
+                } else {
+                    const float corr = ml[3 * h + 2];
+                    *to = make_float2(fmaf(to->x, corr, o[y][0]), fmaf(to->y, corr, o[y][1]));
+                }
             }
         }
     }
@@ -318,10 +332,11 @@ __global__ void __launch_bounds__(NT) attn_decode_kernel(const __grid_constant__
         return;
     }
     const size_t sp = blockIdx.x;
-    for (int i = tid; i < nh * l.vw4; i += NT) {
-        const int h = i / l.vw4, e = i - h * l.vw4;
-        a.part[(sp * a.H + h0 + h) * l.vw4 + e] = e < vw ? total(h, e) : 0.0f;
-    }
+    if (!straight || !live)
+        for (int i = tid; i < nh * l.vw4; i += NT) {
+            const int h = i / l.vw4, e = i - h * l.vw4;
+            a.part[(sp * a.H + h0 + h) * l.vw4 + e] = live && e < vw ? total(h, e) : 0.0f;
+        }
     for (int h = tid; h < nh; h += NT) {
         a.part_ml[(sp * a.H + h0 + h) * 2] = ml[3 * h];
         a.part_ml[(sp * a.H + h0 + h) * 2 + 1] = ml[3 * h + 1];
@@ -445,46 +460,55 @@ int launch_latent_absorb(const LatentAttn& t, const float* proj, float* q, void*
 }
 
 namespace {
-constexpr int VC = 32;                                  // value rows of a CTA
+constexpr int VC = 32, kMaxCluster = 8;                 // value rows of a CTA; CTAs of a head
 }
+// The CTAs of a head form a cluster: each merges a share of the latents and hands it to the others' shared memory, then
+// multiplies its own value rows.
 __global__ void __launch_bounds__(NT) latent_expand_kernel(const LatentAttn t, const __grid_constant__ AttnDecode a, int kt, float* __restrict__ out) {
-    extern __shared__ __align__(16) float smf[];        // sum of latents [lat], then partial sums
+    extern __shared__ __align__(16) float smf[];        // sum of latents [lat], partial sums [4 NT]
     __shared__ float wgt[kMaxSplitsRow];
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, v0 = blockIdx.x * VC, nv = min(VC, t.vdim - v0);
+    namespace cg = cooperative_groups;
+    cg::cluster_group cluster = cg::this_cluster();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, n = gridDim.x, v0 = blockIdx.x * VC, nv = min(VC, t.vdim - v0);
     const uint16_t* w = t.uv + ((size_t)h * t.vp + v0) * t.lat;
     for (int i = tid * 64; i < nv * t.lat; i += NT * 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(w + i));
+    for (int i = t.rank + tid; i < t.lat; i += NT) smf[i] = 0.0f;
     const Range r = range_of(a.state->pos + 1, a.window, kt, a.max_splits, 0);
     pdl_wait();
     pdl_trigger();
-    if (a.state->done | a.state->error) return;
+    if (a.state->done | a.state->error) return;         // the same in every CTA
     if (warp == 0) {
         float x[2];
         split_weights(a.part_ml, a.H, h, r.splits, a.has_sink, x);
         wgt[lane] = x[0];
         wgt[lane + 32] = x[1];
     }
-    __syncthreads();
+    cluster.sync();                                     // weights; every CTA of the cluster runs
     // four latents a thread, the splits dealt out over what is left of the block
-    const int vw4 = (a.vw + 3) / 4 * 4, n4 = vw4 / 4, lanes = max(1, NT / n4);
-    float* part = smf + t.lat;                          // [lanes][lat]
-    for (int i = tid; i < n4 * lanes; i += NT) {
-        const int sg = i / n4, r4 = (i - sg * n4) * 4;
-        float4 o = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    const int vw4 = (a.vw + 3) / 4 * 4, n4 = vw4 / 4, u0 = n4 * (int)blockIdx.x / n, u1 = n4 * ((int)blockIdx.x + 1) / n;
+    float* part = smf + t.lat;
+    for (int ub = u0; ub < u1; ub += NT) {
+        const int nu = min(NT, u1 - ub), lanes = NT / nu, sg = tid / nu, u = tid - sg * nu;
+        if (sg < lanes) {
+            float4 o = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll 8
-        for (int s = sg; s < r.splits; s += lanes) {
-            const float4 x = __ldcg((const float4*)(a.part + ((size_t)s * a.H + h) * vw4 + r4));
-            o.x = fmaf(wgt[s], x.x, o.x); o.y = fmaf(wgt[s], x.y, o.y); o.z = fmaf(wgt[s], x.z, o.z); o.w = fmaf(wgt[s], x.w, o.w);
+            for (int s = sg; s < r.splits; s += lanes) {
+                const float4 x = __ldcg((const float4*)(a.part + ((size_t)s * a.H + h) * vw4 + (ub + u) * 4));
+                o.x = fmaf(wgt[s], x.x, o.x); o.y = fmaf(wgt[s], x.y, o.y); o.z = fmaf(wgt[s], x.z, o.z); o.w = fmaf(wgt[s], x.w, o.w);
+            }
+            *(float4*)(part + (sg * nu + u) * 4) = o;
         }
-        *(float4*)(part + (size_t)sg * t.lat + r4) = o;
+        __syncthreads();
+        for (int i = tid; i < nu * 4; i += NT) {
+            float o = 0.0f;
+            for (int s = 0; s < lanes; ++s) o += part[s * nu * 4 + i];
+            const int at = ub * 4 + i;
+            if (at < t.rank)
+                for (int c = 0; c < n; ++c) cluster.map_shared_rank(smf, c)[at] = o;
+        }
+        __syncthreads();
     }
-    __syncthreads();
-    for (int i = tid; i < t.lat; i += NT) {
-        float o = 0.0f;
-        if (i < t.rank)
-            for (int s = 0; s < lanes; ++s) o += part[(size_t)s * t.lat + i];
-        smf[i] = o;
-    }
-    __syncthreads();
+    cluster.sync();
 #pragma unroll 4
     for (int v = warp; v < nv; v += NT / 32) {
         float s = 0.0f;
@@ -502,11 +526,11 @@ __global__ void __launch_bounds__(NT) latent_expand_kernel(const LatentAttn t, c
 int launch_latent_expand(const LatentAttn& t, const AttnDecode& a, float* out, cudaStream_t st) {
     Plan l;
     FC_TRY(make_plan(a, &l));
-    const int n4 = (a.vw + 3) / 4, lanes = std::max(1, NT / n4);
-    const size_t smem = (size_t)(1 + lanes) * t.lat * 4 + 16;
-    if (smem > 200 * 1024) return fail(FC_E_SHAPE, "latents of %d values", t.rank);
+    const int n = (t.vdim + VC - 1) / VC;
+    const size_t smem = (size_t)(t.lat + 4 * NT) * 4;
+    if (n > kMaxCluster || smem > 200 * 1024) return fail(FC_E_SHAPE, "latents of %d values, value heads of %d", t.rank, t.vdim);
     if (smem > 47 * 1024) FC_CUDA(cudaFuncSetAttribute(latent_expand_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    FC_CUDA(launch_pdl(latent_expand_kernel, dim3((t.vdim + VC - 1) / VC, t.H), dim3(NT), smem, st, t, a, l.kt, out));
+    FC_CUDA(launch_pdl_cluster(latent_expand_kernel, dim3(n, t.H), dim3(NT), n, smem, st, t, a, l.kt, out));
     ++g_launches;
     return FC_OK;
 }
