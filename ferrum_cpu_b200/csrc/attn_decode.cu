@@ -159,6 +159,7 @@ __global__ void __launch_bounds__(NT) attn_decode_kernel(const __grid_constant__
         float inv = t.scale;
         if (t.q_norm) {
             float s = 0.0f;
+#pragma unroll 8
             for (int i = tid; i < qn; i += NT) s = fmaf(a.q[i], a.q[i], s);
             inv = t.scale / sqrtf(block_sum_of<NT>(s, red) / (float)qn + t.eps);
         }

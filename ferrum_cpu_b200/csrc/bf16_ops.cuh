@@ -197,16 +197,20 @@ struct GemvSeg {
     float* y;
     int epi;
     float c0, c1;
-    // the product again with other weights (experts chosen on the device): rep r reads the rows index[r] * w_step weights further on
-    // and the input x_step * r values further on (mode 0), and writes y_step * r values further on
+    // the product again with the weights of every chosen expert (GemvGroup): rep r reads the rows expert * w_step weights
+    // further on and the input x_step * r values further on, and writes y_step * r values further on. sum: one row of results
+    // instead, the sum over the repetitions with the experts' weights (w_step a multiple of 64).
     int reps;             // 0 or 1: once
-    const int* index;
+    int sum;
     size_t w_step;
     int x_step, y_step;
-    int early;            // the indices were there before the kernel ahead began (its own wait is behind this one's launch)
     int cost0, cost;      // filled by the launcher
 };
 constexpr int kGemvSegs = 16;
+struct Router {
+    int experts = 0, top = 0, groups = 1, keep = 1;
+    const uint16_t* w = nullptr; int ld = 0;         // [experts][ld]
+};
 struct GemvGroup {
     GemvSeg seg[kGemvSegs];
     int n_seg;
@@ -221,6 +225,9 @@ struct GemvGroup {
     const float* mu[kMixes];
     float* shift; size_t shift_slot;   // two slots of h, read at position parity, written at the other
     int d;
+    // experts > 0 (mode 0): the segments' experts are chosen from the logits z and left in expert / weight [top]; a segment that
+    // is a sum reads these instead
+    Router router; const float* z; int* expert; float* weight;
     StepState* state;
     int share, rest;      // filled by the launcher: cost of a CTA, and what the division leaves
 };
@@ -293,10 +300,6 @@ int attn_decode_blocks(const AttnDecode& a);         // blocks of heads: counter
 int launch_latent_expand(const LatentAttn& t, const AttnDecode& a, float* out, cudaStream_t st);
 
 // ---- experts.cu: routed feed-forwards -----------------------------------------------------------------
-struct Router {
-    int experts = 0, top = 0, groups = 1, keep = 1;
-    const uint16_t* w = nullptr; int ld = 0;         // [experts][ld]
-};
 // Routes M rows of x (f32, d apart; the same as operand rows in `plane`, ld apart): chosen expert and weight (softmax over all
 // experts, not renormalised) of every slot, the places of the slots' rows once they are grouped by expert, those rows (bf16 or
 // f32, ld apart) and the row tiles of the products. counts starts as zeros.
@@ -309,16 +312,6 @@ struct RouteRows {
 };
 int max_row_tiles(const Router& r, int M, int tile_rows);
 int launch_route_rows(const RouteRows& p, const void* plane, bool f32_rows, cudaStream_t st);
-// One token: the residual before it (PostNorm), logits, choice. expert / weight [top]; scratch: logits [experts] and a counter.
-struct RouteStep {
-    Router r;
-    PostNorm post; const float* x_in; float* x_out; float eps; int d;
-    float* z; unsigned int* counter;
-    int* expert; float* weight;
-    const StepState* state;
-};
-int launch_route_step(const RouteStep& p, cudaStream_t st);
-
 // mixer_decode.cu: attention splits and recurrence heads of one token in one launch.
 struct MixerDecode {
     TalkAttn t;

@@ -6,21 +6,18 @@
 //                        place within its expert from an atomic counter (the order of an expert's rows does not matter)
 //   gather_rows_kernel   a CTA per token: places become rows (prefix sums of the counts), its operand row copied to each; the
 //                        first CTA writes the table of row tiles
-//   route_step_kernel    one token: residual and norm ahead of it, a warp per expert, the last CTA to finish chooses
-// The products themselves: launch_gemm_bf16_ragged (portions), launch_gemv_bf16_group with indexed segments (one token).
+// The products themselves: launch_gemm_bf16_ragged. One token: launch_gemv_bf16_group, for the logits, the first matrices (whose
+// launch chooses) and the second (whose rows run through all chosen experts).
 //
 // Bound: fp32 FMA (2 experts d FLOP per token) and L2; the gather HBM / L2.
 #include <algorithm>
 
-#include "pdl.cuh"
-#include "post_norm.cuh"
-#include "rot_rows.cuh"
+#include "route.cuh"
 
 namespace fc {
 
 namespace {
 constexpr int NT = 256, TOK = 8, EPW = 4;      // tokens a CTA, experts a warp holds at once
-constexpr int kMaxExperts = 1024, kMaxGroups = 256;
 
 // Place of column k in shared memory: within 256 values, lane l's eight are two float4 at 4 l and 128 + 4 l.
 __device__ __forceinline__ int spot(int k) {
@@ -32,73 +29,6 @@ __device__ __forceinline__ void dot8(const uint4& w, const float4& u, const floa
     s = fmaf(__uint_as_float(w.y << 16), u.z, s); s = fmaf(__uint_as_float(w.y & 0xffff0000u), u.w, s);
     s = fmaf(__uint_as_float(w.z << 16), v.x, s); s = fmaf(__uint_as_float(w.z & 0xffff0000u), v.y, s);
     s = fmaf(__uint_as_float(w.w << 16), v.z, s); s = fmaf(__uint_as_float(w.w & 0xffff0000u), v.w, s);
-}
-// The place and value of the largest entry (the first of equals), in every lane. n may exceed what a lane sees.
-__device__ __forceinline__ int warp_argmax(const float* z, int n, float* best) {
-    const int lane = threadIdx.x & 31;
-    float b = -INFINITY;
-    int at = 1 << 30;
-    for (int i = lane; i < n; i += 32)
-        if (z[i] > b) { b = z[i]; at = i; }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-        const float ob = __shfl_xor_sync(0xffffffffu, b, o);
-        const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-        if (ob > b || (ob == b && oa < at)) { b = ob; at = oa; }
-    }
-    *best = b;
-    return at;
-}
-// One warp chooses from logits z (overwritten) of a token; gs: room for the groups' scores. emit(slot, expert, weight) runs in
-// one lane per slot. Softmax keeps the logits' order, so they are compared in its place; of equals the first counts as larger.
-// Few entries are ranked by counting those ahead of each, more are taken one by one.
-constexpr int kRankBy = 128;
-__device__ __forceinline__ int rank_of(const float* z, int n, int i) {
-    const float v = z[i];
-    int ahead = 0;
-#pragma unroll 8
-    for (int k = 0; k < n; ++k) ahead += z[k] > v || (z[k] == v && k < i);
-    return ahead;
-}
-template <class F>
-__device__ void choose(float* z, float* gs, const Router& r, F emit) {
-    const int lane = threadIdx.x & 31, E = r.experts;
-    for (int i = lane; i < E; i += 32)
-        if (z[i] != z[i]) z[i] = -INFINITY;                          // what is not a number comes last: every slot gets an expert
-    __syncwarp();
-    float top;
-    warp_argmax(z, E, &top);
-    float sum = 0.0f;
-    for (int i = lane; i < E; i += 32) sum += expf(z[i] - top);
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-    if (r.keep < r.groups) {
-        const int size = E / r.groups;
-        for (int g = lane; g < r.groups; g += 32) {
-            float m = -INFINITY;
-            for (int i = 0; i < size; ++i) m = fmaxf(m, z[g * size + i]);
-            gs[g] = m;
-        }
-        __syncwarp();
-        for (int i = lane; i < E; i += 32)
-            if (rank_of(gs, r.groups, i / size) >= r.keep) z[i] = -INFINITY;
-        __syncwarp();
-    }
-    if (E <= kRankBy) {
-        for (int i = lane; i < E; i += 32) {
-            const int k = rank_of(z, E, i);
-            if (k < r.top) emit(k, i, expf(z[i] - top) / sum);
-        }
-        return;
-    }
-    for (int k = 0; k < r.top; ++k) {
-        float v;
-        int e = warp_argmax(z, E, &v);
-        if (e >= E) e = 0;                                           // only where logits are not numbers
-        __syncwarp();
-        if (lane == 0) { z[e] = -INFINITY; emit(k, e, expf(v - top) / sum); }
-        __syncwarp();
-    }
 }
 // Sums over the warp of 32 values a lane holds: lane i receives value i's.
 __device__ __forceinline__ float warp_sums32(float (&v)[32]) {
@@ -230,67 +160,6 @@ int launch_route_rows(const RouteRows& p, const void* plane, bool f32_rows, cuda
     FC_LAUNCHED();
     gather_rows_kernel<<<p.M, NT, (size_t)r.experts * sizeof(int), st>>>(p, (const unsigned char*)plane, p.ld * (f32_rows ? 4 : 2) / 16);
     FC_LAUNCHED();
-    return FC_OK;
-}
-
-// ------------------------------------------------------------------------------------------------ one token
-__global__ void __launch_bounds__(NT) route_step_kernel(const __grid_constant__ RouteStep p) {
-    extern __shared__ __align__(16) float sm[];              // x [ld up to 256s] | z [experts] | groups
-    __shared__ float red[NT / 32];
-    __shared__ bool is_last;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, d = p.d, E = p.r.experts, ld = p.r.ld, cap = (ld + 255) / 256 * 256;
-    float* xs = sm;
-    float* z = sm + cap;
-    float* gs = z + E;
-    const int e = blockIdx.x * (NT / 32) + warp;
-    const uint16_t* w = p.r.w + (size_t)min(e, E - 1) * ld;
-    uint4 pre[8];
-#pragma unroll
-    for (int c = 0; c < 8; ++c) pre[c] = c * 256 + lane * 8 < ld ? __ldg((const uint4*)(w + c * 256 + lane * 8)) : make_uint4(0, 0, 0, 0);
-    PostRow<NT, 4> row;
-    row.load(p.post.norm_w, d);
-    for (int c = d + tid; c < cap; c += NT) xs[spot(c)] = 0.0f;
-    pdl_wait();
-    pdl_trigger();
-    if (p.state->done | p.state->error) return;
-    row.run(p.post, p.x_in, d, p.eps, [&](int c, float x) {
-        xs[spot(c)] = x;
-        if (blockIdx.x == 0) p.x_out[c] = x;
-    }, [&](float v) { return block_sum_of<NT>(v, red); }, [&](int c) -> float& { return xs[spot(c)]; });
-    __syncthreads();
-    float s = 0.0f;
-#pragma unroll
-    for (int c = 0; c < 8; ++c)
-        if (c * 256 < ld) dot8(pre[c], *(const float4*)(xs + c * 256 + lane * 4), *(const float4*)(xs + c * 256 + lane * 4 + 128), s);
-    for (int c = 8; c * 256 < ld; ++c)
-        if (c * 256 + lane * 8 < ld)
-            dot8(__ldg((const uint4*)(w + c * 256 + lane * 8)), *(const float4*)(xs + c * 256 + lane * 4), *(const float4*)(xs + c * 256 + lane * 4 + 128), s);
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-    if (lane == 0 && e < E) p.z[e] = s;
-    __threadfence();
-    __syncthreads();
-    if (tid == 0) is_last = atomicAdd(p.counter, 1u) == gridDim.x - 1;
-    __syncthreads();
-    if (!is_last) return;
-    __threadfence();
-    if (tid == 0) *p.counter = 0;
-    for (int i = tid; i < E; i += NT) z[i] = __ldcg(p.z + i);
-    __syncthreads();
-    if (warp == 0)
-        choose(z, gs, p.r, [&](int k, int x, float v) {
-            p.expert[k] = x;
-            p.weight[k] = v;
-        });
-}
-int launch_route_step(const RouteStep& p, cudaStream_t st) {
-    const Router& r = p.r;
-    if (r.experts > kMaxExperts || r.groups > kMaxGroups) return fail(FC_E_SHAPE, "%d experts in %d groups", r.experts, r.groups);
-    const size_t smem = (size_t)((r.ld + 255) / 256 * 256 + r.experts + r.groups) * sizeof(float);
-    if (smem > 200 * 1024) return fail(FC_E_SHAPE, "rows of %d values exceed the router's staging", p.d);
-    if (smem > 47 * 1024) FC_CUDA(cudaFuncSetAttribute(route_step_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    FC_CUDA(launch_pdl(route_step_kernel, dim3((r.experts + NT / 32 - 1) / (NT / 32)), dim3(NT), smem, st, p));
-    ++g_launches;
     return FC_OK;
 }
 

@@ -75,7 +75,7 @@ struct ZogevikCache : fc_decoder_cache {
     float *x[2] = {}, *proj = nullptr, *q = nullptr, *att = nullptr, *outs = nullptr, *hid = nullptr, *y = nullptr, *z = nullptr, *weight = nullptr;
     float *part = nullptr, *part_ml = nullptr;
     int* expert = nullptr;
-    unsigned int* counter = nullptr;    // [0]: the router's, then one a block of heads
+    unsigned int* counter = nullptr;    // one a block of heads
     int max_splits = 1;
     int create() override;
     Layer& layer(int l) const { return *static_cast<Zogevik*>(m)->layers[l]; }
@@ -461,7 +461,7 @@ AttnDecode ZogevikCache::attend(int l) const {
         const RotAttn& t = w.att;
         const int from = w.kv_from < 0 ? l : w.kv_from;
         a.KV = t.KV; a.kw = t.kp; a.vw = t.vdim; a.k_head = t.kp; a.v_ld = w.vrow; a.v_head = t.vp;
-        a.kc = kc[from]; a.vc = vc[from]; a.prep = t; a.q = proj; a.has_sink = t.has_sink; a.out = att; a.counter = counter + 1;
+        a.kc = kc[from]; a.vc = vc[from]; a.prep = t; a.q = proj; a.has_sink = t.has_sink; a.out = att; a.counter = counter;
     }
     // splits of a tile each, but no more CTAs than two per SM
     a.max_splits = std::max(1, std::min(max_splits, 296 / attn_decode_blocks(a)));
@@ -495,13 +495,13 @@ int ZogevikCache::create() {
     FC_TRY(a.alloc_n(&att, (size_t)att_max));
     FC_TRY(a.alloc_n(&outs, (size_t)kOutSplits * d));
     FC_TRY(a.alloc_n(&hid, (size_t)std::max(n->max_ff_top, 1)));
-    FC_TRY(a.alloc_n(&y, (size_t)std::max(n->max_top, 1) * d));
+    FC_TRY(a.alloc_n(&y, (size_t)d));
     FC_TRY(a.alloc_n(&z, (size_t)std::max(n->max_experts, 1)));
     FC_TRY(a.alloc_n(&weight, (size_t)std::max(n->max_top, 1)));
     FC_TRY(n->zeroed_n(a, &expert, (size_t)std::max(n->max_top, 1)));
     FC_TRY(a.alloc_n(&part, (size_t)max_splits * part_max));
     FC_TRY(a.alloc_n(&part_ml, (size_t)max_splits * heads * 2));
-    return n->zeroed_n(a, &counter, (size_t)1 + blocks);
+    return n->zeroed_n(a, &counter, (size_t)blocks);
 }
 
 int Zogevik::step(fc_decoder_cache* sc, bool with_head) {
@@ -545,22 +545,24 @@ int Zogevik::step(fc_decoder_cache* sc, bool with_head) {
         prev = PostNorm();
         prev.y = s->outs; prev.n_parts = n; prev.part_rows = 1; prev.norm_w = w.norm1;
         if (!w.ff) continue;
-        RouteStep r = {};
-        r.r = w.router; r.post = prev; r.x_in = s->x[cur]; r.x_out = s->x[cur ^ 1]; r.eps = (float)eps; r.d = d;
-        r.z = s->z; r.counter = s->counter; r.expert = s->expert; r.weight = s->weight; r.state = s->state;
+        // logits on the residual; the first product chooses from them; rows of the second run through the chosen experts
+        GemvGroup r = base, up = base, down = base;
+        r.mode = 3; r.post = prev; r.x_in = s->x[cur]; r.x_out = s->x[cur ^ 1];
         cur ^= 1;
-        FC_TRY(launch_route_step(r, st));
-        GemvGroup up = base, down = base;
+        add(r, w.router.w, w.router.ld, w.router.experts, d, 0, s->z);
+        FC_TRY(launch_gemv_bf16_group(r, st));
         up.x[0] = s->x[cur];
-        down.x[0] = s->hid;
+        up.router = w.router; up.z = s->z;
+        up.expert = down.expert = s->expert; up.weight = down.weight = s->weight;
         GemvSeg& u = add(up, w.up.w, w.up.K_pad, w.ff, d, 0, s->hid);
-        u.epi = ROW_GELU; u.reps = w.router.top; u.index = s->expert; u.w_step = (size_t)w.ff * w.up.K_pad; u.y_step = w.down.K_pad;
-        GemvSeg& v = add(down, w.down.w, w.down.K_pad, d, w.ff, 0, s->y);
-        v.reps = w.router.top; v.index = s->expert; v.w_step = (size_t)d * w.down.K_pad; v.x_step = w.down.K_pad; v.y_step = d; v.early = 1;
+        u.epi = ROW_GELU; u.reps = w.router.top; u.w_step = (size_t)w.ff * w.up.K_pad; u.y_step = w.down.K_pad;
         FC_TRY(launch_gemv_bf16_group(up, st));
+        down.x[0] = s->hid;
+        GemvSeg& v = add(down, w.down.w, w.down.K_pad, d, w.ff, 0, s->y);
+        v.reps = w.router.top; v.sum = 1; v.w_step = (size_t)d * w.down.K_pad; v.x_step = w.down.K_pad;
         FC_TRY(launch_gemv_bf16_group(down, st));
         prev = PostNorm();
-        prev.y = s->y; prev.n_parts = w.router.top; prev.part_rows = 1; prev.weight = s->weight; prev.norm_w = w.norm2;
+        prev.y = s->y; prev.n_parts = 1; prev.part_rows = 1; prev.norm_w = w.norm2;
     }
     if (!with_head) return FC_OK;
     GemvGroup g = base;
