@@ -1,7 +1,8 @@
 // Routing of feed-forwards that are cut into experts: which experts a token uses and with what weight, and the rows of a
 // portion regrouped so that every expert's products read consecutive rows.
 //
-//   route_rows_kernel    8 tokens a CTA: logits in f32 (rows in shared memory, a warp holds four experts at a time), softmax
+//   route_rows_kernel    8 tokens a CTA: logits in f32 (rows in shared memory, a warp holds four experts at a time,
+//                        the block's halves every other 256 columns), softmax
 //                        over all experts, the best groups (a group's score is its largest), the best experts in them; a slot's
 //                        place within its expert from an atomic counter (the order of an expert's rows does not matter)
 //   gather_rows_kernel   a CTA per token: places become rows (prefix sums of the counts), its operand row copied to each; the
@@ -17,7 +18,7 @@
 namespace fc {
 
 namespace {
-constexpr int NT = 256, TOK = 8, EPW = 4;      // tokens a CTA, experts a warp holds at once
+constexpr int NT = 256, RT = 512, TOK = 8, EPW = 4;      // tokens a CTA, experts a warp holds at once
 
 // Place of column k in shared memory: within 256 values, lane l's eight are two float4 at 4 l and 128 + 4 l.
 __device__ __forceinline__ int spot(int k) {
@@ -46,13 +47,13 @@ __device__ __forceinline__ float warp_sums32(float (&v)[32]) {
 }
 }  // namespace
 
-__global__ void __launch_bounds__(NT) route_rows_kernel(const RouteRows p, int kc) {
-    extern __shared__ __align__(16) float sm[];              // x [TOK][kc] | z [TOK][experts] | groups [TOK][groups]
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, E = p.r.experts, t0 = blockIdx.x * TOK, nt = min(TOK, p.M - t0);
+__global__ void __launch_bounds__(RT) route_rows_kernel(const RouteRows p, int kc) {
+    extern __shared__ __align__(16) float sm[];              // x [TOK][kc] | z of either half [TOK][experts] | groups [TOK][groups]
+    const int tid = threadIdx.x, lane = tid & 31, half = tid / (RT / 2), warp = (tid >> 5) % (RT / 64), E = p.r.experts, t0 = blockIdx.x * TOK, nt = min(TOK, p.M - t0);
     float* xs = sm;
     float* z = sm + TOK * kc;
-    float* gs = z + TOK * E;
-    for (int i = tid; i < TOK * E; i += NT) z[i] = 0.0f;
+    float* gs = z + 2 * TOK * E;
+    for (int i = tid; i < 2 * TOK * E; i += RT) z[i] = 0.0f;
     const bool vec = p.d % 4 == 0;
     for (int k0 = 0; k0 < p.r.ld; k0 += kc) {                // all columns at once where they fit
         __syncthreads();
@@ -60,17 +61,17 @@ __global__ void __launch_bounds__(NT) route_rows_kernel(const RouteRows p, int k
             const float* x = p.x + (size_t)(t0 + t) * p.d;
             if (vec) {
 #pragma unroll 4
-                for (int k = tid * 4; k < kc; k += NT * 4)
+                for (int k = tid * 4; k < kc; k += RT * 4)
                     *(float4*)(xs + t * kc + spot(k)) = t < nt && k0 + k < p.d ? *(const float4*)(x + k0 + k) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             } else {
-                for (int k = tid; k < kc; k += NT) xs[t * kc + spot(k)] = t < nt && k0 + k < p.d ? x[k0 + k] : 0.0f;
+                for (int k = tid; k < kc; k += RT) xs[t * kc + spot(k)] = t < nt && k0 + k < p.d ? x[k0 + k] : 0.0f;
             }
         }
         __syncthreads();
-        for (int e0 = warp * EPW; e0 < E; e0 += NT / 32 * EPW) {
+        for (int e0 = warp * EPW; e0 < E; e0 += RT / 64 * EPW) {
             float s[EPW * TOK] = {};
 #pragma unroll 2
-            for (int c = 0; c < kc; c += 256) {
+            for (int c = half * 256; c < kc; c += 512) {          // the halves of the block take turns
                 const int k = k0 + c + lane * 8;
                 uint4 w[EPW];
 #pragma unroll
@@ -85,12 +86,14 @@ __global__ void __launch_bounds__(NT) route_rows_kernel(const RouteRows p, int k
             }
             static_assert(EPW * TOK == 32, "a sum a lane");
             const float v = warp_sums32(s);
-            if (e0 + lane / TOK < E) z[(lane % TOK) * E + e0 + lane / TOK] += v;
+            if (e0 + lane / TOK < E) z[(half * TOK + lane % TOK) * E + e0 + lane / TOK] += v;
         }
     }
     __syncthreads();
+    for (int i = tid; i < TOK * E; i += RT) z[i] += z[TOK * E + i];
+    __syncthreads();
     const int t = warp;
-    if (t < nt)
+    if (half == 0 && t < nt)
         choose(z + t * E, gs + t * p.r.groups, p.r, [&](int k, int e, float w) {
             const size_t at = (size_t)(t0 + t) * p.r.top + k;
             p.expert[at] = e;
@@ -153,10 +156,10 @@ int max_row_tiles(const Router& r, int M, int tile_rows) {
 int launch_route_rows(const RouteRows& p, const void* plane, bool f32_rows, cudaStream_t st) {
     const Router& r = p.r;
     if (r.experts > kMaxExperts || r.groups > kMaxGroups || r.top > 64) return fail(FC_E_SHAPE, "%d experts in %d groups, %d chosen", r.experts, r.groups, r.top);
-    const int rest = TOK * (r.experts + r.groups) * 4, kc = std::min(pad_to(r.ld, 256), (200 * 1024 - rest) / (TOK * 4) / 256 * 256);
+    const int rest = TOK * (2 * r.experts + r.groups) * 4, kc = std::min(pad_to(r.ld, 256), (200 * 1024 - rest) / (TOK * 4) / 256 * 256);
     const size_t smem = (size_t)TOK * kc * 4 + rest;
     if (smem > 47 * 1024) FC_CUDA(cudaFuncSetAttribute(route_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    route_rows_kernel<<<(p.M + TOK - 1) / TOK, NT, smem, st>>>(p, kc);
+    route_rows_kernel<<<(p.M + TOK - 1) / TOK, RT, smem, st>>>(p, kc);
     FC_LAUNCHED();
     gather_rows_kernel<<<p.M, NT, (size_t)r.experts * sizeof(int), st>>>(p, (const unsigned char*)plane, p.ld * (f32_rows ? 4 : 2) / 16);
     FC_LAUNCHED();

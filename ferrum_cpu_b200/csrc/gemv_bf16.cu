@@ -80,7 +80,7 @@ template <int MODE, int LAY>
 __global__ void __launch_bounds__(NT, 1) gemv_bf16_group_kernel(const __grid_constant__ GemvGroup g, int x_cap) {
     extern __shared__ __align__(16) float sm[];    // staged input [x_cap] | h [d] | token-shift row [d]; or expert logits behind xs
     __shared__ float2 red[NW];
-    __shared__ unsigned sum_at[LAY == kSum ? kSumChunks : 1];      // where 256 weights of a row begin, in 64s
+    __shared__ unsigned sum_at[LAY == kSum ? kSumChunks : 1];      // where 256 weights of a row begin, in 64s, times 8; plus how many 64s
     __shared__ int chosen[MODE == kChoose ? kMaxChosen : 1];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, d = g.d;
     float* xs = sm;
@@ -132,8 +132,8 @@ __global__ void __launch_bounds__(NT, 1) gemv_bf16_group_kernel(const __grid_con
             const uint16_t* src = base + (size_t)(warp + ri * NW) * ldw + lane * 8;
 #pragma unroll
             for (int c = 0; c < 8; ++c) {
-                const int ci = c0 + c;
-                p.w[c] = i < items && ci < chunks && lane * 8 + ci % per_rep * 256 < K_pad ? ld_stream(src + (size_t)sum_at[ci] * 64) : make_uint4(0, 0, 0, 0);
+                const unsigned at = c0 + c < chunks ? sum_at[c0 + c] : 0;
+                p.w[c] = i < items && lane < (int)(at & 7) * 8 ? ld_stream(src + (size_t)(at >> 3) * 64) : make_uint4(0, 0, 0, 0);
             }
         } else if constexpr (L == 3) {
             const int ri = i / pieces, k0 = (i - ri * pieces) * PIECE + lane * 8;
@@ -188,7 +188,10 @@ __global__ void __launch_bounds__(NT, 1) gemv_bf16_group_kernel(const __grid_con
             if constexpr (LAY == kSum) {
                 const GemvSeg& s = g.seg[0];
                 const int n = (s.K_pad + 255) / 256;
-                for (int i = tid; i < s.reps * n; i += NT) sum_at[i] = (unsigned)((size_t)__ldcg(g.expert + i / n) * s.w_step / 64) + i % n * 4;
+                for (int i = tid; i < s.reps * n; i += NT) {
+                    const int r = i / n, c = i - r * n;
+                    sum_at[i] = ((unsigned)((size_t)__ldcg(g.expert + r) * (s.w_step / 64)) + c * 4) * 8 + min(4, s.K_pad / 64 - c * 4);
+                }
                 __syncthreads();
                 continue;
             }

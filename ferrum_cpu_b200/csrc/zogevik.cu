@@ -141,6 +141,7 @@ int Zogevik::parse(const Json& j) {
         }
         if (c.experts % c.groups || c.keep > c.groups || c.top > c.experts / c.groups * c.keep)
             return fail(FC_E_DIM, "config.json: %s: %d of %d experts cannot be chosen from %d of %d equal groups", at.c_str(), c.top, c.experts, c.keep, c.groups);
+        if ((int64_t)c.experts * width * pad_to(c.ff, 64) >= (int64_t)1 << 35) return fail(FC_E_SHAPE, "%s: experts of more than 2^35 weights", at.c_str());
         if (c.top > kMaxTop) return fail(FC_E_SHAPE, "%s: a token uses at most %d experts", at.c_str(), kMaxTop);
     }
     return FC_OK;
