@@ -19,10 +19,10 @@ CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libferrum_cuda.so")
 # what every decoder of a model folder needs, and what each design adds
-FOLDER = ["common.cu", "model_dir.cpp", "decoder.cu", "gemm_bf16.cu", "gemv_bf16.cu", "flash_tc.cu", "flash_f32.cu", "llama_ops.cu", "sample.cu"]
+FOLDER = ["common.cu", "codec.cpp", "model_dir.cpp", "decoder.cu", "gemm_bf16.cu", "gemv_bf16.cu", "flash_tc.cu", "flash_f32.cu", "llama_ops.cu", "sample.cu"]
 NURINEX = ["mix_rows.cu", "talk_attn.cu", "wkv.cu", "mixer_decode.cu", "nurinex.cu"]
 ZOGEVIK = ["post_norm_rows.cu", "rot_attn.cu", "attn_decode.cu", "experts.cu", "zogevik.cu"]
-SOURCES = ["codec.cpp", "gguf_load.cpp", "gemv.cu", "gemv_stream.cu", "rowops.cu", "attn.cu", "gemm_simt.cu", "gemm_tc.cu", "attn_tc.cu",
+SOURCES = ["gguf_load.cpp", "gemv.cu", "gemv_stream.cu", "rowops.cu", "attn.cu", "gemm_simt.cu", "gemm_tc.cu", "attn_tc.cu",
            "decode_mega.cu", "decode_batch.cu", "llama.cu", "rowq.cu", "ggml_linear.cu", "api.cu"] + FOLDER + NURINEX + ZOGEVIK
 COMPONENTS = {"nurinex": FOLDER + NURINEX, "zogevik": FOLDER + ZOGEVIK}
 NVCC_FLAGS = [

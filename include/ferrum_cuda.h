@@ -457,16 +457,22 @@ float fc_llama_last_decode_ms(const fc_llama_cache* c);
 /* The architecture a folder's config.json names ("architecture"), for choosing the model class. */
 int fc_model_dir_architecture(const char* dir, char* out, int cap);
 
-/* Nurinex: a decoder whose layers put attention (scores mixed across heads, learned distance bias, sink, query
- * temperature, normed values), a linear-attention recurrence with per-channel decay (RWKV form) and a dense feed-forward
- * side by side on one norm. No counterpart in the reference; it is served as the imported models are. Every size and
- * constant comes from the folder's config.json; a layer may use another layer's tensors. Weights are bf16 and stay so.
- * math_mode: FC_MATH_BF16 (bf16 operands and caches; norms, scores, softmax, decays, recurrence and the residual are f32)
- * or FC_MATH_FP32 (f32 everywhere, caches too). ctx: positions a cache holds. */
+/* Decoders whose model is such a folder. The design is the one the configuration names; every size and constant comes from
+ * there. No counterparts in the reference; they are served as the imported models are.
+ *   Nurinex: layers that put attention (scores mixed across heads, learned distance bias, sink, query temperature, normed
+ *   values), a linear-attention recurrence with per-channel decay (RWKV form) and a dense feed-forward side by side on one
+ *   norm; a layer may use another layer's tensors.
+ *   Zogevik: windowed attention with rotary positions, either latent (one cached latent row and rotated key part per token) or
+ *   grouped-query (normed queries and keys, one added to the softmax denominator; a layer may use another's cached keys and
+ *   values), and feed-forwards of routed experts; sublayers read the residual as it is and their output is normed.
+ * Weights are bf16 and stay so. math_mode: FC_MATH_BF16 (bf16 operands and caches; norms, positions, scores, softmax, routers,
+ * decays, recurrences and the residual are f32) or FC_MATH_FP32 (f32 everywhere, caches too). ctx: positions a cache holds. */
 typedef struct fc_decoder fc_decoder;
-typedef struct fc_decoder_cache fc_decoder_cache;   /* key / value rows, recurrence states, token-shift rows, position */
+typedef struct fc_decoder_cache fc_decoder_cache;   /* what one sequence holds: cached rows, states, position */
 typedef struct fc_decoder_info {
-    int32_t vocab, width, n_layers, n_own_layers, ctx, pad;
+    int32_t vocab, width, n_layers;
+    int32_t n_own_layers;   /* layers with tensors (Nurinex) or keys and values (Zogevik) of their own */
+    int32_t ctx, pad;
     int64_t weight_bytes;   /* bytes of matrices one decoded token reads */
 } fc_decoder_info;
 /* Validates a folder without a GPU. */

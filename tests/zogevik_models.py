@@ -38,6 +38,11 @@ def configs():
             LAT(heads=20, dim=80, rot=32, rank=328, vdim=72, window=90, mlp=MOE(40, 9, 136, 8, 5)),
             ATT(heads=36, kv_heads=2, dim=72, vdim=100, rot=48, window=130, mlp=MOE(65, 4, 72, 13, 6)),
         ]),
+        # more experts than are ranked by counting
+        "many": MD.zogevik_config(120, 48, [
+            ATT(heads=2, kv_heads=2, dim=16, vdim=24, rot=4, window=31, mlp=MOE(150, 6, 24, 5, 3)),
+            LAT(heads=2, dim=16, rot=4, rank=24, vdim=16, window=45, mlp=MOE(140, 30, 16)),
+        ]),
         # query tiles too wide to stay in shared memory, value heads of four chunks, nothing masked but the future
         "huge": MD.zogevik_config(150, 64, [
             ATT(heads=2, kv_heads=1, dim=520, vdim=256, rot=130, window=None, mlp=MOE(3, 2, 520)),
