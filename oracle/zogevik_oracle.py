@@ -46,7 +46,7 @@ def rotate_halves(x, ang):
 
 
 def visible(i, window):
-    """Positions that position i sees: itself and the window - 1 before it (None: all)."""
+    """The last `window` positions up to i, i included (None: all of them)."""
     return np.arange(0 if window is None else max(0, i - window + 1), i + 1)
 
 

@@ -27,7 +27,7 @@ def test_rotations_turn_pairs_and_keep_distances():
         assert np.allclose(dots, dots[0]) and not np.isclose(dots[0], q @ k)
 
 
-def test_windows_hold_the_token_itself_and_those_before_it():
+def test_windows_end_with_the_token():
     assert ZO.visible(5, 1).tolist() == [5]
     assert ZO.visible(5, 3).tolist() == [3, 4, 5]
     assert ZO.visible(2, 3).tolist() == [0, 1, 2] and ZO.visible(1, 3).tolist() == [0, 1]
